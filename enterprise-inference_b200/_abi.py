@@ -30,7 +30,8 @@ class StackLayer(C.Structure):
                [(n, C.c_int32) for n in ("kv_rank", "rot_dim", "mixer_flags")] + [("gate_cap", C.c_float)] + \
                [(n, C.c_int32) for n in ("act", "ungated", "sigmoid_scores", "weight_input", "shared_ff")] + \
                [(n, C.c_int32) for n in ("window", "q_rank", "kv_share", "conv_taps", "decay_rank", "gate_rank", "norm_groups")] + \
-               [("act_limit", C.c_float), ("route_chosen", C.c_int32)]
+               [("act_limit", C.c_float), ("route_chosen", C.c_int32), ("softcap", C.c_float)] + \
+               [(n, C.c_int32) for n in ("bias_dist", "side", "side_inner", "side_state", "side_rank", "side_taps", "loop_add", "loop_step")]
 
 
 class StackCfg(C.Structure):
@@ -42,25 +43,29 @@ class StackCfg(C.Structure):
                 ("residual_mult", C.c_float)]
 
 
-MIXER_ATTENTION, MIXER_LATENT, MIXER_MLSTM, MIXER_DELTA, MIXER_SSD = 1, 2, 3, 4, 5
+MIXER_ATTENTION, MIXER_LATENT, MIXER_MLSTM, MIXER_DELTA, MIXER_SSD, MIXER_RETENTION, MIXER_SELECTIVE = 1, 2, 3, 4, 5, 6, 7
 MLP_NONE, MLP_MOE, MLP_DENSE = 0, 1, 2
 ACT_SILU, ACT_GELU_TANH, ACT_RELU2, ACT_RELU, ACT_SWIGLU_CLAMP, ACT_POLYNORM = 0, 1, 2, 3, 4, 5
 ACTS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "relu2": ACT_RELU2, "relu": ACT_RELU, "swiglu_clamp": ACT_SWIGLU_CLAMP,
         "polynorm": ACT_POLYNORM}
-FORM_SANDWICH, FORM_PARALLEL, FORM_POSTNORM, FORM_HYPER = 0, 1, 2, 3
+FORM_SANDWICH, FORM_PARALLEL, FORM_POSTNORM, FORM_HYPER, FORM_LOOPED = 0, 1, 2, 3, 4
 MIXF_SINK, MIXF_GATE, MIXF_HEAD_NORM, MIXF_VALUE_IS_KEY, MIXF_SINK_ONE, MIXF_HEAD_GATE = 1, 2, 4, 8, 16, 32
-MIXF_ROT_HALF, MIXF_NO_QK_NORM, MIXF_HEAD_DECAY = 64, 128, 256
+MIXF_ROT_HALF, MIXF_NO_QK_NORM, MIXF_HEAD_DECAY, MIXF_QKV_BIAS = 64, 128, 256, 512
 MAX_STREAMS = 8
 (SW_EMBED, SW_FINAL_NORM, SW_HEAD, SW_NORM_MIX_PRE, SW_NORM_MIX_POST, SW_NORM_MLP_PRE, SW_NORM_MLP_POST, SW_QKV, SW_Q_NORM,
  SW_K_NORM, SW_O, SW_ROUTER, SW_ROUTER_BIAS, SW_EXPERT_GATE_UP, SW_EXPERT_DOWN, SW_BIGRAM, SW_CANON, SW_DEPTH_AVG, SW_UK_T, SW_UV,
  SW_SINK, SW_GATES, SW_GATES_BIAS, SW_HEAD_NORM, SW_MLP_GATE_UP, SW_MLP_DOWN, SW_SHARED_UP, SW_SHARED_DOWN, SW_NORM_MIX_POST_BIAS,
  SW_NORM_MLP_POST_BIAS, SW_FINAL_NORM_BIAS, SW_Q_LATENT_NORM, SW_UQ, SW_CONV, SW_DECAY_UP, SW_DECAY_BIAS, SW_DECAY_LOG,
  SW_GATE_UP, SW_MLP_GATE_UP_INTERLEAVED, SW_NORM_MIX_PRE_BIAS, SW_NORM_MLP_PRE_BIAS, SW_SCALE_MIX, SW_SCALE_MLP, SW_HC_MIX, SW_HC_MLP,
- SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT) = range(49)
+ SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT, SW_EMBED_NORM, SW_LOOP_STEP, SW_QKV_BIAS, SW_DIST_BIAS, SW_DECAY, SW_SIDE_CONV,
+ SW_SIDE_CONV_BIAS, SW_SIDE_PROJ, SW_SIDE_DT, SW_SIDE_DT_BIAS, SW_SIDE_A, SW_SIDE_SKIP, SW_SIDE_O, SW_OUT_MAIN, SW_OUT_SIDE,
+ SW_MLP_UP_BIAS, SW_MLP_DOWN_BIAS) = range(66)
 SW_F32 = {SW_FINAL_NORM, SW_NORM_MIX_PRE, SW_NORM_MIX_POST, SW_NORM_MLP_PRE, SW_NORM_MLP_POST, SW_Q_NORM, SW_K_NORM, SW_ROUTER_BIAS,
           SW_CANON, SW_DEPTH_AVG, SW_SINK, SW_GATES_BIAS, SW_HEAD_NORM, SW_NORM_MIX_POST_BIAS, SW_NORM_MLP_POST_BIAS,
           SW_FINAL_NORM_BIAS, SW_Q_LATENT_NORM, SW_CONV, SW_DECAY_BIAS, SW_DECAY_LOG, SW_NORM_MIX_PRE_BIAS, SW_NORM_MLP_PRE_BIAS,
-          SW_SCALE_MIX, SW_SCALE_MLP, SW_HC_MIX, SW_HC_MLP, SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT}
+          SW_SCALE_MIX, SW_SCALE_MLP, SW_HC_MIX, SW_HC_MLP, SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT,
+          SW_EMBED_NORM, SW_LOOP_STEP, SW_DIST_BIAS, SW_DECAY, SW_SIDE_CONV, SW_SIDE_CONV_BIAS, SW_SIDE_DT_BIAS, SW_SIDE_A, SW_SIDE_SKIP,
+          SW_OUT_MAIN, SW_OUT_SIDE}
 
 W_EMBED, W_LN1, W_QKV, W_QKV_BIAS, W_O, W_LN2, W_GATE_UP, W_DOWN, W_FINAL_NORM, W_LM_HEAD, W_GATE_UP_INTERLEAVED = range(11)
 
@@ -188,6 +193,21 @@ SIGNATURES = {
     "b200_linear_scan": (C.c_int, [_i32, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32,
                                    _vp]),
     "b200_head_norm_gate_act": (C.c_int, [_i32, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _f32, _i32, _vp]),
+    "b200_rms_sandwich": (C.c_int, [_i32, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _f32, _vp]),
+    "b200_retention_step": (C.c_int, [_i32, _vp, _i64, _vp, _i32, _i32, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _f32,
+                                      _i32, _vp]),
+    "b200_retention_chunk_supported": (C.c_int, [_i32, _i32]),
+    "b200_retention_chunk_workspace_bytes": (_i64, [_i32, _i32, _i32, _i32, _i32]),
+    "b200_retention_chunk": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _f32,
+                                       _i32, _vp, _vp]),
+    "b200_conv_inputs": (C.c_int, [_i32, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32,
+                                   _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
+    "b200_selective_rows": (_i32, [_i32, _i32]),
+    "b200_selective_scan": (C.c_int, [_i32, _vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32,
+                                      _vp]),
+    "b200_paged_attn_biased": (C.c_int, [_i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32,
+                                         _f32, _vp, _i32, _vp, _i64, _vp, _i32, _vp, _vp]),
+    "b200_linear_bias_act": (C.c_int, [_i32, _i32, _vp, _i64, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _i64, _vp]),
     "b200_ssd_prep": (C.c_int, [_i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32,
                                 _i32, _i32, _i32, _vp]),
     "b200_ssd_gate_norm": (C.c_int, [_i32, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp]),

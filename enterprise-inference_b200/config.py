@@ -203,6 +203,11 @@ class AttentionSpec:
     sink_one: bool = False                 # one more unit in the softmax denominator
     qk_norm: bool = True                   # False: plain q/k/v projections, no norm of q and k at all
     rot_half: bool = False                 # rotated dimension i pairs with i + rot.dims / 2 (else 2i with 2i + 1)
+    bias: bool = False                     # q, k and v projections have biases
+    conv: int = 0                          # taps of a causal per-channel convolution over q, k and v (0: none)
+    softcap: float = 0.0                   # scores: softcap * tanh(score / softcap) (0: none)
+    bias_max: float = 0.0                  # > 0: a learned bias by distance joins the score, one table row from this distance on
+    head_gate: bool = False                # one sigmoid gate per head, read from the mixer's input
     sink: bool = False                     # a learned per-head term exp(sink) in the softmax denominator
 
 
@@ -217,8 +222,9 @@ class MoESpec:
 
 @dataclass
 class StackLayerSpec:
-    mixer: object                     # AttentionSpec | LatentAttentionSpec | ChannelDeltaSpec | HeadDeltaSpec | StateSpaceSpec
+    mixer: object                     # AttentionSpec | LatentAttentionSpec | ChannelDeltaSpec | HeadDeltaSpec | StateSpaceSpec | RetentionSpec
     mlp: Optional[object] = None      # MoESpec | FeedForwardSpec
+    side: Optional[object] = None     # SelectiveScanSpec: a second mixer that reads the same input; the results are normed and averaged
 
 
 @dataclass
@@ -348,6 +354,7 @@ class FeedForwardSpec:
     gated: Optional[bool] = None           # None: the design's default shape (dense gated, experts ungated)
     limit: float = 0.0                     # act "swiglu_clamp": min(gate, limit) * sigmoid(1.702 gate) * (clamp(up, +-limit) + 1)
     router: str = ""                       # "chosen_softmax": bias inside the logits, weights = softmax over the chosen logits
+    bias: bool = False                     # dense: both projections have biases
 
 
 @dataclass
@@ -728,6 +735,170 @@ class RudolixConfig:
                              streams=streams, residual_mult=float(c.get("residual_mult", 1.0)), layers=layers)
 
 
+# ---- Bofusun ----------------------------------------------------------------------------------------------------------------
+@dataclass
+class RetentionSpec:
+    """Linear attention with a fixed decay per head: `heads` heads of key size `dim` and value size `vdim`, rotated q and k, unit-RMS
+    read-out times silu of a gate projection."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float] = field(default_factory=list)
+    rot: Optional[RotarySpec] = None
+    rot_half: bool = True
+    kind: str = "retention"
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+
+@dataclass
+class SelectiveScanSpec:
+    """Selective scan (Mamba): `inner` channels with `state` states each, step sizes through a projection of rank `dt_rank`, a causal
+    convolution of `conv` taps with bias over the channels."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+    kind: str = "selective"
+
+    @property
+    def dt_pad(self) -> int:
+        return (self.dt_rank + 7) // 8 * 8
+
+    @property
+    def proj_rows(self) -> int:
+        """Rows of the projection to dt | B | C, dt and the total padded to multiples of 8 (b200_selective_rows)."""
+        return (self.dt_pad + 2 * self.state + 7) // 8 * 8
+
+
+@dataclass
+class BofusunConfig:
+    """Bofusun: decoder-only, RMS norms before and after every sublayer with weights stored around zero, a normed embedding, and a run
+    of layers that is passed several times with the same weights (each pass with its own cache and state; ahead of every pass but the
+    first the embedding output is added again, ahead of every pass a learned vector).  Mixers: retention; attention beside a selective
+    scan (grouped-query attention with biased, convolved q/k/v, a sliding window, capped scores, a learned bias by distance and one
+    gate per head), whose normed results are averaged.  Feed-forwards: dense with biases and squared relu."""
+    name: str = "bofusun"
+    width: int = 256
+    vocab: int = 1024
+    norm_eps: float = 1e-5
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0                    # 0: no loop
+    layers: List[StackLayerSpec] = field(default_factory=list)
+    architecture: str = "Bofusun"
+    embed_scale: float = 1.0
+
+    @property
+    def hidden(self) -> int:
+        return self.width
+
+    def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
+        """(layer, pass) in the order they run; pass is None outside the loop."""
+        n = len(self.layers)
+        if self.loop_times <= 0:
+            return [(i, None) for i in range(n)]
+        a, b = self.loop_start, self.loop_stop
+        return [(i, None) for i in range(a)] + [(i, t) for t in range(self.loop_times) for i in range(a, b)] + [(i, None) for i in range(b, n)]
+
+    @property
+    def n_layers(self) -> int:
+        """Layer runs: every pass of a looped layer counts, with a cache and a state of its own."""
+        return len(self.layer_runs())
+
+    @property
+    def needs_state(self) -> bool:
+        return True
+
+    def to_dict(self):
+        return asdict(self)
+
+    def _layer_params(self, L) -> int:
+        W, a, s = self.width, L.mixer, L.side
+        if isinstance(a, RetentionSpec):
+            n = 2 * W * a.heads * (a.dim + a.vdim) + a.heads * a.vdim * W
+        else:
+            n = W * (a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + (a.heads if a.head_gate else 0)) + a.heads * a.vdim * W
+        if s is not None:
+            n += 3 * W * s.inner + s.inner * (s.proj_rows + s.dt_pad)
+        if L.mlp is not None:
+            n += 2 * L.mlp.ff * W
+        return n
+
+    def decode_params(self) -> int:
+        """Weights one decode row multiplies (a looped layer counts in every pass)."""
+        return self.vocab * self.width + sum(self._layer_params(self.layers[i]) for i, _ in self.layer_runs())
+
+    def weight_bytes(self) -> int:
+        return 2 * (2 * self.vocab * self.width + sum(self._layer_params(L) for L in self.layers))
+
+    def kv_bytes_per_token(self, f32: bool = False) -> int:
+        n = 0
+        for i, _ in self.layer_runs():
+            a = self.layers[i].mixer
+            if isinstance(a, AttentionSpec):
+                n += a.kv_heads * (a.dim + a.vdim)
+        return n * (4 if f32 else 2)
+
+    @staticmethod
+    def _attention(m: dict, where: str) -> AttentionSpec:
+        a = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]),
+                          scale=float(m["scale"]), window=int((m.get("mask") or {}).get("size") or 0), qk_norm=False, bias=True,
+                          conv=int(m.get("conv") or 0), softcap=float(m.get("softcap") or 0.0), bias_max=float(m.get("bias_max") or 0.0), head_gate=True)
+        if a.heads % a.kv_heads:
+            raise ValueError(f"{where}: {a.heads} heads over {a.kv_heads} key heads")
+        return a
+
+    @staticmethod
+    def from_dict(c: dict, name: str = "bofusun") -> "BofusunConfig":
+        layers = []
+        for i, l in enumerate(c["layers"]):
+            kind, m, side = l.get("type"), l["mixer"], None
+            if kind == "retention":
+                rot, r = None, m.get("rot")
+                if r and int(r.get("dims") or 0) > 0:
+                    rot = RotarySpec(base=float(r["base"]), dims=int(r["dims"]))
+                    if rot.dims % 2 or rot.dims > int(m["dim"]):
+                        raise ValueError(f"layer {i}: {rot.dims} rotated dimensions in heads of {m['dim']}")
+                mixer = RetentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]), decay=[float(d) for d in m["decay"]], rot=rot)
+                if len(mixer.decay) != mixer.heads:
+                    raise ValueError(f"layer {i}: {len(mixer.decay)} decays for {mixer.heads} heads")
+            elif kind == "parallel":
+                mixer = BofusunConfig._attention(m["left"], f"layer {i}")
+                b = m["right"]
+                side = SelectiveScanSpec(inner=int(b["inner"]), state=int(b["state"]), dt_rank=int(b["dt_rank"]), conv=int(b.get("conv") or 1))
+            else:
+                raise ValueError(f"layer {i}: unsupported mixer type {kind!r} (this design has retention, parallel)")
+            mlp, f = None, l.get("mlp")
+            if f:
+                if f.get("kind", "dense") != "dense":
+                    raise ValueError(f"layer {i}: unsupported feed-forward kind {f.get('kind')!r}")
+                mlp = FeedForwardSpec(kind="dense", ff=int(f["ff"]), act="relu2", gated=False, bias=True)
+            layers.append(StackLayerSpec(mixer=mixer, mlp=mlp, side=side))
+        loop = c.get("loop") or {}
+        start, stop, times = int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 0))
+        if loop and not (0 <= start < stop <= len(layers) and times >= 1):
+            raise ValueError(f"loop over layers {start} .. {stop - 1} of {len(layers)}, {times} times")
+        return BofusunConfig(name=name, width=int(c["width"]), vocab=int(c["vocab"]), norm_eps=float((c.get("norm") or {}).get("eps", 1e-5)),
+                             loop_start=start, loop_stop=stop, loop_times=times, layers=layers)
+
+
+def distance_bucket(n: int, rows: int, far: float) -> int:
+    """Row of a learned distance table: the distance itself below rows / 2, then logarithmic, the last row from `far` on."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
+
+
+def distance_entries(window: int, far: float) -> int:
+    """Distances that need an entry of their own: what the window shows, and no further than the distance the last row starts at."""
+    n = math.ceil(far) + 1
+    return min(n, window) if window > 0 else n
+
+
 def checkpoint_shapes(path: str) -> Dict[str, list]:
     """Tensor name -> shape of every *.safetensors file under `path`, from the files' headers alone (8-byte little-endian
     length, then that many bytes of JSON)."""
@@ -746,7 +917,7 @@ def checkpoint_shapes(path: str) -> Dict[str, list]:
 
 # config.json "architecture" -> reader.  HF-style configs (model_type) go through from_hf_config.
 ARCHITECTURES = {"Bopilorn": BopilornConfig.from_dict, "Dupolorn": DupolornConfig.from_dict, "Futidra": FutidraConfig.from_dict,
-                 "Rudolix": RudolixConfig.from_dict}
+                 "Rudolix": RudolixConfig.from_dict, "Bofusun": BofusunConfig.from_dict}
 NEEDS_SHAPES = {"Futidra"}   # readers that take the checkpoint's tensor shapes for sizes config.json does not name
 
 

@@ -1,6 +1,6 @@
 // Paged causal softmax attention (optionally over a sliding window of the last `window` keys) for heads of any size
 // (query/key size `dim`, value size `vdim`, dim != vdim allowed),
-// any block size, a caller-given score scale, fp32 queries and a bf16 or fp32 cache.  The tcgen05 kernels of attn_tc.cu /
+// any block size, a caller-given score scale (with an optional cap and a bias by distance: AttnExtra), fp32 queries and a bf16 or fp32 cache.  The tcgen05 kernels of attn_tc.cu /
 // attn_prefill.cu are built for 128-wide heads; this file serves every other head shape on CUDA cores with fp32 scores,
 // fp32 softmax weights and fp32 accumulation.
 //
@@ -52,7 +52,8 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
                        const int32_t* __restrict__ block_table, int bt_stride, const int32_t* __restrict__ row_to_seq,
                        const int32_t* __restrict__ ctx_lens, const int32_t* __restrict__ positions,
                        const float* __restrict__ vrot, int64_t max_pos, AT* __restrict__ out, int heads, int kv_heads,
-                       int dim, int vdim, int block_size, float scale, int kst, int vst, const float* __restrict__ sink, int window) {
+                       int dim, int vdim, int block_size, float scale, int kst, int vst, const float* __restrict__ sink, int window,
+                       AttnExtra ex) {
   extern __shared__ float sm[];
   float* qs = sm;                 // [dim]
   float* ps = qs + dim;           // [128] weights of the tile
@@ -66,6 +67,7 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
   const int ctx = ctx_lens[t];
   const int32_t* bt = block_table + (int64_t)(row_to_seq ? row_to_seq[t] : t) * bt_stride;
   for (int d = tid; d < dim; d += kAdThreads) qs[d] = q[((int64_t)t * heads + h) * dim + d];
+  const float* brow = ex.dist_bias ? ex.dist_bias + (int64_t)h * ex.bias_dist : nullptr;
   float m = -INFINITY, l = 0.f;
   float acc[kAdMaxVPer];
 #pragma unroll
@@ -81,7 +83,7 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
       const CT* kp = kc + (((int64_t)blk * kv_heads + g) * block_size + j % block_size) * kst;
       float a = 0.f;
       for (int d = 0; d < dim; ++d) a = fmaf(qs[d], cache_load<CT>(kp, d), a);
-      sc = a * scale;
+      sc = score_shape(a * scale, ex.softcap, brow, ctx - 1 - j, ex.bias_dist);
     }
     const float tm = block_max128(sc, red);
     const float mn = fmaxf(m, tm);
@@ -114,7 +116,8 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
 #pragma unroll
     for (int i = 0; i < kAdMaxVPer; ++i) acc[i] *= corr;
   }
-  const float inv = l > 0.f ? 1.0f / l : 0.f;
+  float inv = l > 0.f ? 1.0f / l : 0.f;
+  if (ex.gate) inv /= 1.0f + expf(-cache_load<AT>(static_cast<const AT*>(ex.gate), t * ex.ldg + h));
 #pragma unroll
   for (int i = 0; i < kAdMaxVPer; ++i) {
     const int d = tid + i * kAdThreads;
@@ -207,7 +210,8 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
                        const int32_t* __restrict__ ctx_lens, const int32_t* __restrict__ positions,
                        const float* __restrict__ vrot, int64_t max_pos, AT* __restrict__ out,
                        const int32_t* __restrict__ runs, const int32_t* __restrict__ n_runs, int heads, int kv_heads, int dim,
-                       int vdim, int block_size, float scale, int kcs, int vcs, const float* __restrict__ sink, int window) {
+                       int vdim, int block_size, float scale, int kcs, int vcs, const float* __restrict__ sink, int window,
+                       AttnExtra ex) {
   extern __shared__ float sm[];
   pdl_wait();
   pdl_launch_dependents();
@@ -267,7 +271,8 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
             const float* kp = Ks + lane * kst;
             float a = 0.f;
             for (int d = 0; d < dim; ++d) a = fmaf(qp[d], kp[d], a);
-            sc = a * scale;
+            const float* brow = ex.dist_bias ? ex.dist_bias + (int64_t)(g * G + qi % G) * ex.bias_dist : nullptr;
+            sc = score_shape(a * scale, ex.softcap, brow, ctx - 1 - j, ex.bias_dist);
           }
           const float mn = fmaxf(m[k], warp_max(sc));
           const float p = (j < ctx && j >= lo) ? expf(sc - mn) : 0.f;
@@ -303,7 +308,8 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
         osc = expf(m[k] - mn);
         lk = lk * osc + expf(sk - mn);
       }
-      const float inv = lk > 0.f ? osc / lk : 0.f;
+      float inv = lk > 0.f ? osc / lk : 0.f;
+      if (ex.gate) inv /= 1.0f + expf(-cache_load<AT>(static_cast<const AT*>(ex.gate), t * ex.ldg + g * G + hh));
       int pos = positions[t];
       pos = pos < 0 ? 0 : (pos >= max_pos ? (int)max_pos - 1 : pos);
       const float* cs = vrot ? vrot + (int64_t)pos * 2 * vhalf : nullptr;
@@ -338,7 +344,7 @@ template <typename CT, typename AT>
 static int paged_attn_anydim_t(const float* q, const void* kc, const void* vc, const int32_t* block_table, int bt_stride,
                                const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, const float* vrot,
                                int64_t max_pos, void* out, int T, int heads, int kv_heads, int dim, int vdim, int block_size,
-                               float scale, int plan, void* ws, cudaStream_t s, int kst, int vst, const float* sink, int window) {
+                               float scale, int plan, void* ws, cudaStream_t s, int kst, int vst, const float* sink, int window, const AttnExtra& ex) {
   const int G = heads / kv_heads;
   const size_t smem_runs = ((size_t)kTileKeys * (dim + 1 + vdim) + (size_t)kRunRows * G * (dim + vdim)) * 4;
   if (plan != 0 && ws != nullptr && kRunRows * G <= 16 * (kTcThreads / 32) && smem_runs <= 200 * 1024) {
@@ -349,13 +355,13 @@ static int paged_attn_anydim_t(const float* q, const void* kc, const void* vc, c
     if (smem_runs > 48 * 1024) B200_CUDA(ensure_dynamic_smem(paged_attn_runs_kernel<CT, AT>, 200 * 1024, done));
     B200_CUDA(launch(paged_attn_runs_kernel<CT, AT>, dim3(T, kv_heads), dim3(kTcThreads), smem_runs, s, q, (const CT*)kc,
                      (const CT*)vc, block_table, bt_stride, row_to_seq, ctx_lens, positions, vrot, max_pos, (AT*)out,
-                     (const int32_t*)runs, (const int32_t*)n_runs, heads, kv_heads, dim, vdim, block_size, scale, kst, vst, sink, window));
+                     (const int32_t*)runs, (const int32_t*)n_runs, heads, kv_heads, dim, vdim, block_size, scale, kst, vst, sink, window, ex));
     return B200_OK;
   }
   const size_t smem = ((size_t)dim + kAdThreads + vdim) * 4;
   B200_CUDA(launch(paged_attn_rows_kernel<CT, AT>, dim3(T, heads), dim3(kAdThreads), smem, s, q, (const CT*)kc, (const CT*)vc,
                    block_table, bt_stride, row_to_seq, ctx_lens, positions, vrot, max_pos, (AT*)out, heads, kv_heads, dim, vdim,
-                   block_size, scale, kst, vst, sink, window));
+                   block_size, scale, kst, vst, sink, window, ex));
   return B200_OK;
 }
 
@@ -364,17 +370,17 @@ static int paged_attn_anydim_t(const float* q, const void* kc, const void* vc, c
 int paged_attn_anydim(bool f32, const float* q, const void* kc, const void* vc, const int32_t* block_table, int bt_stride,
                       const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, const float* vrot,
                       int64_t max_pos, void* out, int T, int heads, int kv_heads, int dim, int vdim, int block_size, float scale,
-                      int plan, void* ws, cudaStream_t s, int kstride, int vstride, const float* sink, int window) {
+                      int plan, void* ws, cudaStream_t s, int kstride, int vstride, const float* sink, int window, const AttnExtra& ex) {
   if (T == 0) return B200_OK;
   const int kst = kstride > 0 ? kstride : dim, vst = vstride > 0 ? vstride : vdim;
   B200_REQUIRE(kst >= dim && vst >= vdim, B200_ERR_INVALID, "attention: cache rows of %d / %d elements for heads of %d / %d", kst, vst, dim, vdim);
   B200_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0, B200_ERR_INVALID, "attention: %d heads over %d kv heads", heads, kv_heads);
   B200_REQUIRE(vdim <= kAdThreads * kAdMaxVPer && dim <= 8192, B200_ERR_UNSUPPORTED, "attention: head sizes %d / %d too large", dim, vdim);
   return f32 ? paged_attn_anydim_t<float, float>(q, kc, vc, block_table, bt_stride, row_to_seq, ctx_lens, positions, vrot, max_pos,
-                                                 out, T, heads, kv_heads, dim, vdim, block_size, scale, plan, ws, s, kst, vst, sink, window)
+                                                 out, T, heads, kv_heads, dim, vdim, block_size, scale, plan, ws, s, kst, vst, sink, window, ex)
              : paged_attn_anydim_t<__nv_bfloat16, __nv_bfloat16>(q, kc, vc, block_table, bt_stride, row_to_seq, ctx_lens,
                                                                  positions, vrot, max_pos, out, T, heads, kv_heads, dim, vdim,
-                                                                 block_size, scale, plan, ws, s, kst, vst, sink, window);
+                                                                 block_size, scale, plan, ws, s, kst, vst, sink, window, ex);
 }
 
 }  // namespace b200

@@ -51,14 +51,15 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-template <int NG>   // 16-column output groups per warp: rank <= 128 NG
+// NG: 16-column output groups per warp (rank <= 128 NG).  EX: score cap, distance bias and per-head gate of AttnExtra.
+template <int NG, bool EX>
 __global__ void __launch_bounds__(kLaThreads)
 latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
                        int kv_heads, const int32_t* __restrict__ block_table,
                        int bt_stride, const int32_t* __restrict__ row_to_seq, const int32_t* __restrict__ ctx_lens,
                        __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ runs, const int32_t* __restrict__ n_runs, int heads,
                        int krow, int rank, int block_size, float scale, const float* __restrict__ sink, int n_splits,
-                       float* __restrict__ part, int window) {
+                       float* __restrict__ part, int window, AttnExtra ex) {
   extern __shared__ __align__(16) unsigned char smraw[];
   pdl_wait();
   pdl_launch_dependents();
@@ -160,8 +161,13 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
       const int row = warp * (kLaPairs / kLaWarps) + rr, c = ctxp[row], lo = lop[row];
       const int j0 = base + lane, j1 = j0 + 32;
       const bool see0 = j0 < c && j0 >= lo, see1 = j1 < c && j1 >= lo;
-      const float s0 = see0 ? Ss[row * kSsStride + lane] * scale : -INFINITY;
-      const float s1 = see1 ? Ss[row * kSsStride + lane + 32] * scale : -INFINITY;
+      float s0 = see0 ? Ss[row * kSsStride + lane] * scale : -INFINITY;
+      float s1 = see1 ? Ss[row * kSsStride + lane + 32] * scale : -INFINITY;
+      if constexpr (EX) {
+        const float* brow = ex.dist_bias ? ex.dist_bias + (int64_t)(g * G + (i0 + row) % G) * ex.bias_dist : nullptr;
+        if (see0) s0 = score_shape(s0, ex.softcap, brow, c - 1 - j0, ex.bias_dist);
+        if (see1) s1 = score_shape(s1, ex.softcap, brow, c - 1 - j1, ex.bias_dist);
+      }
       const float m_old = mrow[row];
       const float m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));
       float p0 = 0.f, p1 = 0.f, cr = 1.f;
@@ -250,7 +256,9 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
       osc = expf(m - mn);
       l = l * osc + expf(sk - mn);
     }
-    const float inv = l > 0.f ? osc / l : 0.f;
+    float inv = l > 0.f ? osc / l : 0.f;
+    if constexpr (EX)
+      if (ex.gate) inv /= 1.0f + expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(ex.gate)[t * ex.ldg + h]));
     __nv_bfloat16* dst = out + ((int64_t)t * heads + h) * rank;
 #pragma unroll
     for (int cg = 0; cg < NG; ++cg) {
@@ -273,7 +281,7 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
 constexpr int kLaMaxSplits = 16;
 __global__ void __launch_bounds__(128)
 latent_attn_merge_kernel(const float* __restrict__ part, __nv_bfloat16* __restrict__ out, int n_pairs, int heads, int rank, int n_splits,
-                         const float* __restrict__ sink) {
+                         const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int64_t ldg) {
   pdl_wait();
   pdl_launch_dependents();
   const int pair = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -286,7 +294,8 @@ latent_attn_merge_kernel(const float* __restrict__ part, __nv_bfloat16* __restri
   const float m = fmaxf(warp_max(mz), sk);
   const float ez = mz != -INFINITY ? expf(mz - m) : 0.f;
   const float l = warp_sum(lz * ez) + (sink ? expf(sk - m) : 0.f);
-  const float fz = l > 0.f ? ez / l : 0.f;
+  float fz = l > 0.f ? ez / l : 0.f;
+  if (gate) fz /= 1.0f + expf(-__bfloat162float(gate[(int64_t)(pair / heads) * ldg + pair % heads]));
   float f[kLaMaxSplits];
 #pragma unroll
   for (int z = 0; z < kLaMaxSplits; ++z) f[z] = __shfl_sync(0xffffffffu, fz, z);
@@ -336,7 +345,7 @@ bool paged_attn_mma_supported(int heads, int kv_heads, int dim, int vdim) {
 static int attn_mma_launch(const float* q, const __nv_bfloat16* kc, const __nv_bfloat16* vc, int kv_heads, const int32_t* block_table,
                            int bt_stride, const int32_t* row_to_seq, const int32_t* ctx_lens, __nv_bfloat16* out, const int32_t* runs,
                            const int32_t* n_runs, int T, int heads, int krow, int rank, int block_size, float scale, const float* sink,
-                           cudaStream_t s, int n_splits, float* part, int window) {
+                           cudaStream_t s, int n_splits, float* part, int window, const AttnExtra& ex) {
   if (n_splits < 1 || part == nullptr) n_splits = 1;
   B200_REQUIRE(n_splits <= kLaMaxSplits, B200_ERR_INVALID, "attention: %d splits (at most %d)", n_splits, kLaMaxSplits);
   B200_REQUIRE(reinterpret_cast<uintptr_t>(kc) % 16 == 0 && reinterpret_cast<uintptr_t>(vc) % 16 == 0, B200_ERR_INVALID,
@@ -344,20 +353,26 @@ static int attn_mma_launch(const float* q, const __nv_bfloat16* kc, const __nv_b
   const size_t smem = la_smem(krow, rank, vc != nullptr);
   // a run has at most 16 rows, so a kv head's group has at most 16 G pairs: G chunks of 16
   const dim3 grid(T, heads, n_splits), block(kLaThreads);
-#define LA(NGV)                                                                                                                     \
+#define LA2(NGV, EXV)                                                                                                               \
   do {                                                                                                                              \
     static bool done[64] = {};                                                                                                      \
-    if (smem > 48 * 1024) B200_CUDA(ensure_dynamic_smem(latent_attn_mma_kernel<NGV>, 200 * 1024, done));                            \
-    B200_CUDA(launch(latent_attn_mma_kernel<NGV>, grid, block, smem, s, q, kc, vc, kv_heads, block_table, bt_stride, row_to_seq, ctx_lens, \
-                     out, runs, n_runs, heads, krow, rank, block_size, scale, sink, n_splits, part, window));                       \
+    if (smem > 48 * 1024) B200_CUDA(ensure_dynamic_smem(latent_attn_mma_kernel<NGV, EXV>, 200 * 1024, done));                       \
+    B200_CUDA(launch(latent_attn_mma_kernel<NGV, EXV>, grid, block, smem, s, q, kc, vc, kv_heads, block_table, bt_stride, row_to_seq, \
+                     ctx_lens, out, runs, n_runs, heads, krow, rank, block_size, scale, sink, n_splits, part, window, ex));         \
+  } while (0)
+#define LA(NGV)                 \
+  do {                          \
+    if (ex.any()) LA2(NGV, true); \
+    else LA2(NGV, false);       \
   } while (0)
   if (rank <= 128) LA(1);
   else if (rank <= 256) LA(2);
   else LA(4);
 #undef LA
+#undef LA2
   if (n_splits > 1)
     B200_CUDA(launch(latent_attn_merge_kernel, dim3((T * heads + 3) / 4), dim3(128), (size_t)0, s, (const float*)part, out, T * heads, heads,
-                     rank, n_splits, sink));
+                     rank, n_splits, sink, static_cast<const __nv_bfloat16*>(ex.gate), ex.ldg));
   return B200_OK;
 }
 
@@ -368,19 +383,19 @@ int latent_attn_mma(const float* q, const __nv_bfloat16* kc, const int32_t* bloc
   if (T == 0) return B200_OK;
   B200_REQUIRE(latent_attn_mma_supported(heads, krow, rank), B200_ERR_UNSUPPORTED, "latent_attn_mma: shape %d / %d / %d", heads, krow, rank);
   return attn_mma_launch(q, kc, nullptr, 1, block_table, bt_stride, row_to_seq, ctx_lens, out, runs, n_runs, T, heads, krow, rank, block_size,
-                         scale, sink, s, n_splits, part, window);
+                         scale, sink, s, n_splits, part, window, AttnExtra());
 }
 
 // caches [block][kv_heads][block_size][dim | vdim] bf16, fp32 queries [T][heads][dim], bf16 output [T][heads][vdim]
 int paged_attn_mma(const float* q, const __nv_bfloat16* kc, const __nv_bfloat16* vc, const int32_t* block_table, int bt_stride,
                    const int32_t* row_to_seq, const int32_t* ctx_lens, __nv_bfloat16* out, const int32_t* runs, const int32_t* n_runs, int T,
                    int heads, int kv_heads, int dim, int vdim, int block_size, float scale, const float* sink, cudaStream_t s, int n_splits,
-                   float* part, int window) {
+                   float* part, int window, const AttnExtra& ex) {
   if (T == 0) return B200_OK;
   B200_REQUIRE(vc && paged_attn_mma_supported(heads, kv_heads, dim, vdim), B200_ERR_UNSUPPORTED, "paged_attn_mma: shape %d / %d / %d / %d", heads,
                kv_heads, dim, vdim);
   return attn_mma_launch(q, kc, vc, kv_heads, block_table, bt_stride, row_to_seq, ctx_lens, out, runs, n_runs, T, heads, dim, vdim, block_size,
-                         scale, sink, s, n_splits, part, window);
+                         scale, sink, s, n_splits, part, window, ex);
 }
 
 }  // namespace b200

@@ -100,6 +100,12 @@ __device__ __forceinline__ float gate_combine(float g, float u, int kind, float 
   return act_apply(g, kind) * u;
 }
 
+// a scaled attention score -> capped (cap > 0) and biased by the distance between query and key (bias_row: the head's entries, or null)
+__device__ __forceinline__ float score_shape(float s, float cap, const float* bias_row, int dist, int n_dist) {
+  if (cap > 0.f) s = cap * tanhf(s / cap);
+  return bias_row ? s + __ldg(bias_row + min(dist, n_dist - 1)) : s;
+}
+
 // ---- Programmatic dependent launch -------------------------------------------------------
 // Every kernel of the step waits for its predecessor's memory here and lets its successor
 // start its prologue early; with no PDL attribute on the launch both are no-ops.
@@ -221,6 +227,7 @@ struct LinearExtra {
   int hq = 0, hkv = 0, block_size = 0;
   float* out_f32 = nullptr;
   int act = 0;                   // mode 1: b200_act_kind of the gate (0: silu)
+  int post_act = 0;              // mode 0: 1 + b200_act_kind applied to the fp32 sum (bias included) before the rounding; 0: none
 };
 int linear_tc(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, const __nv_bfloat16* bias,
               __nv_bfloat16* y, int64_t ldy, int T, int n_out, int k, void* ws, int64_t ws_bytes,
@@ -310,12 +317,22 @@ int rotate_back_rows(const __nv_bfloat16* in, int in_stride, __nv_bfloat16* out,
                      int heads, int vdim, int64_t max_pos, cudaStream_t s);
 int convert_f32_to_bf16(const float* in, __nv_bfloat16* out, int64_t n, cudaStream_t s);
 int convert_bf16_to_f32(const __nv_bfloat16* in, float* out, int64_t n, cudaStream_t s);
+// What a score and an output row may take besides scale, window and sink: score cap, bias by distance, one sigmoid gate per head
+struct AttnExtra {
+  float softcap = 0.f;               // > 0: s = softcap tanh(s / softcap)
+  const float* dist_bias = nullptr;  // [heads][bias_dist] fp32, added after the cap: entry min(i - j, bias_dist - 1)
+  int bias_dist = 0;
+  const void* gate = nullptr;        // gate[t * ldg + h], activation type
+  int64_t ldg = 0;
+  bool any() const { return softcap > 0.f || dist_bias != nullptr || gate != nullptr; }
+};
 // paged softmax attention for any head sizes (attn_anydim.cu)
 int64_t paged_attn_anydim_workspace_bytes(int T);
 int paged_attn_anydim(bool f32, const float* q, const void* kc, const void* vc, const int32_t* block_table, int bt_stride,
                       const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, const float* vrot,
                       int64_t max_pos, void* out, int T, int heads, int kv_heads, int dim, int vdim, int block_size, float scale,
-                      int plan, void* ws, cudaStream_t s, int kstride = 0, int vstride = 0, const float* sink = nullptr, int window = 0);
+                      int plan, void* ws, cudaStream_t s, int kstride = 0, int vstride = 0, const float* sink = nullptr, int window = 0,
+                      const AttnExtra& ex = AttnExtra());
 // kstride / vstride: elements per cache row when they exceed dim / vdim (0: dim / vdim; the value cache may then be the key
 // cache itself, a value being the leading vdim entries of the row); sink [heads]: exp(sink[h]) joins the softmax denominator
 int paged_attn_runs_plan(const int32_t* row_to_seq, const int32_t* ctx_lens, int T, void* ws, cudaStream_t s);
@@ -330,7 +347,7 @@ bool paged_attn_mma_supported(int heads, int kv_heads, int dim, int vdim);
 int paged_attn_mma(const float* q, const __nv_bfloat16* kc, const __nv_bfloat16* vc, const int32_t* block_table, int bt_stride,
                    const int32_t* row_to_seq, const int32_t* ctx_lens, __nv_bfloat16* out, const int32_t* runs, const int32_t* n_runs, int T,
                    int heads, int kv_heads, int dim, int vdim, int block_size, float scale, const float* sink, cudaStream_t s,
-                   int n_splits = 1, float* part = nullptr, int window = 0);
+                   int n_splits = 1, float* part = nullptr, int window = 0, const AttnExtra& ex = AttnExtra());
 // context splits for a step (1: none); part holds T * heads * n_splits * (rank + 2) floats
 int latent_attn_splits(int T, int heads, int rank, int max_ctx, int64_t ws_bytes);
 // mixture of experts (moe.cu)
@@ -432,6 +449,28 @@ int delta_scan(const float* qn, const float* kn, const float* vn, const float* b
                int kv_heads, int dim, int vd, cudaStream_t s);
 // true-fp32 CUDA-core linear (linear_simt.cu)
 int linear_simt(bool x_f32, bool y_f32, const void* x, int64_t ldx, const __nv_bfloat16* w, void* y, int64_t ldy, int T, int n_out,
-                int k, cudaStream_t s);
+                int k, cudaStream_t s, const __nv_bfloat16* bias = nullptr, int act = -1);
+// looped layer form: RMS sandwich over the stream (rms_stream.cu), retention (retention.cu), convolved attention inputs and the
+// selective scan (selective.cu)
+int rms_sandwich(bool f32, float* x, const void* y, const void* y_b, const float* w_a, const float* w_b, const float* w_post, bool init,
+                 float* e_out, float* tap, const float* e, const float* step, const float* w_next, void* out, const int32_t* rows, int R,
+                 int width, float eps, cudaStream_t s);
+int retention_step(bool f32, const void* fused, int64_t ld, const float* rot, int rot_dims, bool half_layout, int64_t max_pos,
+                   const float* decay, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state,
+                   int64_t slot_stride, void* out, int S, int heads, int dim, int vdim, float eps, int max_rows, cudaStream_t s);
+bool retention_chunk_supported(int dim, int vdim);
+int64_t retention_chunk_workspace_bytes(int T, int S, int heads, int dim, int vdim);
+int retention_chunk(const void* fused, int64_t ld, const float* rot, int rot_dims, bool half_layout, int64_t max_pos, const float* decay,
+                    const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state, int64_t slot_stride, void* out,
+                    int T, int S, int heads, int dim, int vdim, float eps, int min_rows, void* ws, cudaStream_t s);
+int conv_inputs(bool f32, const void* fused, int64_t ld, const float* conv_a, int taps_a, float* tails_a, const float* conv_x, const float* bias_x,
+                int taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
+                const int32_t* seq_slots, const int32_t* slots, float* qout, void* kc, void* vc, void* xc, int T, int heads, int kv_heads,
+                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s);
+int selective_dt_pad(int rank);
+int selective_rows(int rank, int state);
+int selective_scan(bool f32, const void* xc, const void* bc, int64_t ldbc, int b_off, const float* dt_pre, const float* dt_bias, const float* A,
+                   const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
+                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, cudaStream_t s);
 
 }  // namespace b200

@@ -195,6 +195,7 @@ struct TcParams {
   const int32_t* grp_pair;
   const float* grp_wt;
   float* grp_out;
+  int post_act;          // kPlain: 1 + b200_act_kind applied to the fp32 sum before the rounding (0: none)
   int tile_n;            // N of the instantiation (kScatter: index of a token inside its tile)
 };
 
@@ -219,7 +220,7 @@ __device__ __forceinline__ void tc_trace(const TcParams& p, int slot) {
 }
 
 // Epilogue modes (template parameter):
-//  kPlain    y[t][row] = bf16(acc + bias)
+//  kPlain    y[t][row] = bf16(acc + bias), or bf16(act(acc + bias)) (TcParams::post_act)
 //  kSiluMul  the slab holds 64 gate rows then the 64 matching up rows (B200_W_GATE_UP_INTERLEAVED):
 //            y[t][m_tile*64 + i] = bf16(bf16(silu(bf16(g_i))) * bf16(u_i))          (R5)
 //            (TcParams::act != 0: bf16(act(bf16(g_i)) * bf16(u_i)) for the other gate activations)
@@ -236,6 +237,10 @@ __device__ __forceinline__ void finalize4(const TcParams& p, int m_tile, int lan
   const int r4 = lane * 4;
   float v[4] = {round_bf16(a.x + bb[0]), round_bf16(a.y + bb[1]), round_bf16(a.z + bb[2]), round_bf16(a.w + bb[3])};
   if constexpr (MODE == kPlain) {
+    if (p.post_act) {
+      v[0] = act_apply(a.x + bb[0], p.post_act - 1), v[1] = act_apply(a.y + bb[1], p.post_act - 1);
+      v[2] = act_apply(a.z + bb[2], p.post_act - 1), v[3] = act_apply(a.w + bb[3], p.post_act - 1);
+    }
     const int row = m_tile * kBlockM + r4;
     __nv_bfloat16* dst = p.y + (int64_t)tok * p.ldy + row;
     if (row + 3 < p.n_out && (p.ldy % 4 == 0) && ((reinterpret_cast<uintptr_t>(p.y) & 7) == 0)) {
@@ -1086,6 +1091,7 @@ int linear_tc(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, const
     p.grp_out = ex->out_f32;   // y[t][row] stays unrounded: row stride n_out
   } else {
     B200_REQUIRE(mode == kPlain, B200_ERR_INVALID, "linear_tc: unknown epilogue mode %d", mode);
+    if (ex) p.post_act = ex->post_act;
   }
   const bool ni = ex && ex->norm_in;
   if (ni) {

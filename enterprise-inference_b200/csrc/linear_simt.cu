@@ -21,7 +21,7 @@ template <> __device__ __forceinline__ void stf<__nv_bfloat16>(__nv_bfloat16* p,
 template <typename XT, typename YT>
 __global__ void __launch_bounds__(256)
 linear_simt_kernel(const XT* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, YT* __restrict__ y, int64_t ldy,
-                   int T, int n_out, int k) {
+                   int T, int n_out, int k, const __nv_bfloat16* __restrict__ bias, int act) {
   __shared__ float xs[kBK][kBM + 1];
   __shared__ float ws[kBK][kBN + 1];
   pdl_wait();
@@ -71,28 +71,32 @@ linear_simt_kernel(const XT* __restrict__ x, int64_t ldx, const __nv_bfloat16* _
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int r = m0 + ty * 4 + i, cidx = n0 + tx * 4 + j;
-      if (r < T && cidx < n_out) stf<YT>(y, (int64_t)r * ldy + cidx, acc[i][j]);
+      if (r < T && cidx < n_out) {
+        const float v = acc[i][j] + (bias ? __bfloat162float(bias[cidx]) : 0.f);
+        stf<YT>(y, (int64_t)r * ldy + cidx, act < 0 ? v : act_apply(v, act));
+      }
     }
 }
 
 }  // namespace
 
-// x_f32 / y_f32: element type of the activations on either side (false: bf16)
+// x_f32 / y_f32: element type of the activations on either side (false: bf16); bias [n_out] (bf16, optional) and then act
+// (b200_act_kind, < 0: none) are applied to the fp32 sum
 int linear_simt(bool x_f32, bool y_f32, const void* x, int64_t ldx, const __nv_bfloat16* w, void* y, int64_t ldy, int T, int n_out,
-                int k, cudaStream_t s) {
+                int k, cudaStream_t s, const __nv_bfloat16* bias, int act) {
   if (T == 0) return B200_OK;
   const dim3 grid((n_out + kBN - 1) / kBN, (T + kBM - 1) / kBM), block(256);
   if (x_f32 && y_f32)
-    B200_CUDA(launch(linear_simt_kernel<float, float>, grid, block, 0, s, (const float*)x, ldx, w, (float*)y, ldy, T, n_out, k));
+    B200_CUDA(launch(linear_simt_kernel<float, float>, grid, block, 0, s, (const float*)x, ldx, w, (float*)y, ldy, T, n_out, k, bias, act));
   else if (!x_f32 && !y_f32)
     B200_CUDA(launch(linear_simt_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, s, (const __nv_bfloat16*)x, ldx, w,
-                     (__nv_bfloat16*)y, ldy, T, n_out, k));
+                     (__nv_bfloat16*)y, ldy, T, n_out, k, bias, act));
   else if (x_f32)
     B200_CUDA(launch(linear_simt_kernel<float, __nv_bfloat16>, grid, block, 0, s, (const float*)x, ldx, w, (__nv_bfloat16*)y, ldy,
-                     T, n_out, k));
+                     T, n_out, k, bias, act));
   else
     B200_CUDA(launch(linear_simt_kernel<__nv_bfloat16, float>, grid, block, 0, s, (const __nv_bfloat16*)x, ldx, w, (float*)y, ldy, T,
-                     n_out, k));
+                     n_out, k, bias, act));
   return B200_OK;
 }
 

@@ -1,0 +1,394 @@
+// Inputs of an attention mixer whose q, k and v pass a short convolution, with a selective scan beside it (B200_MIXER_SELECTIVE), and
+// the scan itself.
+//
+//  * conv_inputs: causal per-channel convolutions over the fused projection rows q | k | v | x.  A thread owns V channels and walks a
+//    run of rows with the earlier inputs in registers, so every input is fetched once; ahead of a portion's first row they come from
+//    the sequence's tails in its state slot.  q, k, v: no activation; q leaves as fp32 rows, k and v go to the paged caches.
+//    x: bias and silu, rows of the activation type (they are also the input of the scan's projection).  In a step whose
+//    sequences bring one row each (decode) the thread that read a channel's tail also shifts it.
+//  * selective_scan: per channel c and state n   S = exp(dt_c A[c][n]) S + dt_c x_c B_n;   y_c = sum_n S[c][n] C_n + D_c x_c;
+//    out_c = y_c silu(z_c), dt = softplus(dt_pre + bias).  Channels and states do not interact except through the sum over n, so a
+//    channel is walked by L neighbouring lanes with NS states each in registers; a CTA of 128 threads takes 128 / L channels of one
+//    sequence and stages 16 rows at a time in shared memory, the next 16 travelling into registers meanwhile.  Only one multiply-add per state is on
+//    the chain from a row to the next; the exponentials depend on dt alone.  The state, fp32 [inner][n_state] in the sequence's slot,
+//    is read ahead of the dependency wait: no launch of the same step before this one writes it.
+//    A sequence whose first row of the step is at position 0 starts from zeros, whatever the slot held.
+#include <algorithm>
+
+#include "common.cuh"
+
+namespace b200 {
+namespace {
+
+template <typename AT, int V> __device__ __forceinline__ void ldv(const AT* p, int64_t i, float* o);
+template <> __device__ __forceinline__ void ldv<float, 1>(const float* p, int64_t i, float* o) { o[0] = p[i]; }
+template <> __device__ __forceinline__ void ldv<__nv_bfloat16, 1>(const __nv_bfloat16* p, int64_t i, float* o) { o[0] = __bfloat162float(p[i]); }
+template <> __device__ __forceinline__ void ldv<float, 4>(const float* p, int64_t i, float* o) {
+  const float4 v = *reinterpret_cast<const float4*>(p + i);
+  o[0] = v.x, o[1] = v.y, o[2] = v.z, o[3] = v.w;
+}
+template <> __device__ __forceinline__ void ldv<__nv_bfloat16, 4>(const __nv_bfloat16* p, int64_t i, float* o) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p + i);
+  o[0] = bf16lo(v.x), o[1] = bf16hi(v.x), o[2] = bf16lo(v.y), o[3] = bf16hi(v.y);
+}
+template <typename AT, int V> __device__ __forceinline__ void stv(AT* p, int64_t i, const float* o);
+template <> __device__ __forceinline__ void stv<float, 1>(float* p, int64_t i, const float* o) { p[i] = o[0]; }
+template <> __device__ __forceinline__ void stv<__nv_bfloat16, 1>(__nv_bfloat16* p, int64_t i, const float* o) { p[i] = __float2bfloat16_rn(o[0]); }
+template <> __device__ __forceinline__ void stv<float, 4>(float* p, int64_t i, const float* o) {
+  *reinterpret_cast<float4*>(p + i) = make_float4(o[0], o[1], o[2], o[3]);
+}
+template <> __device__ __forceinline__ void stv<__nv_bfloat16, 4>(__nv_bfloat16* p, int64_t i, const float* o) {
+  *reinterpret_cast<uint2*>(p + i) = make_uint2(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]));
+}
+
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+
+constexpr int kConvThreads = 128;
+
+template <typename AT>
+struct ConvArgs {
+  const AT* fused;
+  int64_t ld;
+  const float *conv_a, *conv_x, *bias_x;
+  float *tails_a, *tails_x;
+  int taps_a, taps_x;
+  int64_t slot_stride;
+  const int32_t *positions, *row_to_seq, *seq_start, *seq_slots, *slots;
+  float* qout;
+  AT *kc, *vc, *xc;
+  int T, heads, kv_heads, dim, vdim, inner, block_size, one_row, run, blocks_a;
+};
+
+// TAPS > 0: known at compile time, earlier inputs in registers; 0: any count, earlier inputs re-read
+template <typename AT, int V, int TAPS>
+__device__ __forceinline__ void conv_walk(const ConvArgs<AT>& a, bool is_x, int c, int col, int n_ch, const float* w, int taps_rt, float* tails) {
+  const int taps = TAPS > 0 ? TAPS : taps_rt;
+  float wr[TAPS > 0 ? TAPS : 1][V], bias[V];
+  float h1[V], h2[V], h3[V];   // TAPS > 0: the inputs of lag 1, 2, 3
+#pragma unroll
+  for (int v = 0; v < V; ++v) h1[v] = h2[v] = h3[v] = bias[v] = 0.f;
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int v = 0; v < V; ++v) wr[j][v] = w ? w[(int64_t)(c + v) * taps + j] : 1.0f;
+  }
+  if (is_x && a.bias_x) ldv<float, V>(a.bias_x, c, bias);
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
+  const int t0 = blockIdx.x * a.run, t1 = min(a.T, t0 + a.run);
+  int last_seq = -1;
+  for (int t = t0; t < t1; ++t) {
+    const int s = a.row_to_seq ? a.row_to_seq[t] : t;
+    const int r = t - a.seq_start[s], pos = a.positions[t];
+    float* tail = tails ? tails + (int64_t)a.seq_slots[s] * a.slot_stride : nullptr;   // [taps - 1][n_ch]
+    auto lagged = [&](int j, float* o) {   // the input of position pos - j, j >= 1
+      if (pos - j < 0) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) o[v] = 0.f;
+      } else if (r - j >= 0) {
+        ldv<AT, V>(a.fused, (int64_t)(t - j) * a.ld + col, o);
+      } else {
+        ldv<float, V>(tail, (int64_t)(taps - 1 + r - j) * n_ch + c, o);
+      }
+    };
+    float cur[V], acc[V];
+    ldv<AT, V>(a.fused, (int64_t)t * a.ld + col, cur);
+    if constexpr (TAPS > 0) {
+      if (s != last_seq) {
+        if constexpr (TAPS > 1) lagged(1, h1);
+        if constexpr (TAPS > 2) lagged(2, h2);
+        if constexpr (TAPS > 3) lagged(3, h3);
+        last_seq = s;
+      }
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        float x = bias[v];
+        if constexpr (TAPS > 3) x = fmaf(wr[TAPS - 4][v], h3[v], x);
+        if constexpr (TAPS > 2) x = fmaf(wr[TAPS - 3][v], h2[v], x);
+        if constexpr (TAPS > 1) x = fmaf(wr[TAPS - 2][v], h1[v], x);
+        acc[v] = fmaf(wr[TAPS - 1][v], cur[v], x);
+      }
+      if (a.one_row) {   // entry i of the tail takes lag taps - 2 - i
+        if constexpr (TAPS > 3) stv<float, V>(tail, (int64_t)(TAPS - 4) * n_ch + c, h2);
+        if constexpr (TAPS > 2) stv<float, V>(tail, (int64_t)(TAPS - 3) * n_ch + c, h1);
+        if constexpr (TAPS > 1) stv<float, V>(tail, (int64_t)(TAPS - 2) * n_ch + c, cur);
+      }
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        h3[v] = h2[v];
+        h2[v] = h1[v];
+        h1[v] = cur[v];
+      }
+    } else {
+#pragma unroll
+      for (int v = 0; v < V; ++v) acc[v] = fmaf(w[(int64_t)(c + v) * taps + taps - 1], cur[v], bias[v]);
+      for (int j = 1; j < taps; ++j) {
+        float o[V];
+        lagged(j, o);
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[v] = fmaf(w[(int64_t)(c + v) * taps + taps - 1 - j], o[v], acc[v]);
+      }
+      if (a.one_row) {   // entry i takes the input of lag taps - 2 - i: what it reads lies above all it has written
+        for (int i = 0; i < taps - 1; ++i) {
+          float o[V];
+          if (i == taps - 2) {
+#pragma unroll
+            for (int v = 0; v < V; ++v) o[v] = cur[v];
+          } else {
+            lagged(taps - 2 - i, o);
+          }
+          stv<float, V>(tail, (int64_t)i * n_ch + c, o);
+        }
+      }
+    }
+    if (is_x) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) acc[v] = silu_f(acc[v]);
+      stv<AT, V>(a.xc, (int64_t)t * a.inner + c, acc);
+    } else if (c < nq) {
+      stv<float, V>(a.qout, (int64_t)t * nq + c, acc);
+    } else {
+      const int slot = a.slots[t];
+      if (slot < 0) continue;
+      const int64_t blk = slot / a.block_size, off = slot % a.block_size;
+      const bool is_k = c < nq + nk;
+      const int e = is_k ? c - nq : c - nq - nk, d = is_k ? a.dim : a.vdim, g = e / d;
+      stv<AT, V>(is_k ? a.kc : a.vc, ((blk * a.kv_heads + g) * a.block_size + off) * d + e % d, acc);
+    }
+  }
+}
+
+template <typename AT, int V>
+__global__ void __launch_bounds__(kConvThreads)
+conv_inputs_kernel(const ConvArgs<AT> a) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int n_a = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
+  const bool is_x = (int)blockIdx.y >= a.blocks_a;
+  const int n_ch = is_x ? a.inner : n_a, by = is_x ? blockIdx.y - a.blocks_a : blockIdx.y;
+  const int c = (by * kConvThreads + threadIdx.x) * V;
+  if (c >= n_ch) return;
+  const int col = is_x ? n_a + c : c;
+  const float* w = is_x ? a.conv_x : a.conv_a;
+  float* tails = is_x ? a.tails_x : a.tails_a;
+  const int taps = is_x ? a.taps_x : a.taps_a;
+  switch (taps) {
+    case 0: case 1: conv_walk<AT, V, 1>(a, is_x, c, col, n_ch, w, 1, tails); break;
+    case 2: conv_walk<AT, V, 2>(a, is_x, c, col, n_ch, w, 2, tails); break;
+    case 3: conv_walk<AT, V, 3>(a, is_x, c, col, n_ch, w, 3, tails); break;
+    case 4: conv_walk<AT, V, 4>(a, is_x, c, col, n_ch, w, 4, tails); break;
+    default: conv_walk<AT, V, 0>(a, is_x, c, col, n_ch, w, taps, tails); break;
+  }
+}
+
+template <typename AT>
+int conv_inputs_t(ConvArgs<AT> a, cudaStream_t s) {
+  a.run = a.one_row ? 1 : (a.T >= 1024 ? 16 : (a.T >= 128 ? 8 : 2));
+  const int n_a = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(a.fused) | reinterpret_cast<uintptr_t>(a.tails_a) | reinterpret_cast<uintptr_t>(a.tails_x) |
+                         reinterpret_cast<uintptr_t>(a.bias_x) | reinterpret_cast<uintptr_t>(a.qout) | reinterpret_cast<uintptr_t>(a.kc) |
+                         reinterpret_cast<uintptr_t>(a.vc) | reinterpret_cast<uintptr_t>(a.xc);
+  // four channels per thread: every group of channels and every row starts at a multiple of four elements
+  const bool v4 = ptrs % 16 == 0 && a.ld % 4 == 0 && a.slot_stride % 4 == 0 && (n_a == 0 || (a.dim % 4 == 0 && a.vdim % 4 == 0)) && a.inner % 4 == 0;
+  const int per = kConvThreads * (v4 ? 4 : 1);
+  a.blocks_a = (n_a + per - 1) / per;
+  const int blocks_x = (a.inner + per - 1) / per;
+  const dim3 grid((a.T + a.run - 1) / a.run, a.blocks_a + blocks_x);
+  if (v4) B200_CUDA(launch(conv_inputs_kernel<AT, 4>, grid, dim3(kConvThreads), (size_t)0, s, a));
+  else B200_CUDA(launch(conv_inputs_kernel<AT, 1>, grid, dim3(kConvThreads), (size_t)0, s, a));
+  return B200_OK;
+}
+
+// ---- the scan ----------------------------------------------------------------------------------------------------------------
+constexpr int kSelThreads = 128, kSelStage = 16;
+
+template <typename AT>
+struct SelArgs {
+  const AT *xc, *bc, *z;
+  int64_t ldbc, ldz, slot_stride;
+  int b_off;
+  const float *dt_pre, *dt_bias, *A, *D;
+  const int32_t *positions, *seq_start, *seq_slots;
+  float* state;
+  AT* out;
+  int inner, n_state;
+};
+
+template <typename AT, int L, int NS>
+__global__ void __launch_bounds__(kSelThreads)
+selective_scan_kernel(const SelArgs<AT> a) {
+  constexpr int CH = kSelThreads / L, NP = L * NS;                                       // channels of the CTA, padded states
+  constexpr int EX = (kSelStage * CH + kSelThreads - 1) / kSelThreads;                    // staged elements per thread: channel rows ..
+  constexpr int EB = (kSelStage * NP + kSelThreads - 1) / kSelThreads;                    // .. B and C rows
+  __shared__ __align__(16) float sB[kSelStage][NP], sC[kSelStage][NP];
+  __shared__ float2 sd[kSelStage][CH];   // dt, dt x
+  __shared__ float sy[kSelStage][CH];
+  const int s = blockIdx.x, c0 = blockIdx.y * CH, tid = threadIdx.x;
+  const int ch = tid / L, n0 = (tid % L) * NS, c = c0 + ch;
+  const int N = a.n_state, inner = a.inner;
+  float A[NS], S[NS];
+  // bounds of the sequence, slots and positions are inputs of the step, the state is the step before's: all are complete when this
+  // launch may start, so they are fetched while the launch before still runs
+  const int start = a.seq_start[s], n_rows = a.seq_start[s + 1] - start;
+  if (n_rows <= 0) {
+    pdl_wait();
+    return;
+  }
+  const bool fresh = a.positions[start] == 0;
+  float* st = a.state + (int64_t)a.seq_slots[s] * a.slot_stride + (int64_t)c * N;
+#pragma unroll
+  for (int i = 0; i < NS; ++i) {
+    const bool live = c < inner && n0 + i < N;
+    A[i] = live ? a.A[(int64_t)c * N + n0 + i] : 0.f;
+    S[i] = live && !fresh ? st[n0 + i] : 0.f;
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  float rx[EX], rdt[EX], rz[EX], rB[EB], rC[EB];
+  auto fetch = [&](int b0) {
+    const int nb = min(kSelStage, n_rows - b0);
+#pragma unroll
+    for (int i = 0; i < EX; ++i) {
+      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
+      const bool live = r < nb && cc < inner;
+      const int64_t o = (int64_t)(start + b0 + (live ? r : 0)) * inner + (live ? cc : 0);
+      float x1[1] = {0.f};
+      if (live) ldv<AT, 1>(a.xc, o, x1);
+      rx[i] = x1[0];
+      rdt[i] = live ? a.dt_pre[o] + a.dt_bias[cc] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < EB; ++i) {
+      const int e = tid + kSelThreads * i, r = e / NP, n = e % NP;
+      float b1[1] = {0.f}, c1[1] = {0.f};
+      if (r < nb && n < N) {
+        const int64_t o = (int64_t)(start + b0 + r) * a.ldbc + a.b_off + n;
+        ldv<AT, 1>(a.bc, o, b1);
+        ldv<AT, 1>(a.bc, o + N, c1);
+      }
+      rB[i] = b1[0];
+      rC[i] = c1[0];
+    }
+  };
+  fetch(0);
+  for (int b0 = 0; b0 < n_rows; b0 += kSelStage) {
+    const int nb = min(kSelStage, n_rows - b0);
+    float xk[EX];   // this stage's x, for the skip term
+#pragma unroll
+    for (int i = 0; i < EX; ++i) {
+      const int e = tid + kSelThreads * i;
+      xk[i] = rx[i];
+      if (EX * kSelThreads == kSelStage * CH || e < kSelStage * CH) {
+        const float dt = softplus_f(rdt[i]);
+        sd[e / CH][e % CH] = make_float2(dt, dt * rx[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < EB; ++i) {
+      const int e = tid + kSelThreads * i;
+      if (EB * kSelThreads == kSelStage * NP || e < kSelStage * NP) {
+        sB[e / NP][e % NP] = rB[i];
+        sC[e / NP][e % NP] = rC[i];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < EX; ++i) {   // this stage's gates arrive during the walk
+      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
+      float z1[1] = {0.f};
+      if (r < nb && cc < inner) ldv<AT, 1>(a.z, (int64_t)(start + b0 + r) * a.ldz + cc, z1);
+      rz[i] = z1[0];
+    }
+    __syncthreads();
+    if (b0 + kSelStage < n_rows) fetch(b0 + kSelStage);
+    auto step = [&](int r) {
+      const float2 d = sd[r][ch];
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < NS; ++i) {
+        S[i] = fmaf(expf(d.x * A[i]), S[i], d.y * sB[r][n0 + i]);
+        y = fmaf(S[i], sC[r][n0 + i], y);
+      }
+#pragma unroll
+      for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+      if (tid % L == 0) sy[r][ch] = y;
+    };
+    if (nb == kSelStage) {
+#pragma unroll 4
+      for (int r = 0; r < kSelStage; ++r) step(r);
+    } else {
+      for (int r = 0; r < nb; ++r) step(r);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < EX; ++i) {
+      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
+      if (r < nb && cc < inner) {
+        float o1[1] = {fmaf(a.D[cc], xk[i], sy[r][e % CH]) * silu_f(rz[i])};
+        stv<AT, 1>(a.out, (int64_t)(start + b0 + r) * inner + cc, o1);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NS; ++i)
+    if (c < inner && n0 + i < N) st[n0 + i] = S[i];
+}
+
+template <typename AT>
+int selective_scan_t(const SelArgs<AT>& a, int S, cudaStream_t s) {
+  const int N = a.n_state;
+#define SEL(LV, NV) B200_CUDA(launch(selective_scan_kernel<AT, LV, NV>, dim3(S, (a.inner + kSelThreads / LV - 1) / (kSelThreads / LV)), dim3(kSelThreads), (size_t)0, s, a))
+  if (N <= 4) SEL(1, 4);
+  else if (N <= 8) SEL(2, 4);
+  else if (N <= 16) SEL(4, 4);
+  else if (N <= 32) SEL(8, 4);
+  else if (N <= 64) SEL(16, 4);
+  else if (N <= 128) SEL(32, 4);
+  else SEL(32, 8);
+#undef SEL
+  return B200_OK;
+}
+
+}  // namespace
+
+int conv_inputs(bool f32, const void* fused, int64_t ld, const float* conv_a, int taps_a, float* tails_a, const float* conv_x, const float* bias_x,
+                int taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
+                const int32_t* seq_slots, const int32_t* slots, float* qout, void* kc, void* vc, void* xc, int T, int heads, int kv_heads,
+                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s) {
+  if (T == 0) return B200_OK;
+  B200_REQUIRE(taps_a <= 1 || (conv_a && tails_a && seq_slots), B200_ERR_INVALID, "conv_inputs: the q/k/v convolution needs its weights and tails");
+  B200_REQUIRE(inner == 0 || (taps_x >= 1 && conv_x && xc && (taps_x == 1 || (tails_x && seq_slots))), B200_ERR_INVALID,
+               "conv_inputs: the second convolution needs its weights, tails and output");
+  B200_REQUIRE(positions && seq_start && (heads == 0 || (slots && qout && kc && vc)), B200_ERR_INVALID, "conv_inputs: null argument");
+  if (f32) {
+    ConvArgs<float> a = {(const float*)fused, ld, conv_a, conv_x, bias_x, tails_a, tails_x, taps_a, taps_x, slot_stride, positions, row_to_seq, seq_start,
+                         seq_slots, slots, qout, (float*)kc, (float*)vc, (float*)xc, T, heads, kv_heads, dim, vdim, inner, block_size,
+                         one_row ? 1 : 0, 1, 0};
+    return conv_inputs_t<float>(a, s);
+  }
+  ConvArgs<__nv_bfloat16> a = {(const __nv_bfloat16*)fused, ld, conv_a, conv_x, bias_x, tails_a, tails_x, taps_a, taps_x, slot_stride, positions, row_to_seq,
+                               seq_start, seq_slots, slots, qout, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, (__nv_bfloat16*)xc, T, heads, kv_heads, dim,
+                               vdim, inner, block_size, one_row ? 1 : 0, 1, 0};
+  return conv_inputs_t<__nv_bfloat16>(a, s);
+}
+
+// rows of W_x's product: dt | B | C, dt and the total padded to multiples of 8 so that both matrix products can be addressed by TMA
+int selective_dt_pad(int rank) { return (rank + 7) / 8 * 8; }
+int selective_rows(int rank, int state) { return (selective_dt_pad(rank) + 2 * state + 7) / 8 * 8; }
+
+int selective_scan(bool f32, const void* xc, const void* bc, int64_t ldbc, int b_off, const float* dt_pre, const float* dt_bias, const float* A,
+                   const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
+                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, cudaStream_t s) {
+  if (S == 0) return B200_OK;
+  B200_REQUIRE(inner > 0 && n_state > 0 && n_state <= 256, B200_ERR_UNSUPPORTED, "selective_scan: %d channels, %d states (at most 256)", inner, n_state);
+  if (f32) {
+    SelArgs<float> a = {(const float*)xc, (const float*)bc, (const float*)z, ldbc, ldz, slot_stride, b_off, dt_pre, dt_bias, A, D, positions, seq_start,
+                        seq_slots, state, (float*)out, inner, n_state};
+    return selective_scan_t<float>(a, S, s);
+  }
+  SelArgs<__nv_bfloat16> a = {(const __nv_bfloat16*)xc, (const __nv_bfloat16*)bc, (const __nv_bfloat16*)z, ldbc, ldz, slot_stride, b_off, dt_pre, dt_bias, A,
+                              D, positions, seq_start, seq_slots, state, (__nv_bfloat16*)out, inner, n_state};
+  return selective_scan_t<__nv_bfloat16>(a, S, s);
+}
+
+}  // namespace b200

@@ -42,6 +42,16 @@
 //                 term -> skip, gate, grouped RMS norm -> W_o
 //     dense:      W_up -> polynomial of unit-RMS powers -> W_down;   experts: chosen-softmax router, clamped gated experts
 //   logit rows: hyper_step over the rows (closes the last sublayer, a = ones, output norm) -> W_head -> fp32 logits -> argmax
+//
+// Looped form (b200_stack_cfg.form = B200_FORM_LOOPED), same step entry, cache, state slots and graph replay; the layer list is unrolled:
+//   e = x = rms(table[id]) * w                                            fp32 residual stream
+//   per entry:  x += e, x += step vector (ahead of a pass);  h = rms(x) * w;  x += rms(mixer(h)) * w';  likewise the feed-forward.
+//     Between two sublayers all of that is one launch (rms_sandwich), which also averages the results of two mixers side by side.
+//     retention:  fused q | k | v | gate -> rotation, recurrence over the state slot, unit RMS, silu gate -> W_o
+//     attention:  fused q | k | v (| x | z of the selective scan) | head gates, with biases -> convolutions, k and v into the paged cache,
+//                 x with silu -> windowed attention with capped, distance-biased scores -> W_o
+//     selective:  W_x -> dt | B | C -> W_dt -> scan over the state slot with skip and gate -> W_o
+//     dense:      W_up with bias and squared relu in its epilogue -> W_down with bias
 #include <math.h>
 #include <stdlib.h>
 
@@ -72,6 +82,10 @@ struct StackLayerW {
   const float *n_mix_pre_b = nullptr, *n_mlp_pre_b = nullptr, *scale_mix = nullptr, *scale_mlp = nullptr, *hc_mix = nullptr, *hc_mlp = nullptr,
               *canon_mlp = nullptr, *conv_b = nullptr, *skip = nullptr, *mlp_act = nullptr;
   int64_t tail2_off = 0, ctail_off = 0;   // floats from the start of a state slot: the feed-forward's input convolution tail, the mixer's own
+  // looped form (tail2_off: the convolution tail of the second mixer, rec_off: the state of the retention or of the selective scan)
+  const float *loop_step = nullptr, *dist_bias = nullptr, *decay = nullptr, *side_conv = nullptr, *side_conv_b = nullptr, *side_dt_b = nullptr,
+              *side_a = nullptr, *side_skip = nullptr, *out_main = nullptr, *out_side = nullptr;
+  const __nv_bfloat16 *qkv_b = nullptr, *side_proj = nullptr, *side_dt = nullptr, *side_o = nullptr, *mlp_up_b = nullptr, *mlp_down_b = nullptr;
 };
 
 struct StackModel {
@@ -114,6 +128,12 @@ struct StackModel {
   float* zero_sink = nullptr;          // [heads] zeros: a sink of score 0 is one more unit in the denominator
   // multi-stream form
   float* xs = nullptr;                 // [streams][max_tokens][width]
+  // looped form
+  const float* embed_norm = nullptr;
+  float *eout = nullptr, *dtp = nullptr;                   // embedding output; step sizes ahead of bias and softplus
+  void *xc = nullptr, *xp = nullptr, *ssy = nullptr;       // convolved channels, dt | B | C, gated scan output
+  void* ret_ws = nullptr;                                  // chunk states of the retention
+  int64_t ret_ws_bytes = 0;
 };
 
 bool paged_attn_tc_supported(int hq, int hkv, int block_size);   // attn_tc.cu
@@ -122,6 +142,8 @@ static bool is_latent(const b200_stack_layer& L) { return L.mixer == B200_MIXER_
 static bool is_mlstm(const b200_stack_layer& L) { return L.mixer == B200_MIXER_MLSTM; }
 static bool is_delta(const b200_stack_layer& L) { return L.mixer == B200_MIXER_DELTA; }
 static bool is_ssd(const b200_stack_layer& L) { return L.mixer == B200_MIXER_SSD; }
+static bool is_retention(const b200_stack_layer& L) { return L.mixer == B200_MIXER_RETENTION; }
+static bool has_side(const b200_stack_layer& L) { return L.side == B200_MIXER_SELECTIVE; }
 static bool head_decay(const b200_stack_layer& L) { return (L.mixer_flags & B200_MIXF_HEAD_DECAY) != 0; }
 
 // bf16 mode, keys and values of 64 to 128 dimensions in blocks of 128 tokens: the tcgen05 attention kernels of the fixed
@@ -136,18 +158,22 @@ static bool layer_attn_tc(const b200_stack_cfg& m, const b200_stack_layer& L) {
 // latent mixers cache one row [latent | rotated key part] per token (no value cache); mLSTM layers cache nothing
 static int cache_kdim(const b200_stack_cfg& m, const b200_stack_layer& L) {
   if (is_latent(L)) return L.kv_share > 0 ? 0 : L.kv_rank + L.rot_dim;
-  if (is_mlstm(L) || is_delta(L) || is_ssd(L)) return 0;
+  if (is_mlstm(L) || is_delta(L) || is_ssd(L) || is_retention(L)) return 0;
   return layer_attn_tc(m, L) ? kHeadDim : L.dim;
 }
 static int cache_vdim(const b200_stack_cfg& m, const b200_stack_layer& L) {
-  if (is_latent(L) || is_mlstm(L) || is_delta(L) || is_ssd(L)) return 0;
+  if (is_latent(L) || is_mlstm(L) || is_delta(L) || is_ssd(L) || is_retention(L)) return 0;
   return layer_attn_tc(m, L) ? kHeadDim : L.vdim;
 }
 
 static int64_t up(int64_t v, int64_t a) { return (v + a - 1) / a * a; }
 
 // rows of the fused projection of the mixer's input
+static int attn_channels(const b200_stack_layer& L) { return L.heads * L.dim + L.kv_heads * (L.dim + L.vdim); }
 static int qkv_rows(const b200_stack_layer& L) {
+  if (is_retention(L)) return 2 * L.heads * (L.dim + L.vdim);                                  // q | k | v | gate
+  if (has_side(L))                                                                             // q | k | v | x | z | head gates
+    return attn_channels(L) + 2 * L.side_inner + ((L.mixer_flags & B200_MIXF_HEAD_GATE) ? L.heads : 0);
   if (is_ssd(L)) return 2 * L.heads * L.vdim + 2 * L.kv_heads * L.dim + L.heads;             // z | x | B | C | dt
   if (is_delta(L) && head_decay(L)) return 2 * L.kv_heads * L.dim + 2 * L.heads * L.vdim + 2 * L.heads;   // q | k | v | gate | b | a
   if (is_delta(L)) return delta_fused_rows(L.heads, L.kv_heads, L.dim, L.vdim, L.decay_rank, L.gate_rank, nullptr);
@@ -157,7 +183,7 @@ static int qkv_rows(const b200_stack_layer& L) {
   if (is_latent(L))
     return L.heads * (L.dim + L.rot_dim) + L.kv_rank + L.rot_dim + ((L.mixer_flags & B200_MIXF_GATE) ? L.heads * L.vdim : 0);
   if (is_mlstm(L)) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim;
-  return L.heads * L.dim + L.kv_heads * (L.dim + L.vdim);
+  return attn_channels(L) + (L.mixer == B200_MIXER_ATTENTION && (L.mixer_flags & B200_MIXF_HEAD_GATE) ? L.heads : 0);
 }
 
 // bf16 mode: the tcgen05 weight-streaming linear wherever TMA can address the operands, else the CUDA-core tile kernel;
@@ -173,6 +199,27 @@ static int stack_linear(b200_ctx* c, const void* x, int64_t ldx, const __nv_bflo
     return linear_tc((const __nv_bfloat16*)x, ldx, w, nullptr, (__nv_bfloat16*)y, ldy, T, n_out, k, c->lin_ws, c->lin_ws_bytes,
                      nullptr, s);
   return linear_simt(false, false, x, ldx, w, y, ldy, T, n_out, k, s);
+}
+
+// y = act(x . w^T + bias) with bias (optional) and act (b200_act_kind, < 0: none) in the epilogue; y_f32: unrounded fp32 rows (no bias,
+// no activation on the tcgen05 path).
+static int linear_ex(bool f32, bool y_f32, const void* x, int64_t ldx, const __nv_bfloat16* w, const __nv_bfloat16* bias, void* y, int64_t ldy,
+                     int T, int n_out, int k, int act, void* ws, int64_t ws_bytes, cudaStream_t s) {
+  if (f32) return linear_simt(true, true, x, ldx, w, y, ldy, T, n_out, k, s, bias, act);
+  static const int tc_env = getenv("B200_STACK_TC") ? atoi(getenv("B200_STACK_TC")) : 1;
+  const bool plain32 = y_f32 && !bias && act < 0 && ldy == n_out && reinterpret_cast<uintptr_t>(y) % 16 == 0;
+  if (tc_env && (!y_f32 || plain32) && k % 8 == 0 && ldx % 8 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0 &&
+      linear_tc_supported(T, n_out, k) && linear_tc_workspace_bytes(T, n_out, k) <= ws_bytes) {
+    LinearExtra ex;
+    if (y_f32) {
+      ex.mode = 4;
+      ex.out_f32 = static_cast<float*>(y);
+      return linear_tc((const __nv_bfloat16*)x, ldx, w, nullptr, nullptr, n_out, T, n_out, k, ws, ws_bytes, &ex, s);
+    }
+    ex.post_act = act < 0 ? 0 : act + 1;
+    return linear_tc((const __nv_bfloat16*)x, ldx, w, bias, (__nv_bfloat16*)y, ldy, T, n_out, k, ws, ws_bytes, &ex, s);
+  }
+  return linear_simt(false, y_f32, x, ldx, w, y, ldy, T, n_out, k, s, bias, act);
 }
 
 // Dense gated feed-forward, first half: act(gate x) * (up x) -> out [T][ff].  Interleaved weights: one tcgen05 launch whose
@@ -284,12 +331,41 @@ static int stack_ready_hyper(const b200_ctx* c) {
   return B200_OK;
 }
 
+static int stack_ready_looped(const b200_ctx* c) {
+  const StackModel* M = c->stack;
+  const b200_stack_cfg& m = M->cfg;
+  B200_REQUIRE(M->embed_norm, B200_ERR_STATE, "step: the embedding's norm is not set");
+  B200_REQUIRE(m.n_state_slots <= 0 || M->state, B200_ERR_STATE, "step: state slots not set");
+  for (size_t l = 0; l < M->layers.size(); ++l) {
+    const b200_stack_layer& L = M->layers[l];
+    const StackLayerW& W = M->w[l];
+    const int li = (int)l;
+    B200_REQUIRE(W.n_mix_pre && W.n_mix_post && W.qkv && W.o, B200_ERR_STATE, "step: layer %d mixer weights incomplete", li);
+    B200_REQUIRE(!L.loop_step || W.loop_step, B200_ERR_STATE, "step: layer %d: the vector of its pass is missing", li);
+    B200_REQUIRE(L.rot_dims == 0 || (L.rot_table >= 0 && M->rot[L.rot_table] && M->rot_half[L.rot_table] * 2 == L.rot_dims), B200_ERR_STATE,
+                 "step: layer %d rotation table missing or of another size", li);
+    if (is_retention(L)) {
+      B200_REQUIRE(W.decay, B200_ERR_STATE, "step: layer %d decays missing", li);
+    } else {
+      B200_REQUIRE(W.kc && W.vc && (!(L.mixer_flags & B200_MIXF_QKV_BIAS) || W.qkv_b) && (L.conv_taps <= 0 || W.conv) && (L.bias_dist <= 0 || W.dist_bias),
+                   B200_ERR_STATE, "step: layer %d attention weights / cache incomplete", li);
+      if (has_side(L))
+        B200_REQUIRE(W.side_conv && W.side_proj && W.side_dt && W.side_dt_b && W.side_a && W.side_skip && W.side_o && W.out_main && W.out_side,
+                     B200_ERR_STATE, "step: layer %d weights of its second mixer incomplete", li);
+    }
+    if (L.mlp == B200_MLP_DENSE)
+      B200_REQUIRE(W.n_mlp_pre && W.n_mlp_post && W.mlp_gate_up && W.mlp_down, B200_ERR_STATE, "step: layer %d feed-forward weights incomplete", li);
+  }
+  return B200_OK;
+}
+
 int stack_ready(const b200_ctx* c) {
   const StackModel* M = c->stack;
   B200_REQUIRE(M->embed && M->head && M->final_norm, B200_ERR_STATE, "step: embedding / output weights not set");
   if (M->cfg.form == B200_FORM_PARALLEL) return stack_ready_parallel(c);
   if (M->cfg.form == B200_FORM_POSTNORM) return stack_ready_postnorm(c);
   if (M->cfg.form == B200_FORM_HYPER) return stack_ready_hyper(c);
+  if (M->cfg.form == B200_FORM_LOOPED) return stack_ready_looped(c);
   for (size_t l = 0; l < M->layers.size(); ++l) {
     const b200_stack_layer& L = M->layers[l];
     const StackLayerW& W = M->w[l];
@@ -731,12 +807,139 @@ static int stack_enqueue_step_hyper(b200_ctx* c, const StepArgs& a, cudaStream_t
   return B200_OK;
 }
 
+// The step of the looped form.
+static int stack_enqueue_step_looped(b200_ctx* c, const StepArgs& a, cudaStream_t s) {
+  StackModel* M = c->stack;
+  const b200_stack_cfg& m = M->cfg;
+  const bool f32 = m.f32 != 0;
+  const int T = a.T, Wd = m.width, nL = m.n_layers;
+  const int64_t es = M->esz;
+  int rc;
+#define STEP(expr)     \
+  do {                 \
+    rc = (expr);       \
+    if (rc) return rc; \
+  } while (0)
+  const int S = a.n_seqs > 0 ? a.n_seqs : T;
+  const int32_t* seq_slots = a.seq_slots;
+  B200_REQUIRE(m.n_state_slots <= 0 || seq_slots, B200_ERR_STATE, "step: the state slots of the step's sequences were not given");
+  B200_REQUIRE(S <= T, B200_ERR_INVALID, "step: %d sequences in %d rows", S, T);
+  const bool one_row_each = (a.n_seqs > 0 && a.n_seqs == T) || a.row_to_seq == nullptr;   // known, not assumed
+  static const int plan_env = getenv("B200_STACK_ATTN_RUNS") ? atoi(getenv("B200_STACK_ATTN_RUNS")) : 1;
+  static const int chunk_env = getenv("B200_STACK_RETENTION_CHUNK") ? atoi(getenv("B200_STACK_RETENTION_CHUNK")) : 1;
+  const bool attn_plan = plan_env && a.row_to_seq && T >= 32 && T >= 2 * S;
+  bool runs_built = false;   // the step's run list is in the attention workspace
+  auto step_runs = [&]() -> int {
+    if (runs_built) return B200_OK;
+    runs_built = true;
+    return paged_attn_runs_plan(a.row_to_seq, a.ctx_lens, T, M->attn_ws, s);
+  };
+  auto linear = [&](const void* x, int64_t ldx, const __nv_bfloat16* w, const __nv_bfloat16* bias, void* y, int n_out, int k, int act, bool y_f32) -> int {
+    return linear_ex(f32, y_f32 || f32, x, ldx, w, bias, y, n_out, T, n_out, k, act, c->lin_ws, c->lin_ws_bytes, s);
+  };
+  bool adds = false;
+  for (const b200_stack_layer& L : M->layers) adds = adds || L.loop_add;
+  float* x = M->x;
+  STEP(seq_bounds(a.row_to_seq, T, S, M->seq_start, s));
+  STEP(embed_scaled(a.ids, M->embed, x, T, Wd, m.vocab, m.embed_scale, s, a.prev_tokens, a.n_prev));
+  STEP(rms_sandwich(f32, x, nullptr, nullptr, nullptr, nullptr, M->embed_norm, true, adds ? M->eout : nullptr, nullptr, nullptr,
+                    M->layers[0].loop_step ? M->w[0].loop_step : nullptr, M->w[0].n_mix_pre, M->hn, nullptr, T, Wd, m.norm_eps, s));
+  constexpr int kShortRows = 8;   // portions up to this length walk the recurrence row by row
+  for (int l = 0; l < nL; ++l) {
+    const b200_stack_layer& L = M->layers[l];
+    const StackLayerW& W = M->w[l];
+    const int qr = qkv_rows(L), av = L.heads * L.vdim;
+    const void* y_side = nullptr;
+    STEP(linear(M->hn, Wd, W.qkv, (L.mixer_flags & B200_MIXF_QKV_BIAS) ? W.qkv_b : nullptr, M->qkv, qr, Wd, -1, false));
+    if (is_retention(L)) {
+      const float* rot = L.rot_dims > 0 ? M->rot[L.rot_table] : nullptr;
+      const int64_t max_pos = rot ? M->rot_pos[L.rot_table] : (1ll << 40);
+      const bool half = (L.mixer_flags & B200_MIXF_ROT_HALF) != 0;
+      const bool chunked = chunk_env && !f32 && !one_row_each && T > kShortRows && retention_chunk_supported(L.dim, L.vdim) &&
+                           (!rot || (half && L.rot_dims % 4 == 0)) &&
+                           retention_chunk_workspace_bytes(T, S, L.heads, L.dim, L.vdim) <= M->ret_ws_bytes;
+      if (!chunked || S > 1)   // chunked: only the sequences that bring a few rows
+        STEP(retention_step(f32, M->qkv, qr, rot, L.rot_dims, half, max_pos, W.decay, a.positions, M->seq_start, seq_slots, M->state + W.rec_off,
+                            M->slot_floats, M->attn, S, L.heads, L.dim, L.vdim, m.norm_eps, chunked ? kShortRows : 0, s));
+      if (chunked)
+        STEP(retention_chunk(M->qkv, qr, rot, L.rot_dims, half, max_pos, W.decay, a.positions, M->seq_start, seq_slots, M->state + W.rec_off,
+                             M->slot_floats, M->attn, T, S, L.heads, L.dim, L.vdim, m.norm_eps, S > 1 ? kShortRows : 0, M->ret_ws, s));
+    } else {
+      const int ch = attn_channels(L), inner = has_side(L) ? L.side_inner : 0;
+      float* tails = L.conv_taps > 1 ? M->state + W.ctail_off : nullptr;
+      float* tails_x = inner && L.side_taps > 1 ? M->state + W.tail2_off : nullptr;
+      STEP(conv_inputs(f32, M->qkv, qr, W.conv, L.conv_taps, tails, W.side_conv, W.side_conv_b, L.side_taps, tails_x, M->slot_floats, a.positions,
+                       a.row_to_seq, M->seq_start, seq_slots, a.slots, M->q, W.kc, W.vc, M->xc, T, L.heads, L.kv_heads, L.dim, L.vdim, inner,
+                       m.block_size, one_row_each, s));
+      if (!one_row_each) {
+        if (tails) STEP(delta_tails(f32, M->qkv, qr, a.positions, M->seq_start, seq_slots, tails, M->slot_floats, S, ch, L.conv_taps, s));
+        if (tails_x)
+          STEP(delta_tails(f32, static_cast<const char*>(M->qkv) + (int64_t)ch * es, qr, a.positions, M->seq_start, seq_slots, tails_x, M->slot_floats, S,
+                           inner, L.side_taps, s));
+      }
+      AttnExtra ex;
+      ex.softcap = L.softcap;
+      ex.dist_bias = L.bias_dist > 0 ? W.dist_bias : nullptr;
+      ex.bias_dist = L.bias_dist;
+      if (L.mixer_flags & B200_MIXF_HEAD_GATE) ex.gate = static_cast<const char*>(M->qkv) + (int64_t)(ch + 2 * inner) * es, ex.ldg = qr;
+      if (!f32 && paged_attn_mma_supported(L.heads, L.kv_heads, L.dim, L.vdim)) {
+        STEP(step_runs());
+        const int seen = L.window > 0 ? std::min(a.max_ctx, L.window + 64) : a.max_ctx;
+        STEP(paged_attn_mma(M->q, (const __nv_bfloat16*)W.kc, (const __nv_bfloat16*)W.vc, a.block_table, a.bt_stride, a.row_to_seq, a.ctx_lens,
+                            (__nv_bfloat16*)M->attn, static_cast<const int32_t*>(M->attn_ws) + 8, static_cast<const int32_t*>(M->attn_ws), T,
+                            L.heads, L.kv_heads, L.dim, L.vdim, m.block_size, L.scale, nullptr, s,
+                            latent_attn_splits(T, L.heads, L.vdim, seen, M->lat_ws_bytes), M->lat_ws, L.window, ex));
+      } else {
+        if (attn_plan) STEP(step_runs());
+        STEP(paged_attn_anydim(f32, M->q, W.kc, W.vc, a.block_table, a.bt_stride, a.row_to_seq, a.ctx_lens, a.positions, nullptr, 1ll << 40,
+                               M->attn, T, L.heads, L.kv_heads, L.dim, L.vdim, m.block_size, L.scale, attn_plan ? 2 : 0, M->attn_ws, s, 0, 0, nullptr,
+                               L.window, ex));
+      }
+      if (inner) {
+        const int rows = selective_rows(L.side_rank, L.side_state), pad = selective_dt_pad(L.side_rank);
+        STEP(linear(M->xc, inner, W.side_proj, nullptr, M->xp, rows, inner, -1, false));
+        STEP(linear(M->xp, rows, W.side_dt, nullptr, M->dtp, inner, pad, -1, true));
+        STEP(selective_scan(f32, M->xc, M->xp, rows, pad, M->dtp, W.side_dt_b, W.side_a, W.side_skip,
+                            static_cast<const char*>(M->qkv) + (int64_t)(ch + inner) * es, qr, a.positions, M->seq_start, seq_slots,
+                            M->state + W.rec_off, M->slot_floats, M->ssy, S, inner, L.side_state, s));
+        STEP(linear(M->ssy, inner, W.side_o, nullptr, M->y2, Wd, inner, -1, false));
+        y_side = M->y2;
+      }
+    }
+    STEP(linear(M->attn, av, W.o, nullptr, M->y, Wd, av, -1, false));
+    const bool last = l + 1 == nL;
+    const void* y_last = M->y;
+    const float *wa = W.out_main, *wb = W.out_side, *w_post = W.n_mix_post;
+    if (L.mlp == B200_MLP_DENSE) {
+      STEP(rms_sandwich(f32, x, M->y, y_side, wa, wb, w_post, false, nullptr, nullptr, nullptr, nullptr, W.n_mlp_pre, M->hn, nullptr, T, Wd, m.norm_eps, s));
+      STEP(linear(M->hn, Wd, W.mlp_gate_up, W.mlp_up_b, M->ffa, L.ff, Wd, L.act, false));
+      STEP(linear(M->ffa, L.ff, W.mlp_down, W.mlp_down_b, M->y, Wd, L.ff, -1, false));
+      y_side = nullptr, wa = wb = nullptr, w_post = W.n_mlp_post;
+    }
+    float* tap = M->tap ? M->tap + (int64_t)l * T * Wd : nullptr;
+    if (!last || tap) {
+      const bool add = !last && M->layers[l + 1].loop_add, stp = !last && M->layers[l + 1].loop_step;
+      STEP(rms_sandwich(f32, x, y_last, y_side, wa, wb, w_post, false, nullptr, tap, add ? M->eout : nullptr, stp ? M->w[l + 1].loop_step : nullptr,
+                        last ? nullptr : M->w[l + 1].n_mix_pre, M->hn, nullptr, T, Wd, m.norm_eps, s));
+      y_last = nullptr, y_side = nullptr, w_post = nullptr;
+    }
+    // logit rows: the last close and the output norm over those rows only
+    if (last)
+      STEP(rms_sandwich(f32, x, y_last, y_side, wa, wb, w_post, false, nullptr, nullptr, nullptr, nullptr, M->final_norm, M->lm_in, a.logit_rows, a.R, Wd,
+                        m.norm_eps, s));
+  }
+  STEP(stack_logits_f32(c, a, 0.f, s));
+#undef STEP
+  return B200_OK;
+}
+
 int stack_enqueue_step(b200_ctx* c, const StepArgs& a, cudaStream_t s) {
   StackModel* M = c->stack;
   const b200_stack_cfg& m = M->cfg;
   if (m.form == B200_FORM_PARALLEL) return stack_enqueue_step_parallel(c, a, s);
   if (m.form == B200_FORM_POSTNORM) return stack_enqueue_step_postnorm(c, a, s);
   if (m.form == B200_FORM_HYPER) return stack_enqueue_step_hyper(c, a, s);
+  if (m.form == B200_FORM_LOOPED) return stack_enqueue_step_looped(c, a, s);
   const bool f32 = m.f32 != 0;
   const int T = a.T, Wd = m.width, nL = m.n_layers;
   int rc;
@@ -838,7 +1041,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
                    cfg->max_blocks_per_seq > 0 && cfg->max_logit_rows > 0,
                B200_ERR_INVALID, "stack_create: bad sizes");
   int max_qkv = 0, max_q = 0, max_a = 0, max_top = 0, max_exp = 0, max_ff = 0, max_lat = 0, max_gates = 0, max_gu = 0, max_ffa = 0;
-  int max_qrank = 0, max_qh = 0, max_dhd = 0, max_dqk = 0, max_dav = 0, max_dh = 0, max_heads = 0;
+  int max_qrank = 0, max_qh = 0, max_dhd = 0, max_dqk = 0, max_dav = 0, max_dh = 0, max_heads = 0, max_inner = 0, max_proj = 0;
   int64_t moe_ws_bytes = 16;
   for (int l = 0; l < cfg->n_layers; ++l) {
     const b200_stack_layer& L = layers[l];
@@ -909,6 +1112,24 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
                    "stack_create: layer %d: the polynomial activation belongs to an ungated dense feed-forward", l);
       B200_REQUIRE(L.act != B200_ACT_SWIGLU_CLAMP || (!L.ungated && L.act_limit > 0.f), B200_ERR_INVALID,
                    "stack_create: layer %d: the clamped gate needs a gate projection and a positive limit", l);
+    } else if (cfg->form == B200_FORM_LOOPED) {
+      B200_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0 && L.window >= 0 && L.kv_heads > 0 && L.heads % L.kv_heads == 0 && cfg->n_state_slots > 0,
+                   B200_ERR_INVALID, "stack_create: layer %d: bad mixer sizes (or no state slots)", l);
+      if (is_retention(L)) {
+        B200_REQUIRE(L.dim <= 256 && L.kv_heads == L.heads && L.rot_dims >= 0 && L.rot_dims <= L.dim && L.rot_dims % 2 == 0 && L.rot_table < 16 && !L.side,
+                     B200_ERR_INVALID, "stack_create: layer %d: bad retention sizes", l);
+      } else {
+        B200_REQUIRE(L.mixer == B200_MIXER_ATTENTION && (L.mixer_flags & B200_MIXF_NO_QK_NORM) && !(L.mixer_flags & (B200_MIXF_HEAD_NORM | B200_MIXF_VALUE_IS_KEY | B200_MIXF_SINK | B200_MIXF_SINK_ONE)),
+                     B200_ERR_UNSUPPORTED, "stack_create: layer %d: mixer %d is not served in the looped form", l, L.mixer);
+        B200_REQUIRE(L.rot_dims == 0 && L.conv_taps >= 0 && L.conv_taps <= 64 && L.softcap >= 0.f && L.bias_dist >= 0, B200_ERR_INVALID,
+                     "stack_create: layer %d: bad attention sizes", l);
+        B200_REQUIRE(L.side == 0 || has_side(L), B200_ERR_UNSUPPORTED, "stack_create: layer %d: second mixer %d", l, L.side);
+        B200_REQUIRE(!has_side(L) || (L.side_inner > 0 && L.side_state > 0 && L.side_state <= 256 && L.side_rank > 0 && L.side_taps >= 1 && L.side_taps <= 64),
+                     B200_ERR_INVALID, "stack_create: layer %d: bad sizes of the selective scan", l);
+      }
+      B200_REQUIRE(L.mlp == B200_MLP_NONE || (L.mlp == B200_MLP_DENSE && L.ungated && L.ff > 0 && L.act >= 0 && L.act <= B200_ACT_RELU), B200_ERR_UNSUPPORTED,
+                   "stack_create: layer %d: the looped form has ungated dense feed-forwards", l);
+      if (has_side(L)) max_inner = std::max(max_inner, L.side_inner), max_proj = std::max(max_proj, selective_rows(L.side_rank, L.side_state));
     } else {
     B200_REQUIRE(L.mixer == B200_MIXER_ATTENTION, B200_ERR_UNSUPPORTED, "stack_create: layer %d: unknown mixer %d", l, L.mixer);
     B200_REQUIRE(L.heads > 0 && L.kv_heads > 0 && L.heads % L.kv_heads == 0 && L.dim > 0 && L.vdim > 0 && L.dim % 2 == 0 &&
@@ -946,6 +1167,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
     if (L.shared_ff > 0) max_gu = std::max(max_gu, 2 * L.shared_ff), max_ffa = std::max(max_ffa, L.shared_ff);
   }
   const bool par = cfg->form == B200_FORM_PARALLEL, post = cfg->form == B200_FORM_POSTNORM, hyp = cfg->form == B200_FORM_HYPER;
+  const bool loop = cfg->form == B200_FORM_LOOPED;
   B200_REQUIRE(par || ((hyp || !cfg->canon_taps) && !cfg->depth_avg && !cfg->bigram_buckets && cfg->logit_softcap == 0.f), B200_ERR_UNSUPPORTED,
                "stack_create: depth average, bigram rows and the logit cap belong to the parallel form, the input convolution to it and the multi-stream form");
   B200_REQUIRE(!hyp || (cfg->streams >= 1 && cfg->streams <= B200_MAX_STREAMS && cfg->canon_taps >= 0 && cfg->canon_taps <= 16 &&
@@ -1014,6 +1236,28 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
     }
     M->slot_floats = std::max<int64_t>(off, 4);
   }
+  if (loop) {
+    // one slot, per entry of the list: attention: the tails of the q | k | v convolution [conv_taps - 1][channels] and of the second mixer's
+    // [side_taps - 1][side_inner], the scan's state [side_inner][side_state]; retention: the state [heads][vdim][dim]
+    int64_t off = 0;
+    for (int l = 0; l < cfg->n_layers; ++l) {
+      const b200_stack_layer& L = layers[l];
+      StackLayerW& W = M->w[l];
+      if (is_retention(L)) {
+        W.rec_off = off;
+        off = up(off + (int64_t)L.heads * L.vdim * L.dim, 4);
+        continue;
+      }
+      W.ctail_off = off;
+      off = up(off + (int64_t)std::max(L.conv_taps - 1, 0) * attn_channels(L), 4);
+      if (!has_side(L)) continue;
+      W.tail2_off = off;
+      off = up(off + (int64_t)(L.side_taps - 1) * L.side_inner, 4);
+      W.rec_off = off;
+      off = up(off + (int64_t)L.side_inner * L.side_state, 4);
+    }
+    M->slot_floats = std::max<int64_t>(off, 4);
+  }
   b200_model_cfg& mc = c->cfg;
   memset(&mc, 0, sizeof(mc));
   mc.hidden = cfg->width;
@@ -1054,6 +1298,11 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       if (layers[l].shared_ff > 0) {
         shapes.push_back({(layers[l].ungated ? 1 : 2) * layers[l].shared_ff, (int)Wd});
         shapes.push_back({(int)Wd, layers[l].shared_ff});
+      }
+      if (has_side(layers[l])) {
+        shapes.push_back({selective_rows(layers[l].side_rank, layers[l].side_state), layers[l].side_inner});
+        shapes.push_back({layers[l].side_inner, selective_dt_pad(layers[l].side_rank)});
+        shapes.push_back({(int)Wd, layers[l].side_inner});
       }
       if (is_latent(layers[l]) && layers[l].q_rank > 0) shapes.push_back({layers[l].heads * layers[l].dim, layers[l].q_rank});
       if (is_delta(layers[l])) {
@@ -1097,7 +1346,13 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       if (is_latent(layers[l]) && latent_attn_mma_supported(layers[l].heads, layers[l].kv_rank + layers[l].rot_dim, layers[l].kv_rank))
         // splitting only happens below one CTA per SM: at most 148 * 16 pairs, 16 splits
         M->lat_ws_bytes = std::max<int64_t>(M->lat_ws_bytes, std::min<int64_t>(T * layers[l].heads, 148 * 16) * 16 * (layers[l].kv_rank + 2) * 4);
-  if ((post || hyp) && !cfg->f32)
+  M->ret_ws_bytes = 16;
+  if (loop && !cfg->f32)
+    for (int l = 0; l < cfg->n_layers; ++l)
+      if (is_retention(layers[l]) && retention_chunk_supported(layers[l].dim, layers[l].vdim))
+        M->ret_ws_bytes = std::max<int64_t>(M->ret_ws_bytes, retention_chunk_workspace_bytes((int)T, (int)std::min<int64_t>(T, cfg->n_state_slots), layers[l].heads,
+                                                                                             layers[l].dim, layers[l].vdim));
+  if ((post || hyp || loop) && !cfg->f32)
     for (int l = 0; l < cfg->n_layers; ++l)
       if (layers[l].mixer == B200_MIXER_ATTENTION && paged_attn_mma_supported(layers[l].heads, layers[l].kv_heads, layers[l].dim, layers[l].vdim))
         M->lat_ws_bytes = std::max<int64_t>(M->lat_ws_bytes, std::min<int64_t>(T * layers[l].heads, 148 * 16) * 16 * (layers[l].vdim + 2) * 4);
@@ -1122,20 +1377,26 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       {(void**)&M->attn_tc_ws, M->attn_tc_ws_bytes},
       {(void**)&M->attn_wide, tc_heads ? T * tc_heads * kHeadDim * 2 : 16},
       {(void**)&c->logits, R * (int64_t)c->logits_ld * 2},
-      {(void**)&c->logits_f32, (cfg->f32 || par || post || hyp) ? R * (int64_t)c->logits_ld * 4 : 16},
+      {(void**)&c->logits_f32, (cfg->f32 || par || post || hyp || loop) ? R * (int64_t)c->logits_ld * 4 : 16},
       {(void**)&M->results, par && cfg->depth_avg ? (int64_t)(cfg->n_layers + 1) * T * Wd * 4 : 16},
       {(void**)&M->h1f, (par || hyp) && cfg->canon_taps >= 1 ? T * Wd * 4 : 16},
       {(void**)&M->hc, (par || hyp) ? T * Wd * es : 16},
       {(void**)&M->xs, hyp ? (int64_t)cfg->streams * T * Wd * 4 : 16},
       {(void**)&M->lat, T * std::max(max_lat, 1) * es},
-      {(void**)&M->y2, (par || post || hyp) ? T * Wd * es : 16},
+      {(void**)&M->y2, (par || post || hyp || loop) ? T * Wd * es : 16},
       {(void**)&M->y3, par ? T * Wd * es : 16},
       {(void**)&M->gu, T * std::max(max_gu, 1) * es},
       {(void**)&M->ffa, T * std::max(max_ffa, 1) * es},
       {(void**)&M->gates_buf, T * std::max(max_gates, 1) * 4},
       {(void**)&M->oraw, (max_gates || max_dav) ? T * max_a * 4 : 16},
-      {(void**)&M->head_f32, (par || post || hyp) ? R * (int64_t)cfg->vocab * 4 : 16},
+      {(void**)&M->head_f32, (par || post || hyp || loop) ? R * (int64_t)cfg->vocab * 4 : 16},
       {(void**)&M->seq_start, (T + 2) * 4},
+      {(void**)&M->eout, loop ? T * Wd * 4 : 16},
+      {(void**)&M->dtp, T * std::max(max_inner, 1) * 4},
+      {(void**)&M->xc, T * std::max(max_inner, 1) * es},
+      {(void**)&M->xp, T * std::max(max_proj, 1) * es},
+      {(void**)&M->ssy, T * std::max(max_inner, 1) * es},
+      {(void**)&M->ret_ws, M->ret_ws_bytes},
       {(void**)&M->cq, T * std::max(max_qrank, 1) * es},
       {(void**)&M->qh, T * std::max(max_qh, 1) * es},
       {(void**)&M->a2, T * std::max(max_dhd, 1) * es},
@@ -1172,7 +1433,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
     *it.p = static_cast<char*>(c->pool) + off;
     off += up(std::max<int64_t>(it.bytes, 16), 1024);
   }
-  if (!cfg->f32 && !par && !post && !hyp) c->logits_f32 = nullptr;
+  if (!cfg->f32 && !par && !post && !hyp && !loop) c->logits_f32 = nullptr;
   *out = c;
   return B200_OK;
 }
@@ -1187,7 +1448,8 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
   const bool post = M->cfg.form == B200_FORM_POSTNORM;
   const bool hyp = M->cfg.form == B200_FORM_HYPER;
   const bool global = kind == B200_SW_EMBED || kind == B200_SW_FINAL_NORM || kind == B200_SW_HEAD || kind == B200_SW_BIGRAM ||
-                      kind == B200_SW_FINAL_NORM_BIAS;
+                      kind == B200_SW_FINAL_NORM_BIAS || kind == B200_SW_EMBED_NORM;
+  const bool loop = M->cfg.form == B200_FORM_LOOPED;
   if (!global) B200_REQUIRE(layer >= 0 && layer < M->cfg.n_layers, B200_ERR_INVALID, "stack_set_weight: layer %d out of range", layer);
   const b200_stack_layer L = global ? b200_stack_layer{} : M->layers[layer];
   switch (kind) {
@@ -1200,7 +1462,23 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_NORM_MIX_POST_BIAS: case B200_SW_NORM_MLP_POST_BIAS: case B200_SW_FINAL_NORM_BIAS: er = Wd; break;
     case B200_SW_Q_LATENT_NORM: er = L.q_rank; break;
     case B200_SW_UQ: er = (int64_t)L.heads * L.dim; ec = L.q_rank; break;
-    case B200_SW_CONV: er = 2 * (int64_t)L.kv_heads * L.dim + (int64_t)L.heads * L.vdim; ec = L.conv_taps; break;
+    case B200_SW_EMBED_NORM: case B200_SW_LOOP_STEP: case B200_SW_OUT_MAIN: case B200_SW_OUT_SIDE: case B200_SW_MLP_DOWN_BIAS: er = Wd; break;
+    case B200_SW_QKV_BIAS: er = qkv_rows(L); break;
+    case B200_SW_DIST_BIAS: er = L.heads; ec = L.bias_dist; break;
+    case B200_SW_DECAY: er = L.heads; break;
+    case B200_SW_SIDE_CONV: er = L.side_inner; ec = L.side_taps; break;
+    case B200_SW_SIDE_CONV_BIAS: case B200_SW_SIDE_DT_BIAS: case B200_SW_SIDE_SKIP: er = L.side_inner; break;
+    case B200_SW_SIDE_PROJ: er = selective_rows(L.side_rank, L.side_state); ec = L.side_inner; break;
+    case B200_SW_SIDE_DT: er = L.side_inner; ec = selective_dt_pad(L.side_rank); break;
+    case B200_SW_SIDE_A: er = L.side_inner; ec = L.side_state; break;
+    case B200_SW_SIDE_O: er = Wd; ec = L.side_inner; break;
+    case B200_SW_MLP_UP_BIAS: er = L.ff; break;
+    case B200_SW_CONV:
+      if (L.mixer == B200_MIXER_ATTENTION) {
+        er = attn_channels(L), ec = L.conv_taps;
+        break;
+      }
+      er = 2 * (int64_t)L.kv_heads * L.dim + (int64_t)L.heads * L.vdim; ec = L.conv_taps; break;
     case B200_SW_CONV_BIAS: er = 2 * (int64_t)L.kv_heads * L.dim + (int64_t)L.heads * L.vdim; break;
     case B200_SW_DECAY_UP: er = (int64_t)L.heads * L.dim; ec = L.decay_rank; break;
     case B200_SW_DECAY_BIAS: er = (head_decay(L) || is_ssd(L)) ? L.heads : (int64_t)L.heads * L.dim; break;
@@ -1232,6 +1510,18 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_SHARED_DOWN: er = Wd; ec = L.shared_ff; break;
     default: B200_REQUIRE(false, B200_ERR_INVALID, "stack_set_weight: unknown kind %d", kind);
   }
+  B200_REQUIRE(kind < B200_SW_EMBED_NORM || loop, B200_ERR_INVALID, "stack_set_weight: kind %d belongs to the looped form", kind);
+  if (loop) {
+    const bool dense = kind == B200_SW_MLP_GATE_UP || kind == B200_SW_MLP_DOWN || kind == B200_SW_MLP_UP_BIAS || kind == B200_SW_MLP_DOWN_BIAS;
+    const bool side = (kind >= B200_SW_SIDE_CONV && kind <= B200_SW_OUT_SIDE);
+    B200_REQUIRE(kind <= B200_SW_QKV || kind == B200_SW_O || kind >= B200_SW_EMBED_NORM || dense || kind == B200_SW_CONV, B200_ERR_INVALID,
+                 "stack_set_weight: kind %d belongs to another layer form", kind);
+    B200_REQUIRE(!side || has_side(L), B200_ERR_INVALID, "stack_set_weight: layer %d has no second mixer", layer);
+    B200_REQUIRE(kind != B200_SW_DECAY || is_retention(L), B200_ERR_INVALID, "stack_set_weight: layer %d has no retention", layer);
+    B200_REQUIRE((kind != B200_SW_CONV && kind != B200_SW_DIST_BIAS) || L.mixer == B200_MIXER_ATTENTION, B200_ERR_INVALID,
+                 "stack_set_weight: layer %d has no attention", layer);
+    B200_REQUIRE(!dense || L.mlp == B200_MLP_DENSE, B200_ERR_INVALID, "stack_set_weight: layer %d has no dense feed-forward", layer);
+  } else {
   B200_REQUIRE(kind < B200_SW_BIGRAM || par || post || hyp, B200_ERR_INVALID, "stack_set_weight: kind %d belongs to another layer form", kind);
   B200_REQUIRE(kind < B200_SW_NORM_MIX_POST_BIAS || post || hyp || kind == B200_SW_MLP_GATE_UP_INTERLEAVED, B200_ERR_INVALID,
                "stack_set_weight: kind %d belongs to the post-norm form", kind);
@@ -1259,6 +1549,7 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
                  "stack_set_weight: interleaved gate|up rows need the bf16 mode, ff %% 64 == 0 and width %% 8 == 0");
   if (kind == B200_SW_MLP_GATE_UP || kind == B200_SW_MLP_DOWN || kind == B200_SW_MLP_GATE_UP_INTERLEAVED)
     B200_REQUIRE(L.mlp == B200_MLP_DENSE, B200_ERR_INVALID, "stack_set_weight: layer %d has no dense feed-forward", layer);
+  }
   B200_REQUIRE(rows == er && cols == ec, B200_ERR_INVALID, "stack_set_weight: kind %d of layer %d expects [%lld,%lld], got [%lld,%lld]",
                kind, layer, (long long)er, (long long)ec, (long long)rows, (long long)cols);
   if ((kind >= B200_SW_ROUTER && kind <= B200_SW_EXPERT_DOWN && kind != B200_SW_ROUTER_BIAS) || kind == B200_SW_SHARED_UP ||
@@ -1316,6 +1607,23 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_CONV_BIAS: M->w[layer].conv_b = f; break;
     case B200_SW_SKIP: M->w[layer].skip = f; break;
     case B200_SW_MLP_ACT: M->w[layer].mlp_act = f; break;
+    case B200_SW_EMBED_NORM: M->embed_norm = f; break;
+    case B200_SW_LOOP_STEP: M->w[layer].loop_step = f; break;
+    case B200_SW_QKV_BIAS: M->w[layer].qkv_b = b; break;
+    case B200_SW_DIST_BIAS: M->w[layer].dist_bias = f; break;
+    case B200_SW_DECAY: M->w[layer].decay = f; break;
+    case B200_SW_SIDE_CONV: M->w[layer].side_conv = f; break;
+    case B200_SW_SIDE_CONV_BIAS: M->w[layer].side_conv_b = f; break;
+    case B200_SW_SIDE_PROJ: M->w[layer].side_proj = b; break;
+    case B200_SW_SIDE_DT: M->w[layer].side_dt = b; break;
+    case B200_SW_SIDE_DT_BIAS: M->w[layer].side_dt_b = f; break;
+    case B200_SW_SIDE_A: M->w[layer].side_a = f; break;
+    case B200_SW_SIDE_SKIP: M->w[layer].side_skip = f; break;
+    case B200_SW_SIDE_O: M->w[layer].side_o = b; break;
+    case B200_SW_OUT_MAIN: M->w[layer].out_main = f; break;
+    case B200_SW_OUT_SIDE: M->w[layer].out_side = f; break;
+    case B200_SW_MLP_UP_BIAS: M->w[layer].mlp_up_b = b; break;
+    case B200_SW_MLP_DOWN_BIAS: M->w[layer].mlp_down_b = b; break;
   }
   return B200_OK;
 }
@@ -1799,4 +2107,89 @@ extern "C" int b200_ssd_gate_norm(int32_t f32, const float* o, const float* xn, 
                                   void* out, int32_t T, int32_t heads, int32_t vdim, int32_t norm_groups, float eps, void* stream) {
   B200_REQUIRE(o && xn && skip && z && w && out && heads > 0 && vdim > 0, B200_ERR_INVALID, "ssd_gate_norm: bad argument");
   return ssd_gate_norm(f32 != 0, o, xn, skip, z, ldz, w, out, T, heads, vdim, norm_groups, eps, (cudaStream_t)stream);
+}
+
+// ---- per-kernel entry points of the looped form -------------------------------------------------------------------------------
+extern "C" int b200_rms_sandwich(int32_t f32, float* x, const void* y, const void* y_b, const float* w_a, const float* w_b, const float* w_post,
+                                 int32_t init, float* e_out, float* tap, const float* e, const float* step, const float* w_next, void* out,
+                                 const int32_t* rows, int32_t R, int32_t width, float eps, void* stream) {
+  B200_REQUIRE(x && width > 0 && R >= 0, B200_ERR_INVALID, "rms_sandwich: bad argument");
+  return rms_sandwich(f32 != 0, x, y, y_b, w_a, w_b, w_post, init != 0, e_out, tap, e, step, w_next, out, rows, R, width, eps, (cudaStream_t)stream);
+}
+
+extern "C" int b200_retention_step(int32_t f32, const void* fused, int64_t ld, const float* rot, int32_t rot_dims, int32_t half_layout, int64_t max_pos,
+                                   const float* decay, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state,
+                                   int64_t slot_stride, void* out, int32_t S, int32_t heads, int32_t dim, int32_t vdim, float eps, int32_t max_rows,
+                                   void* stream) {
+  B200_REQUIRE(fused && decay && positions && seq_start && seq_slots && state && out && max_pos > 0, B200_ERR_INVALID, "retention_step: null argument");
+  return retention_step(f32 != 0, fused, ld, rot, rot ? rot_dims : 0, half_layout != 0, max_pos, decay, positions, seq_start, seq_slots, state, slot_stride,
+                        out, S, heads, dim, vdim, eps, max_rows, (cudaStream_t)stream);
+}
+
+extern "C" int b200_retention_chunk_supported(int32_t dim, int32_t vdim) { return retention_chunk_supported(dim, vdim) ? 1 : 0; }
+
+extern "C" int64_t b200_retention_chunk_workspace_bytes(int32_t T, int32_t S, int32_t heads, int32_t dim, int32_t vdim) {
+  return retention_chunk_workspace_bytes(T, S, heads, dim, vdim);
+}
+
+extern "C" int b200_retention_chunk(const void* fused, int64_t ld, const float* rot, int32_t rot_dims, int32_t half_layout, int64_t max_pos,
+                                    const float* decay, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state,
+                                    int64_t slot_stride, void* out, int32_t T, int32_t S, int32_t heads, int32_t dim, int32_t vdim, float eps,
+                                    int32_t min_rows, void* ws, void* stream) {
+  B200_REQUIRE(fused && decay && positions && seq_start && seq_slots && state && out && max_pos > 0, B200_ERR_INVALID, "retention_chunk: null argument");
+  return retention_chunk(fused, ld, rot, rot ? rot_dims : 0, half_layout != 0, max_pos, decay, positions, seq_start, seq_slots, state, slot_stride, out, T, S,
+                         heads, dim, vdim, eps, min_rows, ws, (cudaStream_t)stream);
+}
+
+extern "C" int b200_conv_inputs(int32_t f32, const void* fused, int64_t ld, const float* conv_a, int32_t taps_a, float* tails_a, const float* conv_x,
+                                const float* bias_x, int32_t taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions,
+                                const int32_t* row_to_seq, const int32_t* seq_start, const int32_t* seq_slots, const int32_t* slots, float* q_out,
+                                void* kc, void* vc, void* xc, int32_t T, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t inner,
+                                int32_t block_size, int32_t one_row, void* stream) {
+  B200_REQUIRE(fused && T >= 0 && heads >= 0 && inner >= 0 && block_size > 0, B200_ERR_INVALID, "conv_inputs: bad argument");
+  return conv_inputs(f32 != 0, fused, ld, conv_a, taps_a, tails_a, conv_x, bias_x, taps_x, tails_x, slot_stride, positions, row_to_seq, seq_start, seq_slots,
+                     slots, q_out, kc, vc, xc, T, heads, kv_heads, dim, vdim, inner, block_size, one_row != 0, (cudaStream_t)stream);
+}
+
+extern "C" int32_t b200_selective_rows(int32_t rank, int32_t state) { return selective_rows(rank, state); }
+
+extern "C" int b200_selective_scan(int32_t f32, const void* xc, const void* bc, int64_t ldbc, int32_t b_off, const float* dt_pre, const float* dt_bias,
+                                   const float* A, const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start,
+                                   const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t S, int32_t inner, int32_t n_state,
+                                   void* stream) {
+  B200_REQUIRE(xc && bc && dt_pre && dt_bias && A && D && z && positions && seq_start && seq_slots && state && out, B200_ERR_INVALID,
+               "selective_scan: null argument");
+  return selective_scan(f32 != 0, xc, bc, ldbc, b_off, dt_pre, dt_bias, A, D, z, ldz, positions, seq_start, seq_slots, state, slot_stride, out, S, inner,
+                        n_state, (cudaStream_t)stream);
+}
+
+extern "C" int b200_paged_attn_biased(int32_t f32, int32_t form, const float* q, const void* kc, const void* vc, const int32_t* block_table,
+                                      int32_t bt_stride, const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, void* out,
+                                      int32_t T, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t block_size, float scale,
+                                      int32_t window, float softcap, const float* dist_bias, int32_t bias_dist, const void* gate, int64_t ldg, void* ws,
+                                      int32_t n_splits, float* part, void* stream) {
+  B200_REQUIRE(q && kc && vc && block_table && ctx_lens && positions && out && block_size > 0 && window >= 0 && (!dist_bias || bias_dist > 0) &&
+                   softcap >= 0.f && (form == 0 || ws) && form >= 0 && form <= 2,
+               B200_ERR_INVALID, "paged_attn_biased: bad argument");
+  AttnExtra ex;
+  ex.softcap = softcap, ex.dist_bias = dist_bias, ex.bias_dist = bias_dist, ex.gate = gate, ex.ldg = ldg;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (form == 2) {
+    B200_REQUIRE(!f32, B200_ERR_UNSUPPORTED, "paged_attn_biased: the tensor-core form takes bf16 caches");
+    int rc = paged_attn_runs_plan(row_to_seq, ctx_lens, T, ws, s);
+    if (rc) return rc;
+    return paged_attn_mma(q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, block_table, bt_stride, row_to_seq, ctx_lens, (__nv_bfloat16*)out,
+                          static_cast<const int32_t*>(ws) + 8, static_cast<const int32_t*>(ws), T, heads, kv_heads, dim, vdim, block_size, scale, nullptr, s,
+                          n_splits, part, window, ex);
+  }
+  return paged_attn_anydim(f32 != 0, q, kc, vc, block_table, bt_stride, row_to_seq, ctx_lens, positions, nullptr, 1ll << 40, out, T, heads, kv_heads, dim,
+                           vdim, block_size, scale, form, ws, s, 0, 0, nullptr, window, ex);
+}
+
+extern "C" int b200_linear_bias_act(int32_t f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy, int32_t T,
+                                    int32_t n_out, int32_t k, int32_t act, void* ws, int64_t ws_bytes, void* stream) {
+  B200_REQUIRE(x && w && y && T >= 0 && n_out > 0 && k > 0 && act <= B200_ACT_RELU, B200_ERR_INVALID, "linear_bias_act: bad argument");
+  if (T == 0) return B200_OK;
+  return linear_ex(f32 != 0, y_f32 != 0 || f32 != 0, x, ldx, (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias, y, ldy, T, n_out, k, act, ws, ws_bytes,
+                   (cudaStream_t)stream);
 }

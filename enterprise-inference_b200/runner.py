@@ -399,6 +399,8 @@ class StackRunner(ModelRunner):
     by layer), fp32 cos|sin tables shared between layers of equal rotation.  dtype "float32" runs activations, caches and
     matrix products in true fp32."""
 
+    _shared_uploads = None   # while weights load: source tensor -> device tensor (layers that run several times)
+
     def __init__(self, cfg, device: Optional[torch.device] = None, *, max_tokens: int = 2048, max_model_len: int = 8192,
                  block_size: int = 64, n_blocks: Optional[int] = None, kv_cache_gib: Optional[float] = None,
                  graphs: bool = True, dtype: str = "bfloat16", max_logit_rows: int = 512, tp_rank: int = 0, tp_world: int = 1,
@@ -437,19 +439,42 @@ class StackRunner(ModelRunner):
                 self._tables.append(spec.table(max(max_model_len, 16)).to(self.device))
             return keys[k]
 
-        from .config import AttentionSpec, ChannelDeltaSpec, DupolornConfig, FutidraConfig, HeadDeltaSpec, MLSTMSpec, RudolixConfig, StateSpaceSpec
+        from .config import (AttentionSpec, BofusunConfig, ChannelDeltaSpec, DupolornConfig, FutidraConfig, HeadDeltaSpec, MLSTMSpec, RetentionSpec,
+                             RudolixConfig, StateSpaceSpec, distance_entries)
         self.parallel = isinstance(cfg, DupolornConfig)
         self.postnorm = isinstance(cfg, FutidraConfig)
         self.hyper = isinstance(cfg, RudolixConfig)
+        self.looped = isinstance(cfg, BofusunConfig)
+        # what runs, in order: a looped layer once per pass, each run with its own cache and state
+        runs = cfg.layer_runs() if self.looped else [(i, None) for i in range(len(cfg.layers))]
+        self.run_layers = [cfg.layers[i] for i, _ in runs]
         # dense feed-forwards of the post-norm form in bf16: gate activation and product in the gate|up linear's epilogue
         self.fuse_gate_up = self.postnorm and not self.f32 and os.environ.get("B200_STACK_FUSE_GATE_UP", "1") != "0"
-        stateful = (self.parallel or self.postnorm or self.hyper) and cfg.needs_state
+        stateful = (self.parallel or self.postnorm or self.hyper or self.looped) and cfg.needs_state
         self.n_state_slots = int(n_state_slots) if stateful else 0
         if stateful and self.n_state_slots <= 0:
             raise ValueError("this model keeps per-sequence state: n_state_slots must be positive")
         layers = (_abi.StackLayer * cfg.n_layers)()
-        for i, L in enumerate(cfg.layers):
+        for i, L in enumerate(self.run_layers):
             a, f = L.mixer, L.mlp
+            if self.looped:
+                if isinstance(a, RetentionSpec):
+                    d = dict(mixer=_abi.MIXER_RETENTION, heads=a.heads, kv_heads=a.heads, dim=a.dim, vdim=a.vdim, rot_dims=a.rot.dims if a.rot else 0,
+                             rot_table=table_of(a.rot), vrot_table=-1, mixer_flags=_abi.MIXF_ROT_HALF if a.rot_half else 0)
+                else:
+                    flags = _abi.MIXF_NO_QK_NORM | (_abi.MIXF_QKV_BIAS if a.bias else 0) | (_abi.MIXF_HEAD_GATE if a.head_gate else 0)
+                    d = dict(mixer=_abi.MIXER_ATTENTION, heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, rot_table=-1, vrot_table=-1,
+                             scale=a.scale, mixer_flags=flags, window=a.window, conv_taps=a.conv, softcap=a.softcap,
+                             bias_dist=distance_entries(a.window, a.bias_max) if a.bias_max > 0 else 0)
+                    if L.side is not None:
+                        s = L.side
+                        d.update(side=_abi.MIXER_SELECTIVE, side_inner=s.inner, side_state=s.state, side_rank=s.dt_rank, side_taps=s.conv)
+                if f is not None:
+                    d.update(mlp=_abi.MLP_DENSE, ff=f.ff, act=_abi.ACTS[f.act], ungated=int(not f.gated))
+                if runs[i][1] is not None and runs[i][0] == cfg.loop_start:
+                    d.update(loop_step=1, loop_add=int(runs[i][1] > 0))
+                layers[i] = _abi.StackLayer(**d)
+                continue
             if self.hyper:
                 if isinstance(a, AttentionSpec):
                     flags = (0 if a.qk_norm else _abi.MIXF_NO_QK_NORM) | (_abi.MIXF_ROT_HALF if a.rot_half else 0) | \
@@ -520,6 +545,8 @@ class StackRunner(ModelRunner):
         if self.hyper:
             sc.form, sc.canon_taps, sc.n_state_slots = _abi.FORM_HYPER, cfg.canon_taps, self.n_state_slots
             sc.streams, sc.residual_mult = cfg.streams, cfg.residual_mult
+        if self.looped:
+            sc.form, sc.n_state_slots = _abi.FORM_LOOPED, self.n_state_slots
         h = C.c_void_p()
         _abi.check(self.lib.b200_stack_create(C.byref(sc), layers, C.byref(h)))
         self.ctx = h
@@ -529,11 +556,11 @@ class StackRunner(ModelRunner):
 
         # paged caches, one pair per layer: [n_blocks][kv_heads][block][row widths the ctx names], zero-filled
         self.cache_dims = []
-        for i in range(len(cfg.layers)):
+        for i in range(len(self.run_layers)):
             kd, vd = C.c_int32(), C.c_int32()
             _abi.check(self.lib.b200_stack_cache_dims(self.ctx, i, C.byref(kd), C.byref(vd)))
             self.cache_dims.append((kd.value, vd.value))
-        kvh = [getattr(L.mixer, "kv_heads", 1) for L in cfg.layers]
+        kvh = [getattr(L.mixer, "kv_heads", 1) for L in self.run_layers]
         per_block = max(sum(h * (kd + vd) for h, (kd, vd) in zip(kvh, self.cache_dims)) * (4 if self.f32 else 2) * block_size, 1)
         if n_blocks is None:
             if kv_cache_gib is None:
@@ -543,7 +570,7 @@ class StackRunner(ModelRunner):
         self.n_blocks = n_blocks
         cdt = torch.float32 if self.f32 else torch.bfloat16
         self.k_cache, self.v_cache = [], []
-        for i, L in enumerate(cfg.layers):
+        for i in range(len(self.run_layers)):
             kd, vd = self.cache_dims[i]
             k = torch.zeros((n_blocks, kvh[i], block_size, kd), dtype=cdt, device=self.device) if kd else None
             v = torch.zeros((n_blocks, kvh[i], block_size, vd), dtype=cdt, device=self.device) if vd else None
@@ -563,6 +590,11 @@ class StackRunner(ModelRunner):
 
     def _set(self, layer: int, kind: int, t: torch.Tensor):
         dt = torch.float32 if kind in _abi.SW_F32 else torch.bfloat16
+        src = t
+        if self._shared_uploads is not None and (id(src), kind) in self._shared_uploads:   # another pass of the same layer
+            t = self._shared_uploads[(id(src), kind)][1]
+            _abi.check(self.lib.b200_stack_set_weight(self.ctx, layer, kind, t.data_ptr(), t.shape[0], t.shape[1] if t.dim() == 2 else 1))
+            return
         t = t.to(device=self.device, dtype=dt)
         if kind == _abi.SW_MLP_GATE_UP and self.fuse_gate_up and (t.shape[0] // 2) % 64 == 0 and t.shape[1] % 8 == 0:
             # the tcgen05 linear activates and multiplies in its epilogue over slabs of 64 gate rows + the 64 matching up rows
@@ -571,13 +603,17 @@ class StackRunner(ModelRunner):
             t, kind = interleave_gate_up(t[:ff], t[ff:]), _abi.SW_MLP_GATE_UP_INTERLEAVED
         t = t.contiguous()
         self._weights.append(t)
+        if self._shared_uploads is not None:
+            self._shared_uploads[(id(src), kind)] = (src, t)
         rows, cols = (t.shape[0], t.shape[1]) if t.dim() == 2 else (t.shape[0], 1)
         _abi.check(self.lib.b200_stack_set_weight(self.ctx, layer, kind, t.data_ptr(), rows, cols))
 
     def load_weights(self, w: Dict[str, torch.Tensor]):
         from .weights import STACK_WEIGHT_MAPS
+        self._shared_uploads = {} if self.looped else None   # source tensor -> device tensor: the passes of a looped layer share one upload
         for layer, kind, t in STACK_WEIGHT_MAPS[self.cfg.architecture](w, self.cfg):
             self._set(layer, kind, t)
+        self._shared_uploads = None
 
     def _init_random_parallel(self, seed: int, std: float):
         from .config import MLSTMSpec
@@ -752,6 +788,58 @@ class StackRunner(ModelRunner):
                 self._set(i, A.SW_EXPERT_GATE_UP, rnd(f.experts * (2 if f.gated else 1) * f.ff, c.width))
                 self._set(i, A.SW_EXPERT_DOWN, rnd(f.experts * c.width, f.ff))
 
+    def _init_random_looped(self, seed: int, std: float):
+        from .config import RetentionSpec, distance_entries
+        c, A = self.cfg, _abi
+        g = torch.Generator(device=self.device)
+        g.manual_seed(seed)
+
+        def rnd(*shape, sd=std):
+            t = torch.empty(shape, dtype=torch.bfloat16, device=self.device)
+            t.normal_(0.0, sd, generator=g)
+            return t
+
+        def full(n, v=1.0):
+            return torch.full((n,), v, device=self.device)
+
+        self._shared_uploads = {}
+        runs = c.layer_runs()
+        self._set(0, A.SW_EMBED, rnd(c.vocab, c.width, sd=1.0))
+        self._set(0, A.SW_EMBED_NORM, full(c.width))
+        self._set(0, A.SW_FINAL_NORM, full(c.width))
+        self._set(0, A.SW_HEAD, rnd(c.vocab, c.width))
+        for r, (i, t) in enumerate(runs):
+            if t is not None and i == c.loop_start:
+                self._set(r, A.SW_LOOP_STEP, rnd(c.width, sd=0.1).float())
+        for i, L in enumerate(c.layers):
+            a, s, f = L.mixer, L.side, L.mlp
+            out = [(A.SW_NORM_MIX_PRE, full(c.width)), (A.SW_NORM_MIX_POST, full(c.width)), (A.SW_O, rnd(c.width, a.heads * a.vdim))]
+            if isinstance(a, RetentionSpec):
+                out += [(A.SW_QKV, rnd(2 * a.heads * (a.dim + a.vdim), c.width)), (A.SW_DECAY, torch.tensor(a.decay, device=self.device))]
+            else:
+                ch = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)
+                rows = ch + (2 * s.inner if s else 0) + (a.heads if a.head_gate else 0)
+                out += [(A.SW_QKV, rnd(rows, c.width)), (A.SW_QKV_BIAS, torch.zeros(rows, device=self.device, dtype=torch.bfloat16))]
+                if a.conv > 0:
+                    out.append((A.SW_CONV, rnd(ch, a.conv, sd=0.5).float()))
+                if a.bias_max > 0:
+                    out.append((A.SW_DIST_BIAS, rnd(a.heads, distance_entries(a.window, a.bias_max), sd=0.5).float()))
+                if s:
+                    states = torch.arange(1, s.state + 1, device=self.device, dtype=torch.float32)
+                    out += [(A.SW_SIDE_CONV, rnd(s.inner, s.conv, sd=0.5).float()), (A.SW_SIDE_CONV_BIAS, full(s.inner, 0.0)),
+                            (A.SW_SIDE_PROJ, rnd(s.proj_rows, s.inner)), (A.SW_SIDE_DT, rnd(s.inner, s.dt_pad)), (A.SW_SIDE_DT_BIAS, full(s.inner, -4.0)),
+                            (A.SW_SIDE_A, -states.repeat(s.inner, 1)), (A.SW_SIDE_SKIP, full(s.inner)), (A.SW_SIDE_O, rnd(c.width, s.inner)),
+                            (A.SW_OUT_MAIN, full(c.width)), (A.SW_OUT_SIDE, full(c.width))]
+            if f is not None:
+                out += [(A.SW_NORM_MLP_PRE, full(c.width)), (A.SW_NORM_MLP_POST, full(c.width)), (A.SW_MLP_GATE_UP, rnd(f.ff, c.width)),
+                        (A.SW_MLP_DOWN, rnd(c.width, f.ff)), (A.SW_MLP_UP_BIAS, torch.zeros(f.ff, device=self.device)),
+                        (A.SW_MLP_DOWN_BIAS, torch.zeros(c.width, device=self.device))]
+            for r, (j, _) in enumerate(runs):
+                if j == i:
+                    for kind, t in out:
+                        self._set(r, kind, t)
+        self._shared_uploads = None
+
     def set_step_slots(self, seq_slots: Optional[torch.Tensor]):
         """Device-pointer steps (step_device) of a model with state slots: int32 device tensor, one slot per sequence of the step."""
         self._step_slots = seq_slots
@@ -765,6 +853,8 @@ class StackRunner(ModelRunner):
             return self._init_random_postnorm(seed, std)
         if self.hyper:
             return self._init_random_hyper(seed, std)
+        if self.looped:
+            return self._init_random_looped(seed, std)
         c, A = self.cfg, _abi
         g = torch.Generator(device=self.device)
         g.manual_seed(seed)

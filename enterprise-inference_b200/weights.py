@@ -293,4 +293,64 @@ def rudolix_weights(w: Dict[str, torch.Tensor], cfg) -> Iterator[Tuple[int, int,
             yield i, A.SW_EXPERT_DOWN, torch.cat([w[f"{p}mlp.e{e}.down"] for e in range(f.experts)], 0)
 
 
-STACK_WEIGHT_MAPS = {"Bopilorn": bopilorn_weights, "Dupolorn": dupolorn_weights, "Futidra": futidra_weights, "Rudolix": rudolix_weights}
+def bofusun_weights(w: Dict[str, torch.Tensor], cfg) -> Iterator[Tuple[int, int, torch.Tensor]]:
+    """(layer RUN, b200_stack_weight kind, tensor) of a Bofusun checkpoint: `embed`, `embed.norm`, `head`, `final.norm`, `loop.step`, and per
+    layer i `l<i>.norm1|norm1b|norm2|norm2b`, the mixer `l<i>.mix.*` and the feed-forward `l<i>.mlp.up|down[.b]`.  A looped layer's
+    tensors are yielded once per pass, the same object every time (the runner uploads it once).  Norm weights stored around zero go
+    over as 1 + w.  Projections of the mixer's input are fused row-wise: retention q | k | v | g; attention beside a scan
+    q | k | v | x | z | g, with q | k | v biases and zeros for the rest; the q, k and v convolution kernels are stacked; the distance table
+    is expanded to one entry per distance and head; dt rows of the scan's projection are padded to a multiple of 8 with zeros; A goes
+    over as -exp(A_log)."""
+    from . import _abi as A
+    from .config import RetentionSpec, distance_bucket, distance_entries
+    runs = cfg.layer_runs()
+
+    def norm(name):
+        return 1.0 + w[name].float()
+
+    yield 0, A.SW_EMBED, w["embed"]
+    yield 0, A.SW_EMBED_NORM, norm("embed.norm")
+    yield 0, A.SW_FINAL_NORM, norm("final.norm")
+    yield 0, A.SW_HEAD, w["head"]
+    for r, (i, t) in enumerate(runs):
+        if t is not None and i == cfg.loop_start:
+            yield r, A.SW_LOOP_STEP, w["loop.step"][t]
+    for i, L in enumerate(cfg.layers):
+        p, a, s = f"l{i}.", L.mixer, L.side
+        out = [(A.SW_NORM_MIX_PRE, norm(p + "norm1")), (A.SW_NORM_MIX_POST, norm(p + "norm1b"))]
+        if isinstance(a, RetentionSpec):
+            m = p + "mix."
+            out += [(A.SW_QKV, torch.cat([w[m + n] for n in "qkvg"], 0)), (A.SW_DECAY, torch.tensor(a.decay, dtype=torch.float64)), (A.SW_O, w[m + "o"])]
+        else:
+            m = p + "mix.left."
+            rows = [w[m + "q"], w[m + "k"], w[m + "v"], w[p + "mix.right.in"], w[m + "g"]]
+            biases = [w[m + n + ".b"] for n in "qkv"]
+            biases.append(torch.zeros(sum(x.shape[0] for x in rows[3:]), dtype=biases[0].dtype))
+            out += [(A.SW_QKV, torch.cat(rows, 0)), (A.SW_QKV_BIAS, torch.cat(biases)), (A.SW_O, w[m + "o"])]
+            if a.conv > 0:
+                out.append((A.SW_CONV, torch.cat([w[m + n + ".conv"] for n in "qkv"], 0)))
+            if a.bias_max > 0:
+                rel = w[m + "rel"].float()
+                idx = torch.tensor([distance_bucket(d, rel.shape[0], a.bias_max) for d in range(distance_entries(a.window, a.bias_max))])
+                out.append((A.SW_DIST_BIAS, rel[idx].T.contiguous()))
+            b = p + "mix.right."
+            x, N = w[b + "x"], s.state
+            proj = torch.zeros((s.proj_rows, s.inner), dtype=x.dtype)
+            proj[:s.dt_rank] = x[:s.dt_rank]
+            proj[s.dt_pad:s.dt_pad + 2 * N] = x[s.dt_rank:]
+            dt = torch.zeros((s.inner, s.dt_pad), dtype=x.dtype)
+            dt[:, :s.dt_rank] = w[b + "dt"]
+            out += [(A.SW_SIDE_CONV, w[b + "conv"]), (A.SW_SIDE_CONV_BIAS, w[b + "conv.b"]), (A.SW_SIDE_PROJ, proj), (A.SW_SIDE_DT, dt),
+                    (A.SW_SIDE_DT_BIAS, w[b + "dt.b"]), (A.SW_SIDE_A, -torch.exp(w[b + "A_log"].double())), (A.SW_SIDE_SKIP, w[b + "D"]),
+                    (A.SW_SIDE_O, w[b + "o"]), (A.SW_OUT_MAIN, w[m + "out"]), (A.SW_OUT_SIDE, w[b + "out"])]
+        if L.mlp is not None:
+            out += [(A.SW_NORM_MLP_PRE, norm(p + "norm2")), (A.SW_NORM_MLP_POST, norm(p + "norm2b")), (A.SW_MLP_GATE_UP, w[p + "mlp.up"]),
+                    (A.SW_MLP_UP_BIAS, w[p + "mlp.up.b"]), (A.SW_MLP_DOWN, w[p + "mlp.down"]), (A.SW_MLP_DOWN_BIAS, w[p + "mlp.down.b"])]
+        for r, (j, _) in enumerate(runs):
+            if j == i:
+                for kind, tensor in out:
+                    yield r, kind, tensor
+
+
+STACK_WEIGHT_MAPS = {"Bopilorn": bopilorn_weights, "Dupolorn": dupolorn_weights, "Futidra": futidra_weights, "Rudolix": rudolix_weights,
+                     "Bofusun": bofusun_weights}

@@ -430,14 +430,40 @@ B200_API int b200_tp_allreduce(b200_ctx* ctx, int32_t buf_idx, const void* parti
  * c2 N(z^3) + c3 with N(v) = v / sqrt(mean(v^2) + eps) over the ff entries of a token;  B200_MLP_MOE with route_chosen: the
  * router bias joins the logits, the `top` largest logits are chosen and the mixing weights are the softmax over the chosen logits
  * alone; experts with B200_ACT_SWIGLU_CLAMP: g = min(gate h, act_limit), u = clamp(up h, -act_limit, act_limit),
- * down(g * sigmoid(1.702 g) * (u + 1)). */
-typedef enum b200_mixer_kind { B200_MIXER_ATTENTION = 1, B200_MIXER_LATENT = 2, B200_MIXER_MLSTM = 3, B200_MIXER_DELTA = 4, B200_MIXER_SSD = 5 } b200_mixer_kind;
+ * down(g * sigmoid(1.702 g) * (u + 1)).
+ *
+ * Fifth layer form (b200_stack_cfg.form = B200_FORM_LOOPED): RMS norms on both sides of every sublayer over one fp32 stream,
+ *   x += rms(sublayer(rms(x) * w_pre)) * w_post   (rms(v) = v / sqrt(mean(v^2) + eps); the weights given here are the whole factors),
+ * x starting from e = rms(table[id]) * w_embed.  Layers may be run several times: a layer list is given UNROLLED, every pass an entry
+ * of its own (its own cache and state; the entries of a layer share weight pointers).  Ahead of an entry with loop_add the stream
+ * takes e once more, ahead of one with loop_step it takes the vector B200_SW_LOOP_STEP of that entry.  Mixers of this form:
+ *
+ * B200_MIXER_RETENTION: linear attention with a fixed decay per head.  Fused rows q | k | v | gate (heads*dim, heads*dim, heads*vdim,
+ * heads*vdim); the leading rot_dims dimensions of q and k turn (B200_MIXF_ROT_HALF: i with i + rot_dims / 2); k *= dim^-1/2; per
+ * head  S = decay S + k v^T,  o = S^T q  (S fp32 [vdim][dim] in the state slot); o is brought to unit RMS per head and multiplied
+ * by silu(gate).
+ *
+ * B200_MIXER_ATTENTION with B200_MIXF_NO_QK_NORM: q / k / v rows with biases (B200_MIXF_QKV_BIAS), then, conv_taps > 0, a causal
+ * per-channel convolution over each of them (no activation; its last conv_taps - 1 inputs in the state slot); no rotation;
+ * score = softcap * tanh(scale q.k / softcap) (softcap 0: scale q.k) + dist_bias[head][min(i - j, bias_dist - 1)] (bias_dist 0: none),
+ * `window`, ordinary softmax; B200_MIXF_HEAD_GATE: one sigmoid gate per head.  With side = B200_MIXER_SELECTIVE a second mixer reads
+ * the same input; the fused rows are then q | k | v | x | z | gate and the mixer's result is half of rms(a) * w_main + rms(b) * w_side.
+ *
+ * B200_MIXER_SELECTIVE (selective scan): x | z of side_inner channels each; x passes a causal convolution of side_taps taps with bias
+ * and silu; dt = softplus(W_dt (W_x x)[:dt_rank] + bias) per channel, B and C the next 2 x side_state entries of W_x x; per channel c and
+ * state n  S = exp(dt A[c][n]) S + dt x B_n;  y = sum_n S C_n + D x;  y *= silu(z).
+ *
+ * Feed-forward of this form: B200_MLP_DENSE, ungated, act B200_ACT_RELU2, optional biases on both projections. */
+typedef enum b200_mixer_kind { B200_MIXER_ATTENTION = 1, B200_MIXER_LATENT = 2, B200_MIXER_MLSTM = 3, B200_MIXER_DELTA = 4, B200_MIXER_SSD = 5,
+                               B200_MIXER_RETENTION = 6, B200_MIXER_SELECTIVE = 7 } b200_mixer_kind;
 typedef enum b200_mlp_kind { B200_MLP_NONE = 0, B200_MLP_MOE = 1, B200_MLP_DENSE = 2 } b200_mlp_kind;
 typedef enum b200_act_kind { B200_ACT_SILU = 0, B200_ACT_GELU_TANH = 1, B200_ACT_RELU2 = 2, B200_ACT_RELU = 3, B200_ACT_SWIGLU_CLAMP = 4,
                              B200_ACT_POLYNORM = 5 } b200_act_kind;
-typedef enum b200_stack_form { B200_FORM_SANDWICH = 0, B200_FORM_PARALLEL = 1, B200_FORM_POSTNORM = 2, B200_FORM_HYPER = 3 } b200_stack_form;
+typedef enum b200_stack_form { B200_FORM_SANDWICH = 0, B200_FORM_PARALLEL = 1, B200_FORM_POSTNORM = 2, B200_FORM_HYPER = 3,
+                               B200_FORM_LOOPED = 4 } b200_stack_form;
 enum { B200_MIXF_SINK = 1, B200_MIXF_GATE = 2, B200_MIXF_HEAD_NORM = 4, B200_MIXF_VALUE_IS_KEY = 8, B200_MIXF_SINK_ONE = 16,
-       B200_MIXF_HEAD_GATE = 32, B200_MIXF_ROT_HALF = 64, B200_MIXF_NO_QK_NORM = 128, B200_MIXF_HEAD_DECAY = 256 };
+       B200_MIXF_HEAD_GATE = 32, B200_MIXF_ROT_HALF = 64, B200_MIXF_NO_QK_NORM = 128, B200_MIXF_HEAD_DECAY = 256,
+       B200_MIXF_QKV_BIAS = 512 };
 enum { B200_MAX_STREAMS = 8 };
 
 typedef struct b200_stack_layer {
@@ -466,6 +492,11 @@ typedef struct b200_stack_layer {
   int32_t norm_groups;                 /* state-space mixer: equal parts of the gated output that are normalised on their own (>= 1) */
   float act_limit;                     /* B200_ACT_SWIGLU_CLAMP: the clamp */
   int32_t route_chosen;                /* router: bias inside the logits, mixing weights = softmax over the chosen logits */
+  float softcap;                       /* attention scores: softcap * tanh(score / softcap) (0: none) */
+  int32_t bias_dist;                   /* attention: entries per head of the distance bias (0: none) */
+  int32_t side;                        /* second mixer beside the first: 0 or B200_MIXER_SELECTIVE */
+  int32_t side_inner, side_state, side_rank, side_taps;   /* selective scan: channels, states per channel, dt rank, taps */
+  int32_t loop_add, loop_step;         /* looped form: what the stream takes ahead of this entry */
 } b200_stack_layer;
 
 typedef struct b200_stack_cfg {
@@ -550,7 +581,26 @@ typedef enum b200_stack_weight {
   B200_SW_CANON_MLP = 45,          /* f32 [width][canon_taps]: input convolution of the feed-forward */
   B200_SW_CONV_BIAS = 46,          /* f32 [conv channels] */
   B200_SW_SKIP = 47,               /* f32 [heads]: D of a state-space mixer */
-  B200_SW_MLP_ACT = 48             /* f32 [4]: c0..c3 of B200_ACT_POLYNORM */
+  B200_SW_MLP_ACT = 48,            /* f32 [4]: c0..c3 of B200_ACT_POLYNORM */
+  /* looped form: the five norm kinds are whole factors [width].  QKV as the form's description says; CONV of an attention mixer is
+     [heads*dim + kv_heads*(dim + vdim)][conv_taps] (q, k, v channels); MLP_GATE_UP of an ungated feed-forward [ff][width]. */
+  B200_SW_EMBED_NORM = 49,         /* f32 [width] */
+  B200_SW_LOOP_STEP = 50,          /* f32 [width], per entry with loop_step */
+  B200_SW_QKV_BIAS = 51,           /* bf16 [fused rows]: bias of the fused projection (zeros where a group has none) */
+  B200_SW_DIST_BIAS = 52,          /* f32 [heads][bias_dist]: score bias by distance */
+  B200_SW_DECAY = 53,              /* f32 [heads]: the fixed decays of a retention mixer */
+  B200_SW_SIDE_CONV = 54,          /* f32 [side_inner][side_taps] */
+  B200_SW_SIDE_CONV_BIAS = 55,     /* f32 [side_inner] */
+  B200_SW_SIDE_PROJ = 56,          /* bf16 [b200_selective_rows][side_inner]: dt rows (padded to a multiple of 8 with zero rows), B, C, zero rows */
+  B200_SW_SIDE_DT = 57,            /* bf16 [side_inner][dt_rank padded to a multiple of 8 with zero columns] */
+  B200_SW_SIDE_DT_BIAS = 58,       /* f32 [side_inner] */
+  B200_SW_SIDE_A = 59,             /* f32 [side_inner][side_state]: A itself (negative) */
+  B200_SW_SIDE_SKIP = 60,          /* f32 [side_inner]: D */
+  B200_SW_SIDE_O = 61,             /* bf16 [width][side_inner] */
+  B200_SW_OUT_MAIN = 62,           /* f32 [width]: norm weights of the two results that are averaged */
+  B200_SW_OUT_SIDE = 63,           /* f32 [width] */
+  B200_SW_MLP_UP_BIAS = 64,        /* bf16 [ff] */
+  B200_SW_MLP_DOWN_BIAS = 65       /* bf16 [width] */
 } b200_stack_weight;
 
 B200_API int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_layer* layers, b200_ctx** out);
@@ -809,6 +859,59 @@ B200_API int b200_ssd_prep(int32_t f32, const void* fused, int64_t ld, const flo
                            void* stream);
 B200_API int b200_ssd_gate_norm(int32_t f32, const float* o, const float* xn, const float* skip, const void* z, int64_t ldz, const float* w,
                                 void* out, int32_t n_tokens, int32_t heads, int32_t vdim, int32_t norm_groups, float eps, void* stream);
+/* ---- per-kernel entry points of the looped form (unit tests, profiling); f32 as above ---- */
+/* One row pass over the fp32 stream x [T][width].  v = y, or half of rms(y) * w_a + rms(y_b) * w_b when y_b is given (activation rows); x += rms(v) *
+ * w_post; tap (optional) receives x; x += e (optional fp32 rows); x += step (optional [width]); with w_next, out = rms(x) * w_next.
+ * init: x = rms(x) * w_post instead of the sum (y NULL), copied to e_out when given.  rows: row r of the launch works on stream row
+ * rows[r], the stream is not written, out is dense. */
+B200_API int b200_rms_sandwich(int32_t f32, float* x, const void* y, const void* y_b, const float* w_a, const float* w_b, const float* w_post,
+                               int32_t init, float* e_out, float* tap, const float* e, const float* step, const float* w_next, void* out,
+                               const int32_t* rows, int32_t n_rows, int32_t width, float eps, void* stream);
+/* Retention, short portions (every sequence brings at most max_rows rows; longer ones are left alone, 0: no limit): fused rows
+ * q | k | v | gate of leading dimension ld -> rotation, k * dim^-1/2, recurrence over state [slot][heads][vdim][dim], unit RMS per head,
+ * silu gate -> out [T][heads*vdim] (activation type). */
+B200_API int b200_retention_step(int32_t f32, const void* fused, int64_t ld, const float* rot, int32_t rot_dims, int32_t half_layout,
+                                 int64_t max_pos, const float* decay, const int32_t* positions, const int32_t* seq_start,
+                                 const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t n_seqs, int32_t heads,
+                                 int32_t dim, int32_t vdim, float eps, int32_t max_rows, void* stream);
+/* The same over portions longer than min_rows rows in chunks of 64 rows on the tensor cores (bf16 rows; dim and vdim multiples of 16 up to
+ * 128 and rot_dims even: b200_retention_chunk_supported).  workspace: b200_retention_chunk_workspace_bytes. */
+B200_API int b200_retention_chunk_supported(int32_t dim, int32_t vdim);
+B200_API int64_t b200_retention_chunk_workspace_bytes(int32_t n_tokens, int32_t n_seqs, int32_t heads, int32_t dim, int32_t vdim);
+B200_API int b200_retention_chunk(const void* fused, int64_t ld, const float* rot, int32_t rot_dims, int32_t half_layout, int64_t max_pos,
+                                  const float* decay, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
+                                  float* state, int64_t slot_stride, void* out, int32_t n_tokens, int32_t n_seqs, int32_t heads, int32_t dim,
+                                  int32_t vdim, float eps, int32_t min_rows, void* workspace, void* stream);
+/* The inputs of an attention mixer with convolutions and of a selective scan beside it.  fused rows of leading dimension ld: q | k | v
+ * (attention channels), then x.  Convolved q -> q_out fp32 [T][heads*dim], k and v -> the paged caches at slot_mapping[t]; convolved x with
+ * bias and silu -> xc [T][inner] (activation type).  conv_w NULL / taps_a 0: no convolution of q, k, v; inner 0: no x.  tails_a [slot][taps_a - 1][q | k | v channels],
+ * tails_x [slot][taps_x - 1][inner] fp32, slot_stride floats apart; read here.  one_row: every sequence brings one row, the tails are
+ * advanced too (otherwise b200_delta_tails does it afterwards). */
+B200_API int b200_conv_inputs(int32_t f32, const void* fused, int64_t ld, const float* conv_a, int32_t taps_a, float* tails_a, const float* conv_x,
+                              const float* bias_x, int32_t taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions,
+                              const int32_t* row_to_seq, const int32_t* seq_start, const int32_t* seq_slots, const int32_t* slot_mapping,
+                              float* q_out, void* k_cache, void* v_cache, void* xc, int32_t n_tokens, int32_t heads, int32_t kv_heads,
+                              int32_t dim, int32_t vdim, int32_t inner, int32_t block_size, int32_t one_row, void* stream);
+/* Rows of W_x's product: dt (padded to a multiple of 8) | B | C, the total padded to a multiple of 8. */
+B200_API int32_t b200_selective_rows(int32_t rank, int32_t state);
+/* Selective scan: xc, z, out [T][inner] (activation type, z of leading dimension ldz), bc rows of leading dimension ldbc with B at b_off and C
+ * at b_off + n_state, dt_pre fp32 [T][inner] ahead of bias and softplus; state [slot][inner][n_state] fp32. */
+B200_API int b200_selective_scan(int32_t f32, const void* xc, const void* bc, int64_t ldbc, int32_t b_off, const float* dt_pre, const float* dt_bias,
+                                 const float* A, const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start,
+                                 const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t n_seqs, int32_t inner,
+                                 int32_t n_state, void* stream);
+/* Paged attention with a score cap and a distance bias: s = softcap tanh(scale q.k / softcap) + dist_bias[h][min(i - j, bias_dist - 1)]
+ * (softcap 0 / dist_bias NULL: off), optional window, per-head gate (gate[t * ldg + h], activation type, sigmoid; NULL: none).  form 0: one
+ * CTA per row and head, 1: runs of rows share K/V tiles, 2: tensor cores (bf16; n_splits, part as b200_paged_attn_mma). */
+B200_API int b200_paged_attn_biased(int32_t f32, int32_t form, const float* q, const void* k_cache, const void* v_cache, const int32_t* block_table,
+                                    int32_t bt_stride, const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, void* out,
+                                    int32_t n_tokens, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t block_size,
+                                    float scale, int32_t window, float softcap, const float* dist_bias, int32_t bias_dist, const void* gate,
+                                    int64_t ldg, void* workspace, int32_t n_splits, float* part, void* stream);
+/* The tcgen05 linear with bias and activation in its epilogue: y = act(x . w^T + bias) (bias NULL: none; act < 0: none, else b200_act_kind);
+ * y_f32: fp32 rows of n_out instead of bf16.  Shapes it cannot address and f32 take the CUDA-core linear. */
+B200_API int b200_linear_bias_act(int32_t f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy,
+                                  int32_t n_tokens, int32_t n_out, int32_t k, int32_t act, void* workspace, int64_t ws_bytes, void* stream);
 /* y[T][n_out] = x[T][k] . w[n_out][k]^T on CUDA cores in true fp32; w bf16, x / y fp32 or bf16. */
 B200_API int b200_linear_simt(int32_t x_f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, void* y, int64_t ldy,
                      int32_t n_tokens, int32_t n_out, int32_t k, void* stream);
