@@ -726,6 +726,42 @@ def _futidra_like_rudolix(Cf, name, z):
     return Cf.FutidraConfig(name=name, width=z["width"], vocab=z["vocab"], postln_alpha=2.0, layers=layers)
 
 
+# Bofusun beside Rudolix (the closest model of the framework: grouped-query attention with a value cache on the same tensor-core
+# kernel, recurrences with one decay per head and per-sequence state slots, ungated dense feed-forwards on the same linears) at equal
+# width, heads, head sizes, recurrence heads and inner size.  A pair of Bofusun layers is retention, then attention beside a selective scan, both
+# with a feed-forward: three mixers.  Rudolix gets the three as layers of their own (delta rule with a feed-forward, attention with
+# a feed-forward, state-space mixer without), one residual stream and no input convolutions, so that both run the same number of mixers and
+# feed-forwards.  The window is wider than every context of the comparison.
+BOFUSUN_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv=4, dim=128, r_heads=16, r_dim=128, r_vdim=128, inner=4096, state=16, dt_rank=128, s_heads=64, s_vdim=64,
+                  s_state=128, conv=4, window=4096, ff=4096, pairs=2, vocab=32768),
+    "w1024": dict(width=1024, heads=16, kv=4, dim=64, r_heads=8, r_dim=128, r_vdim=128, inner=2048, state=16, dt_rank=64, s_heads=32, s_vdim=64,
+                  s_state=64, conv=4, window=4096, ff=2048, pairs=2, vocab=32768),
+}
+
+
+def _bofusun_config(Cf, name, z):
+    ff = Cf.FeedForwardSpec(kind="dense", ff=z["ff"], act="relu2", gated=False, bias=True)
+    ret = Cf.RetentionSpec(heads=z["r_heads"], dim=z["r_dim"], vdim=z["r_vdim"], rot=Cf.RotarySpec(base=10000.0, dims=z["r_dim"]),
+                           decay=[1.0 - 2.0 ** (-5.0 - 5.0 * h / z["r_heads"]) for h in range(z["r_heads"])])
+    att = Cf.AttentionSpec(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5, window=z["window"], qk_norm=False,
+                           bias=True, conv=z["conv"], softcap=30.0, bias_max=1024.0, head_gate=True)
+    scan = Cf.SelectiveScanSpec(inner=z["inner"], state=z["state"], dt_rank=z["dt_rank"], conv=z["conv"])
+    pair = [Cf.StackLayerSpec(mixer=ret, mlp=ff), Cf.StackLayerSpec(mixer=att, mlp=ff, side=scan)]
+    return Cf.BofusunConfig(name=name, width=z["width"], vocab=z["vocab"], layers=pair * z["pairs"])
+
+
+def _rudolix_like_bofusun(Cf, name, z):
+    ff = Cf.FeedForwardSpec(kind="dense", ff=z["ff"], act="polynorm", gated=False)
+    att = Cf.AttentionSpec(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5,
+                           rot=Cf.RotarySpec(base=10000.0, dims=z["dim"]), qk_norm=False, rot_half=True, sink=True)
+    layers = [Cf.StackLayerSpec(mixer=Cf.HeadDeltaSpec(heads=z["r_heads"], kv_heads=z["r_heads"], dim=z["r_dim"], vdim=z["r_vdim"], conv=z["conv"]), mlp=ff),
+              Cf.StackLayerSpec(mixer=att, mlp=ff),
+              Cf.StackLayerSpec(mixer=Cf.StateSpaceSpec(heads=z["s_heads"], vdim=z["s_vdim"], state=z["s_state"], groups=1, norm_groups=1, conv=z["conv"]))]
+    return Cf.RudolixConfig(name=name, width=z["width"], vocab=z["vocab"], embed_scale=1.0, canon_taps=0, streams=1, residual_mult=1.0,
+                            layers=layers * z["pairs"])
+
+
 def _design_batch(R, n_seqs, ctx, n_new, bs, vocab):
     """n_seqs sequences that already hold ctx tokens and bring n_new rows each; the last row of each is a logit row."""
     import numpy as np
@@ -775,8 +811,8 @@ def run_design(args):
     sampler.start()
     t0 = time.monotonic()
     out = []
-    dup, fut, rud = args.design == "dupolorn", args.design == "futidra", args.design == "rudolix"
-    sizes = RUDOLIX_SIZES if rud else (FUTIDRA_SIZES if fut else (DUPOLORN_SIZES if dup else DESIGN_SIZES))
+    dup, fut, rud, bof = (args.design == n for n in ("dupolorn", "futidra", "rudolix", "bofusun"))
+    sizes = BOFUSUN_SIZES if bof else RUDOLIX_SIZES if rud else (FUTIDRA_SIZES if fut else (DUPOLORN_SIZES if dup else DESIGN_SIZES))
     names = [n for n in sizes if args.design_size in ("all", n)]
     for name in names:
         z = sizes[name]
@@ -784,6 +820,8 @@ def run_design(args):
             z = dict(z, experts=1, top=1, groups=1, keep=1)
         if rud:
             z = dict(z, groups=1, keep=1)
+        if bof:
+            z = dict(z, experts=1, top=1, groups=1, keep=1, layers=1)
         rot = Cf.RotarySpec(base=10000.0, dims=z["dim"], factor=4.0, original=4096, fast=32.0, slow=1.0, scaled=True)
         att = Cf.AttentionSpec(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5, rot=rot,
                                value_rot=Cf.RotarySpec(base=10000.0, dims=z["dim"]))
@@ -792,7 +830,10 @@ def run_design(args):
             z = {k: v for k, v in z.items() if k not in ("groups", "keep")}
         arms = {"bopilorn": Cf.BopilornConfig(name=name, width=z["width"], vocab=z["vocab"], embed_scale=1.0,
                                               layers=[Cf.StackLayerSpec(mixer=att, mlp=moe) for _ in range(z["layers"])])}
-        if rud:
+        if bof:
+            z = dict(sizes[name])
+            arms = {"bofusun": _bofusun_config(Cf, name, z), "rudolix": _rudolix_like_bofusun(Cf, name, z)}
+        elif rud:
             arms = {"rudolix": _rudolix_config(Cf, name, z), "futidra": _futidra_like_rudolix(Cf, name, z)}
         elif fut:
             arms = {"futidra": _futidra_config(Cf, name, z), "dupolorn": _dupolorn_dense_config(Cf, name, z)}
@@ -822,8 +863,9 @@ def run_design(args):
             torch.cuda.empty_cache()
         out.append(rec)
     clocks = sampler.stop(t0, time.monotonic())
-    emit({"metric": "design_compare", "design": "Rudolix" if rud else ("Futidra" if fut else ("Dupolorn" if dup else "Bopilorn")),
-          "closest": "futidra (attention with a value cache, delta rule on the same scan, state slots, dense feed-forwards)" if rud else
+    emit({"metric": "design_compare", "design": "Bofusun" if bof else "Rudolix" if rud else ("Futidra" if fut else ("Dupolorn" if dup else "Bopilorn")),
+          "closest": "rudolix with one stream (attention with a value cache, delta rule and state-space recurrence with state slots, ungated dense feed-forwards)"
+                     if bof else "futidra (attention with a value cache, delta rule on the same scan, state slots, dense feed-forwards)" if rud else
                      "dupolorn with dense feed-forwards (latent attention, matrix-memory recurrence, state slots)" if fut else
                      ("bopilorn (layer-list model with routed experts)" if dup else "llama (fixed decoder stack)"), "dtype": "bf16",
           "data": "synthetic, random-init weights", "steps": K, "warmup": W, "l2": "flushed between steps (512 MiB written)",
@@ -839,10 +881,10 @@ def main():
     ap.add_argument("--workload", default="llama8b-bs64", choices=sorted(WORKLOADS))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--headline-only", action="store_true", help="skip the `also` and `tp` sections of the default run")
-    ap.add_argument("--design", default=None, choices=["bopilorn", "dupolorn", "futidra", "rudolix"],
+    ap.add_argument("--design", default=None, choices=["bopilorn", "dupolorn", "futidra", "rudolix", "bofusun"],
                     help="instead of the default workload: prefill / decode throughput of this design beside the closest fixed-stack "
                          "model at equal size")
-    ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(DESIGN_SIZES) | set(DUPOLORN_SIZES) | set(FUTIDRA_SIZES) | set(RUDOLIX_SIZES)))
+    ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(DESIGN_SIZES) | set(DUPOLORN_SIZES) | set(FUTIDRA_SIZES) | set(RUDOLIX_SIZES) | set(BOFUSUN_SIZES)))
     args = ap.parse_args()
     claim_stdout()
     if args.design:
