@@ -204,7 +204,7 @@ SIGNATURES = {
                                    _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
     "b200_selective_rows": (_i32, [_i32, _i32]),
     "b200_selective_scan": (C.c_int, [_i32, _vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32,
-                                      _vp]),
+                                      _i32, _vp]),
     "b200_paged_attn_biased": (C.c_int, [_i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32,
                                          _f32, _vp, _i32, _vp, _i64, _vp, _i32, _vp, _vp]),
     "b200_linear_bias_act": (C.c_int, [_i32, _i32, _vp, _i64, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _i64, _vp]),

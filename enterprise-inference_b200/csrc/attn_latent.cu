@@ -165,8 +165,9 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
       float s1 = see1 ? Ss[row * kSsStride + lane + 32] * scale : -INFINITY;
       if constexpr (EX) {
         const float* brow = ex.dist_bias ? ex.dist_bias + (int64_t)(g * G + (i0 + row) % G) * ex.bias_dist : nullptr;
-        if (see0) s0 = score_shape(s0, ex.softcap, brow, c - 1 - j0, ex.bias_dist);
-        if (see1) s1 = score_shape(s1, ex.softcap, brow, c - 1 - j1, ex.bias_dist);
+        const float inv_cap2 = ex.softcap > 0.f ? 2.0f / ex.softcap : 0.f;
+        if (see0) s0 = score_shape_fast(s0, ex.softcap, inv_cap2, brow, c - 1 - j0, ex.bias_dist);
+        if (see1) s1 = score_shape_fast(s1, ex.softcap, inv_cap2, brow, c - 1 - j1, ex.bias_dist);
       }
       const float m_old = mrow[row];
       const float m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));

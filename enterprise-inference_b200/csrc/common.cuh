@@ -106,6 +106,13 @@ __device__ __forceinline__ float score_shape(float s, float cap, const float* bi
   return bias_row ? s + __ldg(bias_row + min(dist, n_dist - 1)) : s;
 }
 
+// the same for scores that come from bf16 products: tanh(z) = 1 - 2 / (1 + e^2z) on the hardware's exponential and reciprocal, an
+// absolute error of a few 1e-7 of the cap
+__device__ __forceinline__ float score_shape_fast(float s, float cap, float inv_cap2, const float* bias_row, int dist, int n_dist) {
+  if (cap > 0.f) s = cap - __fdividef(2.0f * cap, 1.0f + __expf(s * inv_cap2));
+  return bias_row ? s + __ldg(bias_row + min(dist, n_dist - 1)) : s;
+}
+
 // ---- Programmatic dependent launch -------------------------------------------------------
 // Every kernel of the step waits for its predecessor's memory here and lets its successor
 // start its prologue early; with no PDL attribute on the launch both are no-ops.
@@ -471,6 +478,6 @@ int selective_dt_pad(int rank);
 int selective_rows(int rank, int state);
 int selective_scan(bool f32, const void* xc, const void* bc, int64_t ldbc, int b_off, const float* dt_pre, const float* dt_bias, const float* A,
                    const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
-                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, cudaStream_t s);
+                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, bool one_row, cudaStream_t s);
 
 }  // namespace b200

@@ -216,11 +216,65 @@ __device__ __forceinline__ bool chunk_item(const int32_t* __restrict__ seq_start
   return true;
 }
 
-// rows row0 .. row0 + n - 1 of q or k (col: first column of the head) turned, times mul[row] -> hi and lo tiles [64][dim + 8]
+// eight fp32 values as eight bf16 hi and eight bf16 lo
+__device__ __forceinline__ void split8(const float (&v)[8], __nv_bfloat16* hi, __nv_bfloat16* lo) {
+  uint32_t h[4], l[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) split2(v[2 * i], v[2 * i + 1], h[i], l[i]);
+  *reinterpret_cast<uint4*>(hi) = make_uint4(h[0], h[1], h[2], h[3]);
+  *reinterpret_cast<uint4*>(lo) = make_uint4(l[0], l[1], l[2], l[3]);
+}
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+  v[0] = bf16lo(u.x), v[1] = bf16hi(u.x), v[2] = bf16lo(u.y), v[3] = bf16hi(u.y);
+  v[4] = bf16lo(u.z), v[5] = bf16hi(u.z), v[6] = bf16lo(u.w), v[7] = bf16hi(u.w);
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+
+// rows row0 .. row0 + n - 1 of q or k (col: first column of the head) turned, times mul (and falling: times pw[n - 1 - row]) -> hi and lo
+// tiles [64][dim + 8].  rot.half a multiple of 8: eight neighbouring entries and their partners at a time; else two.
 __device__ __forceinline__ void stage_rotated(const __nv_bfloat16* __restrict__ fused, int64_t ld, int64_t col, const RetRot& rot,
                                               const int32_t* __restrict__ positions, int row0, int n, int dim, float mul, const float* pw, bool falling,
                                               __nv_bfloat16* hi, __nv_bfloat16* lo) {
-  const int ks = dim + 8, hp = rot.half / 2, per = hp + (dim - 2 * rot.half) / 2;   // two neighbouring entries (and their partners) at a time
+  const int ks = dim + 8;
+  if (rot.half % 8 == 0) {
+    const int hp = rot.half / 8, per = hp + (dim - 2 * rot.half) / 8;
+#pragma unroll 2
+    for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
+      const int r = e / per, p = e - r * per;
+      const bool live = r < n;
+      const __nv_bfloat16* src = fused + (int64_t)(row0 + (live ? r : 0)) * ld + col;
+      const float m = live ? mul * (falling ? pw[n - 1 - r] : 1.0f) : 0.f;
+      if (p < hp) {
+        const int i = 8 * p;
+        const float* cs = rot_row(rot, positions[row0 + (live ? r : 0)]);
+        const uint4 ua = *reinterpret_cast<const uint4*>(src + i), ub = *reinterpret_cast<const uint4*>(src + i + rot.half);
+        float c[8], sn[8], a[8], b[8], x[8], y[8];
+        load8(cs + i, c);
+        load8(cs + rot.half + i, sn);
+        unpack8(ua, a);
+        unpack8(ub, b);
+#pragma unroll
+        for (int v = 0; v < 8; ++v) {
+          x[v] = fmaf(a[v], c[v], -b[v] * sn[v]) * m;
+          y[v] = fmaf(b[v], c[v], a[v] * sn[v]) * m;
+        }
+        split8(x, hi + r * ks + i, lo + r * ks + i);
+        split8(y, hi + r * ks + i + rot.half, lo + r * ks + i + rot.half);
+      } else {
+        const int i = 2 * rot.half + 8 * (p - hp);
+        float a[8];
+        unpack8(*reinterpret_cast<const uint4*>(src + i), a);
+#pragma unroll
+        for (int v = 0; v < 8; ++v) a[v] *= m;
+        split8(a, hi + r * ks + i, lo + r * ks + i);
+      }
+    }
+    return;
+  }
+  const int hp = rot.half / 2, per = hp + (dim - 2 * rot.half) / 2;
   for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
     const int r = e / per, p = e - r * per;
     const bool live = r < n;
@@ -249,13 +303,19 @@ __device__ __forceinline__ void stage_rotated(const __nv_bfloat16* __restrict__ 
   }
 }
 
-// value rows [64][vd + 8], zero past n
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src));
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// value rows [64][vd + 8], zero past n (asynchronously: cp_async_wait_all before the barrier that opens the tile)
 __device__ __forceinline__ void stage_values(const __nv_bfloat16* __restrict__ fused, int64_t ld, int64_t col, int row0, int n, int vd, __nv_bfloat16* vs) {
-  const int per = vd / 2;
+  const int per = vd / 8;
   for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
     const int r = e / per, p = e - r * per;
-    *reinterpret_cast<uint32_t*>(vs + r * (vd + 8) + 2 * p) =
-        r < n ? *reinterpret_cast<const uint32_t*>(fused + (int64_t)(row0 + r) * ld + col + 2 * p) : 0u;
+    __nv_bfloat16* dst = vs + r * (vd + 8) + 8 * p;
+    if (r < n) cp_async16(dst, fused + (int64_t)(row0 + r) * ld + col + 8 * p);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
   }
 }
 
@@ -277,8 +337,9 @@ retention_chunk_state_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld
   __nv_bfloat16* Vs = Kl + kRc * ks;                             // [64][vs]
   fill_powers(pw, decay[h]);
   __syncthreads();
-  stage_rotated(fused, ld, (int64_t)(heads + h) * dim, rot, positions, row0, n, dim, 1.0f / sqrtf((float)dim), pw, true, Kh, Kl);
   stage_values(fused, ld, (int64_t)2 * heads * dim + (int64_t)h * vd, row0, n, vd, Vs);
+  stage_rotated(fused, ld, (int64_t)(heads + h) * dim, rot, positions, row0, n, dim, 1.0f / sqrtf((float)dim), pw, true, Kh, Kl);
+  cp_async_wait_all();
   __syncthreads();
   float* U = ws + ((int64_t)item * heads + h) * vd * dim;
   // a warp takes a strip of 16 value columns x 64 key channels
@@ -324,11 +385,17 @@ retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __re
                             int heads, int elems) {
   pdl_wait();
   pdl_launch_dependents();
-  const int s = blockIdx.x, h = blockIdx.y, e = (blockIdx.z * 128 + threadIdx.x) * 4;
+  const int s = blockIdx.x, h = blockIdx.y, e = (blockIdx.z * 128 + threadIdx.x) * 8;
   const int start = seq_start[s], rows = seq_start[s + 1] - start;
   if (rows <= min_rows || e >= elems) return;
   float* st = state + (int64_t)seq_slots[s] * slot_stride + (int64_t)h * elems + e;
-  float4 S = positions[start] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
+  float S[8];
+  if (positions[start] == 0) {
+#pragma unroll
+    for (int v = 0; v < 8; ++v) S[v] = 0.f;
+  } else {
+    load8(st, S);
+  }
   const int chunks = (rows + kRc - 1) / kRc;
   float* U = ws + ((int64_t)(start / kRc + s) * heads + h) * elems + e;
   const int64_t stride = (int64_t)heads * elems;
@@ -338,10 +405,10 @@ retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __re
   const float gf = (float)full;
   constexpr int kAhead = 4;   // chunk loads in flight
   for (int c0 = 0; c0 < chunks; c0 += kAhead) {
-    float4 u[kAhead];
+    float u[kAhead][8];
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
-      if (c0 + i < chunks) u[i] = *reinterpret_cast<const float4*>(U + (c0 + i) * stride);
+      if (c0 + i < chunks) load8(U + (c0 + i) * stride, u[i]);
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
       const int c = c0 + i;
@@ -354,14 +421,14 @@ retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __re
           if (x & 1) r *= b;
         g = (float)r;
       }
-      uint32_t h0, l0, h1, l1;
-      split2(S.x, S.y, h0, l0);
-      split2(S.z, S.w, h1, l1);
-      *reinterpret_cast<uint4*>(U + c * stride) = make_uint4(h0, h1, l0, l1);   // 4 x hi, then 4 x lo
-      S = make_float4(fmaf(g, S.x, u[i].x), fmaf(g, S.y, u[i].y), fmaf(g, S.z, u[i].z), fmaf(g, S.w, u[i].w));
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(U + c * stride);
+      split8(S, dst, dst + 8);   // 8 x hi, then 8 x lo
+#pragma unroll
+      for (int v = 0; v < 8; ++v) S[v] = fmaf(g, S[v], u[i][v]);
     }
   }
-  *reinterpret_cast<float4*>(st) = S;
+  *reinterpret_cast<float4*>(st) = make_float4(S[0], S[1], S[2], S[3]);
+  *reinterpret_cast<float4*>(st + 4) = make_float4(S[4], S[5], S[6], S[7]);
 }
 
 // 3. outputs of a chunk.  Warp w: rows 16 (w & 3) .., half w >> 2 of the keys (scores) and of the value columns (outputs).
@@ -388,16 +455,16 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
   __nv_bfloat16* Ph = Sl + vd * ks;                              // [64][ps]
   __nv_bfloat16* Pl = Ph + kRc * ps;
   fill_powers(pw, decay[h]);
-  const float* U = ws + ((int64_t)item * heads + h) * vd * dim;
-  for (int e = threadIdx.x; e < vd * dim / 4; e += kRcThreads) {
-    const uint4 v = *reinterpret_cast<const uint4*>(U + (int64_t)e * 4);
-    const int j = e * 4 / dim, d = e * 4 - j * dim;
-    *reinterpret_cast<uint2*>(Sh + j * ks + d) = make_uint2(v.x, v.y);
-    *reinterpret_cast<uint2*>(Sl + j * ks + d) = make_uint2(v.z, v.w);
+  const __nv_bfloat16* U = reinterpret_cast<const __nv_bfloat16*>(ws + ((int64_t)item * heads + h) * vd * dim);
+  const int per_s = dim / 8;
+  for (int e = threadIdx.x; e < vd * per_s; e += kRcThreads) {
+    const int j = e / per_s, d = (e - j * per_s) * 8;
+    cp_async16(Sh + j * ks + d, U + (int64_t)e * 16);
+    cp_async16(Sl + j * ks + d, U + (int64_t)e * 16 + 8);
   }
+  stage_values(fused, ld, (int64_t)2 * heads * dim + (int64_t)h * vd, row0, n, vd, Vs);
   stage_rotated(fused, ld, (int64_t)h * dim, rot, positions, row0, n, dim, 1.0f, pw, false, Qh, Ql);
   stage_rotated(fused, ld, (int64_t)(heads + h) * dim, rot, positions, row0, n, dim, 1.0f / sqrtf((float)dim), pw, false, Kh, Kl);
-  stage_values(fused, ld, (int64_t)2 * heads * dim + (int64_t)h * vd, row0, n, vd, Vs);
   __syncthreads();
   const int r0 = (warp & 3) * 16, half = warp >> 2;
   const int rl = r0 + (lane >> 2);   // this lane's rows: rl and rl + 8
@@ -444,6 +511,8 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
       }
     }
   }
+  cp_async_wait_all();
+  __syncthreads();   // both halves' scores, the values and the state are in place
   // the state's part: 16 rows x this half's value columns (up to 64)
   const int cols = vd / 2, j0 = half * cols;   // multiple of 8
   float o[8][4];
@@ -476,7 +545,6 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
 #pragma unroll
     for (int i = 0; i < 8; ++i) o[i][0] *= d0, o[i][1] *= d0, o[i][2] *= d1, o[i][3] *= d1;
   }
-  __syncthreads();   // both halves' scores are in place
   for (int k0 = 0; k0 <= r0; k0 += 16) {   // keys past the warp's rows carry zero weight
     uint32_t ah[4], al[4];
     ldsm_x4(ah, Ph + (r0 + (lane & 15)) * ps + k0 + (lane >> 4) * 8);
@@ -587,7 +655,7 @@ int retention_chunk(const void* fused, int64_t ld, const float* rot, int rot_dim
   if (T == 0 || S == 0) return B200_OK;
   B200_REQUIRE(retention_chunk_supported(dim, vdim), B200_ERR_UNSUPPORTED, "retention_chunk: heads of %d x %d", dim, vdim);
   B200_REQUIRE(!rot || (half_layout && rot_dims % 4 == 0 && rot_dims <= dim), B200_ERR_UNSUPPORTED, "retention_chunk: %d rotated dimensions", rot_dims);
-  B200_REQUIRE(ws && ld % 2 == 0 && reinterpret_cast<uintptr_t>(fused) % 4 == 0 && reinterpret_cast<uintptr_t>(state) % 16 == 0 && slot_stride % 4 == 0,
+  B200_REQUIRE(ws && ld % 8 == 0 && reinterpret_cast<uintptr_t>(fused) % 16 == 0 && (!rot || reinterpret_cast<uintptr_t>(rot) % 16 == 0) && reinterpret_cast<uintptr_t>(state) % 16 == 0 && slot_stride % 4 == 0,
                B200_ERR_INVALID, "retention_chunk: misaligned operands or no workspace");
   const RetRot rr = {rot, rot ? rot_dims / 2 : 0, 1, max_pos};
   const __nv_bfloat16* f = (const __nv_bfloat16*)fused;
@@ -599,7 +667,7 @@ int retention_chunk(const void* fused, int64_t ld, const float* rot, int rot_dim
   B200_CUDA(launch(retention_chunk_state_kernel, dim3(items, heads), dim3(kRcThreads), sm1, s, f, ld, rr, decay, positions, seq_start, S, min_rows,
                    (float*)ws, heads, dim, vdim));
   const int elems = dim * vdim;
-  B200_CUDA(launch(retention_chunk_scan_kernel, dim3(S, heads, (elems / 4 + 127) / 128), dim3(128), (size_t)0, s, decay, positions, seq_start, seq_slots,
+  B200_CUDA(launch(retention_chunk_scan_kernel, dim3(S, heads, (elems / 8 + 127) / 128), dim3(128), (size_t)0, s, decay, positions, seq_start, seq_slots,
                    min_rows, (float*)ws, state, slot_stride, heads, elems));
   B200_CUDA(launch(retention_chunk_out_kernel, dim3(items, heads), dim3(kRcThreads), sm3, s, f, ld, rr, decay, positions, seq_start, S, min_rows,
                    (const float*)ws, (__nv_bfloat16*)out, heads, dim, vdim, eps));

@@ -9,7 +9,7 @@
 //  * selective_scan: per channel c and state n   S = exp(dt_c A[c][n]) S + dt_c x_c B_n;   y_c = sum_n S[c][n] C_n + D_c x_c;
 //    out_c = y_c silu(z_c), dt = softplus(dt_pre + bias).  Channels and states do not interact except through the sum over n, so a
 //    channel is walked by L neighbouring lanes with NS states each in registers; a CTA of 128 threads takes 128 / L channels of one
-//    sequence and stages 16 rows at a time in shared memory, the next 16 travelling into registers meanwhile.  Only one multiply-add per state is on
+//    sequence and stages 16 or 32 rows at a time in shared memory, the next ones travelling into registers meanwhile.  Only one multiply-add per state is on
 //    the chain from a row to the next; the exponentials depend on dt alone.  The state, fp32 [inner][n_state] in the sequence's slot,
 //    is read ahead of the dependency wait: no launch of the same step before this one writes it.
 //    A sequence whose first row of the step is at position 0 starts from zeros, whatever the slot held.
@@ -201,7 +201,39 @@ int conv_inputs_t(ConvArgs<AT> a, cudaStream_t s) {
 }
 
 // ---- the scan ----------------------------------------------------------------------------------------------------------------
-constexpr int kSelThreads = 128, kSelStage = 16;
+constexpr int kSelThreads = 128;
+
+__device__ __forceinline__ float ldf(float v) { return v; }
+__device__ __forceinline__ float ldf(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// exp(x log 2) of the decays: the 32-bit mode takes the library's exp2f, the serving mode the hardware's approximation of it (two
+// units in the last place, in fp32 as well)
+template <typename AT> __device__ __forceinline__ float decay_exp2(float x);
+template <> __device__ __forceinline__ float decay_exp2<float>(float x) { return exp2f(x); }
+template <> __device__ __forceinline__ float decay_exp2<__nv_bfloat16>(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// four rows' partial sums over L neighbouring lanes -> the row totals; lane l of a group holds row l & 3 (L >= 4) or all four (L < 4)
+template <int L>
+__device__ __forceinline__ void group_sums(float (&y)[4], int lane) {
+  if constexpr (L >= 4) {   // transposing: three exchanges for four sums, then plain rounds over the groups of four
+    const bool o1 = lane & 1, o2 = lane & 2;
+    const float a = __shfl_xor_sync(0xffffffffu, o1 ? y[0] : y[1], 1), b = __shfl_xor_sync(0xffffffffu, o1 ? y[2] : y[3], 1);
+    const float p = (o1 ? y[1] : y[0]) + a, q = (o1 ? y[3] : y[2]) + b;   // rows (lane & 1) and 2 + (lane & 1)
+    float r = (o2 ? q : p) + __shfl_xor_sync(0xffffffffu, o2 ? p : q, 2);
+#pragma unroll
+    for (int o = 4; o < L; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+    y[0] = r;
+  } else {
+#pragma unroll
+    for (int o = 1; o < L; o <<= 1)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] += __shfl_xor_sync(0xffffffffu, y[i], o);
+  }
+}
 
 template <typename AT>
 struct SelArgs {
@@ -215,9 +247,11 @@ struct SelArgs {
   int inner, n_state;
 };
 
-template <typename AT, int L, int NS>
+// ONE: every sequence of the step brings one row (decode)
+template <typename AT, int L, int NS, bool ONE>
 __global__ void __launch_bounds__(kSelThreads)
 selective_scan_kernel(const SelArgs<AT> a) {
+  constexpr int kSelStage = ONE ? 4 : (L >= 2 && L * NS <= 32 ? 32 : 16);                                // rows staged at a time
   constexpr int CH = kSelThreads / L, NP = L * NS;                                       // channels of the CTA, padded states
   constexpr int EX = (kSelStage * CH + kSelThreads - 1) / kSelThreads;                    // staged elements per thread: channel rows ..
   constexpr int EB = (kSelStage * NP + kSelThreads - 1) / kSelThreads;                    // .. B and C rows
@@ -240,92 +274,107 @@ selective_scan_kernel(const SelArgs<AT> a) {
 #pragma unroll
   for (int i = 0; i < NS; ++i) {
     const bool live = c < inner && n0 + i < N;
-    A[i] = live ? a.A[(int64_t)c * N + n0 + i] : 0.f;
+    A[i] = live ? a.A[(int64_t)c * N + n0 + i] * 1.4426950408889634f : 0.f;   // log2(e): decays are powers of two
     S[i] = live && !fresh ? st[n0 + i] : 0.f;
   }
   pdl_wait();
   pdl_launch_dependents();
-  float rx[EX], rdt[EX], rz[EX], rB[EB], rC[EB];
+  // A thread stages one channel of rows r0, r0 + L, ...  What is not there is read at a clamped address and dropped when it is
+  // staged: no branch and no conversion stands between the loads, so that all of them are in flight together.
+  const int xc_ch = tid % CH, r0 = tid / CH, ccx = min(c0 + xc_ch, inner - 1);
+  const bool live_x = c0 + xc_ch < inner;
+  const float dtb = a.dt_bias[ccx], skip = a.D[ccx];
+  AT rx[EX], rz[EX], rB[EB], rC[EB];
+  float rdt[EX];
   auto fetch = [&](int b0) {
-    const int nb = min(kSelStage, n_rows - b0);
+    const int last = min(kSelStage, n_rows - b0) - 1;
+    const int64_t row = start + b0;
 #pragma unroll
     for (int i = 0; i < EX; ++i) {
-      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
-      const bool live = r < nb && cc < inner;
-      const int64_t o = (int64_t)(start + b0 + (live ? r : 0)) * inner + (live ? cc : 0);
-      float x1[1] = {0.f};
-      if (live) ldv<AT, 1>(a.xc, o, x1);
-      rx[i] = x1[0];
-      rdt[i] = live ? a.dt_pre[o] + a.dt_bias[cc] : 0.f;
+      const int64_t t = row + min(r0 + L * i, last);
+      rx[i] = a.xc[t * inner + ccx];
+      rdt[i] = a.dt_pre[t * inner + ccx];
+      rz[i] = a.z[t * a.ldz + ccx];
     }
 #pragma unroll
     for (int i = 0; i < EB; ++i) {
-      const int e = tid + kSelThreads * i, r = e / NP, n = e % NP;
-      float b1[1] = {0.f}, c1[1] = {0.f};
-      if (r < nb && n < N) {
-        const int64_t o = (int64_t)(start + b0 + r) * a.ldbc + a.b_off + n;
-        ldv<AT, 1>(a.bc, o, b1);
-        ldv<AT, 1>(a.bc, o + N, c1);
-      }
-      rB[i] = b1[0];
-      rC[i] = c1[0];
+      const int e = tid + kSelThreads * i;
+      const AT* p = a.bc + (row + min(e / NP, last)) * a.ldbc + a.b_off + min(e % NP, N - 1);
+      rB[i] = p[0];
+      rC[i] = p[N];
     }
   };
   fetch(0);
   for (int b0 = 0; b0 < n_rows; b0 += kSelStage) {
     const int nb = min(kSelStage, n_rows - b0);
-    float xk[EX];   // this stage's x, for the skip term
+    float xk[EX];   // this stage's x and gates, for the outputs
+    AT zk[EX];
 #pragma unroll
     for (int i = 0; i < EX; ++i) {
-      const int e = tid + kSelThreads * i;
-      xk[i] = rx[i];
-      if (EX * kSelThreads == kSelStage * CH || e < kSelStage * CH) {
-        const float dt = softplus_f(rdt[i]);
-        sd[e / CH][e % CH] = make_float2(dt, dt * rx[i]);
+      const int r = r0 + L * i;
+      const float x = ldf(rx[i]);
+      xk[i] = x;
+      zk[i] = rz[i];
+      if (EX * kSelThreads == kSelStage * CH || r < kSelStage) {
+        const float dt = r < nb && live_x ? softplus_f(rdt[i] + dtb) : 0.f;
+        sd[r][xc_ch] = make_float2(dt, dt * x);
       }
     }
 #pragma unroll
     for (int i = 0; i < EB; ++i) {
       const int e = tid + kSelThreads * i;
       if (EB * kSelThreads == kSelStage * NP || e < kSelStage * NP) {
-        sB[e / NP][e % NP] = rB[i];
-        sC[e / NP][e % NP] = rC[i];
+        const bool live = e / NP < nb && e % NP < N;
+        sB[e / NP][e % NP] = live ? ldf(rB[i]) : 0.f;
+        sC[e / NP][e % NP] = live ? ldf(rC[i]) : 0.f;
       }
-    }
-#pragma unroll
-    for (int i = 0; i < EX; ++i) {   // this stage's gates arrive during the walk
-      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
-      float z1[1] = {0.f};
-      if (r < nb && cc < inner) ldv<AT, 1>(a.z, (int64_t)(start + b0 + r) * a.ldz + cc, z1);
-      rz[i] = z1[0];
     }
     __syncthreads();
     if (b0 + kSelStage < n_rows) fetch(b0 + kSelStage);
-    auto step = [&](int r) {
-      const float2 d = sd[r][ch];
-      float y = 0.f;
+    // four rows at a time: everything but the state's own chain is independent of the rows before (rows past nb have dt = 0 and
+    // leave the state as it is)
+    for (int r = 0; r < nb; r += 4) {
+      float2 d[4];
+      float dec[4][NS], u[4][NS], y[4];
 #pragma unroll
-      for (int i = 0; i < NS; ++i) {
-        S[i] = fmaf(expf(d.x * A[i]), S[i], d.y * sB[r][n0 + i]);
-        y = fmaf(S[i], sC[r][n0 + i], y);
+      for (int k = 0; k < 4; ++k) d[k] = sd[r + k][ch];
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int i = 0; i < NS; i += 4) {
+          const float4 b = *reinterpret_cast<const float4*>(&sB[r + k][n0 + i]);
+          u[k][i] = d[k].y * b.x, u[k][i + 1] = d[k].y * b.y, u[k][i + 2] = d[k].y * b.z, u[k][i + 3] = d[k].y * b.w;
+#pragma unroll
+          for (int x = 0; x < 4; ++x) dec[k][i + x] = decay_exp2<AT>(d[k].x * A[i + x]);
+        }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        y[k] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NS; i += 4) {
+          const float4 q = *reinterpret_cast<const float4*>(&sC[r + k][n0 + i]);
+          S[i] = fmaf(dec[k][i], S[i], u[k][i]), S[i + 1] = fmaf(dec[k][i + 1], S[i + 1], u[k][i + 1]);
+          S[i + 2] = fmaf(dec[k][i + 2], S[i + 2], u[k][i + 2]), S[i + 3] = fmaf(dec[k][i + 3], S[i + 3], u[k][i + 3]);
+          y[k] = fmaf(S[i], q.x, y[k]), y[k] = fmaf(S[i + 1], q.y, y[k]), y[k] = fmaf(S[i + 2], q.z, y[k]), y[k] = fmaf(S[i + 3], q.w, y[k]);
+        }
       }
+      group_sums<L>(y, tid);
+      if constexpr (L >= 4) {
+        if (tid % L < 4) sy[r + tid % L][ch] = y[0];
+      } else {
+        if (tid % L == 0) {
 #pragma unroll
-      for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (tid % L == 0) sy[r][ch] = y;
-    };
-    if (nb == kSelStage) {
-#pragma unroll 4
-      for (int r = 0; r < kSelStage; ++r) step(r);
-    } else {
-      for (int r = 0; r < nb; ++r) step(r);
+          for (int k = 0; k < 4; ++k) sy[r + k][ch] = y[k];
+        }
+      }
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < EX; ++i) {
-      const int e = tid + kSelThreads * i, r = e / CH, cc = c0 + e % CH;
-      if (r < nb && cc < inner) {
-        float o1[1] = {fmaf(a.D[cc], xk[i], sy[r][e % CH]) * silu_f(rz[i])};
-        stv<AT, 1>(a.out, (int64_t)(start + b0 + r) * inner + cc, o1);
+      const int r = r0 + L * i;
+      if (r < nb && live_x) {
+        float o1[1] = {fmaf(skip, xk[i], sy[r][xc_ch]) * silu_f(ldf(zk[i]))};
+        stv<AT, 1>(a.out, (int64_t)(start + b0 + r) * inner + ccx, o1);
       }
     }
   }
@@ -335,9 +384,14 @@ selective_scan_kernel(const SelArgs<AT> a) {
 }
 
 template <typename AT>
-int selective_scan_t(const SelArgs<AT>& a, int S, cudaStream_t s) {
+int selective_scan_t(const SelArgs<AT>& a, int S, bool one, cudaStream_t s) {
   const int N = a.n_state;
-#define SEL(LV, NV) B200_CUDA(launch(selective_scan_kernel<AT, LV, NV>, dim3(S, (a.inner + kSelThreads / LV - 1) / (kSelThreads / LV)), dim3(kSelThreads), (size_t)0, s, a))
+#define SEL(LV, NV)                                                                                                                              \
+  do {                                                                                                                                           \
+    const dim3 grid(S, (a.inner + kSelThreads / LV - 1) / (kSelThreads / LV));                                                                    \
+    if (one) B200_CUDA(launch(selective_scan_kernel<AT, LV, NV, true>, grid, dim3(kSelThreads), (size_t)0, s, a));                                \
+    else B200_CUDA(launch(selective_scan_kernel<AT, LV, NV, false>, grid, dim3(kSelThreads), (size_t)0, s, a));                                   \
+  } while (0)
   if (N <= 4) SEL(1, 4);
   else if (N <= 8) SEL(2, 4);
   else if (N <= 16) SEL(4, 4);
@@ -378,17 +432,17 @@ int selective_rows(int rank, int state) { return (selective_dt_pad(rank) + 2 * s
 
 int selective_scan(bool f32, const void* xc, const void* bc, int64_t ldbc, int b_off, const float* dt_pre, const float* dt_bias, const float* A,
                    const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
-                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, cudaStream_t s) {
+                   float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, bool one_row, cudaStream_t s) {
   if (S == 0) return B200_OK;
   B200_REQUIRE(inner > 0 && n_state > 0 && n_state <= 256, B200_ERR_UNSUPPORTED, "selective_scan: %d channels, %d states (at most 256)", inner, n_state);
   if (f32) {
     SelArgs<float> a = {(const float*)xc, (const float*)bc, (const float*)z, ldbc, ldz, slot_stride, b_off, dt_pre, dt_bias, A, D, positions, seq_start,
                         seq_slots, state, (float*)out, inner, n_state};
-    return selective_scan_t<float>(a, S, s);
+    return selective_scan_t<float>(a, S, one_row, s);
   }
   SelArgs<__nv_bfloat16> a = {(const __nv_bfloat16*)xc, (const __nv_bfloat16*)bc, (const __nv_bfloat16*)z, ldbc, ldz, slot_stride, b_off, dt_pre, dt_bias, A,
                               D, positions, seq_start, seq_slots, state, (__nv_bfloat16*)out, inner, n_state};
-  return selective_scan_t<__nv_bfloat16>(a, S, s);
+  return selective_scan_t<__nv_bfloat16>(a, S, one_row, s);
 }
 
 }  // namespace b200

@@ -901,7 +901,7 @@ static int stack_enqueue_step_looped(b200_ctx* c, const StepArgs& a, cudaStream_
         STEP(linear(M->xp, rows, W.side_dt, nullptr, M->dtp, inner, pad, -1, true));
         STEP(selective_scan(f32, M->xc, M->xp, rows, pad, M->dtp, W.side_dt_b, W.side_a, W.side_skip,
                             static_cast<const char*>(M->qkv) + (int64_t)(ch + inner) * es, qr, a.positions, M->seq_start, seq_slots,
-                            M->state + W.rec_off, M->slot_floats, M->ssy, S, inner, L.side_state, s));
+                            M->state + W.rec_off, M->slot_floats, M->ssy, S, inner, L.side_state, one_row_each, s));
         STEP(linear(M->ssy, inner, W.side_o, nullptr, M->y2, Wd, inner, -1, false));
         y_side = M->y2;
       }
@@ -2156,11 +2156,11 @@ extern "C" int32_t b200_selective_rows(int32_t rank, int32_t state) { return sel
 extern "C" int b200_selective_scan(int32_t f32, const void* xc, const void* bc, int64_t ldbc, int32_t b_off, const float* dt_pre, const float* dt_bias,
                                    const float* A, const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start,
                                    const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t S, int32_t inner, int32_t n_state,
-                                   void* stream) {
+                                   int32_t one_row, void* stream) {
   B200_REQUIRE(xc && bc && dt_pre && dt_bias && A && D && z && positions && seq_start && seq_slots && state && out, B200_ERR_INVALID,
                "selective_scan: null argument");
   return selective_scan(f32 != 0, xc, bc, ldbc, b_off, dt_pre, dt_bias, A, D, z, ldz, positions, seq_start, seq_slots, state, slot_stride, out, S, inner,
-                        n_state, (cudaStream_t)stream);
+                        n_state, one_row != 0, (cudaStream_t)stream);
 }
 
 extern "C" int b200_paged_attn_biased(int32_t f32, int32_t form, const float* q, const void* kc, const void* vc, const int32_t* block_table,

@@ -895,11 +895,12 @@ B200_API int b200_conv_inputs(int32_t f32, const void* fused, int64_t ld, const 
 /* Rows of W_x's product: dt (padded to a multiple of 8) | B | C, the total padded to a multiple of 8. */
 B200_API int32_t b200_selective_rows(int32_t rank, int32_t state);
 /* Selective scan: xc, z, out [T][inner] (activation type, z of leading dimension ldz), bc rows of leading dimension ldbc with B at b_off and C
- * at b_off + n_state, dt_pre fp32 [T][inner] ahead of bias and softplus; state [slot][inner][n_state] fp32. */
+ * at b_off + n_state, dt_pre fp32 [T][inner] ahead of bias and softplus; state [slot][inner][n_state] fp32.  one_row: every sequence
+ * of the step brings one row. */
 B200_API int b200_selective_scan(int32_t f32, const void* xc, const void* bc, int64_t ldbc, int32_t b_off, const float* dt_pre, const float* dt_bias,
                                  const float* A, const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start,
                                  const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t n_seqs, int32_t inner,
-                                 int32_t n_state, void* stream);
+                                 int32_t n_state, int32_t one_row, void* stream);
 /* Paged attention with a score cap and a distance bias: s = softcap tanh(scale q.k / softcap) + dist_bias[h][min(i - j, bias_dist - 1)]
  * (softcap 0 / dist_bias NULL: off), optional window, per-head gate (gate[t * ldg + h], activation type, sigmoid; NULL: none).  form 0: one
  * CTA per row and head, 1: runs of rows share K/V tiles, 2: tensor cores (bf16; n_splits, part as b200_paged_attn_mma). */

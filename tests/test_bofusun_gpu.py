@@ -340,7 +340,7 @@ def test_selective_scan_in_portions_with_three_sequences_and_dirty_slots(f32, in
     st = dev(torch.full((5, slot_f), -3.0))
     slots, got = {"a": 4, "b": 1, "c": 0}, {k: torch.zeros(n, inner) for k, n in lens.items()}
     ldbc, off = 2 * state + 11, 7
-    sizes = {"a": [1, 2, 16, 1, 17, 33], "b": [32, 1], "c": [1] * 5}
+    sizes = {"a": [1, 2, 16, 1, 17, 33], "b": [32, 1], "c": [1] * 5}      # the last step of c and its like bring one row each
     Ad, Dd, dtbd = dev(A), dev(D), dev(dtb)
     for step in _steps(lens, sizes, {"a": 0, "b": 1, "c": 2}):
         pos, _, start = _meta(step)
@@ -353,7 +353,7 @@ def test_selective_scan_in_portions_with_three_sequences_and_dirty_slots(f32, in
         out = torch.zeros(T, inner, dtype=adt, device=DEV)
         check(lib().b200_selective_scan(f32, dev(cat("x"), adt).data_ptr(), dev(bc, adt).data_ptr(), ldbc, off, dev(cat("dt")).data_ptr(), dtbd.data_ptr(),
                                         Ad.data_ptr(), Dd.data_ptr(), dev(zz, adt).data_ptr(), inner + 3, i32(pos).data_ptr(), i32(start).data_ptr(),
-                                        i32([slots[k] for k, _, _ in step]).data_ptr(), st.data_ptr(), slot_f, out.data_ptr(), S, inner, state, None))
+                                        i32([slots[k] for k, _, _ in step]).data_ptr(), st.data_ptr(), slot_f, out.data_ptr(), S, inner, state, int(T == S), None))
         sync()
         for si, (k, lo, n) in enumerate(step):
             got[k][lo:lo + n] = out[start[si]:start[si + 1]].float().cpu()
