@@ -242,7 +242,7 @@ __device__ __forceinline__ void stage_rotated(const __nv_bfloat16* __restrict__ 
   if (rot.half % 8 == 0) {
     const int hp = rot.half / 8, per = hp + (dim - 2 * rot.half) / 8;
 #pragma unroll 2
-    for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
+    for (int e = threadIdx.x; e < kRc * per; e += (int)blockDim.x) {
       const int r = e / per, p = e - r * per;
       const bool live = r < n;
       const __nv_bfloat16* src = fused + (int64_t)(row0 + (live ? r : 0)) * ld + col;
@@ -275,7 +275,7 @@ __device__ __forceinline__ void stage_rotated(const __nv_bfloat16* __restrict__ 
     return;
   }
   const int hp = rot.half / 2, per = hp + (dim - 2 * rot.half) / 2;
-  for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
+  for (int e = threadIdx.x; e < kRc * per; e += (int)blockDim.x) {
     const int r = e / per, p = e - r * per;
     const bool live = r < n;
     const __nv_bfloat16* src = fused + (int64_t)(row0 + (live ? r : 0)) * ld + col;
@@ -311,7 +311,7 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 // value rows [64][vd + 8], zero past n (asynchronously: cp_async_wait_all before the barrier that opens the tile)
 __device__ __forceinline__ void stage_values(const __nv_bfloat16* __restrict__ fused, int64_t ld, int64_t col, int row0, int n, int vd, __nv_bfloat16* vs) {
   const int per = vd / 8;
-  for (int e = threadIdx.x; e < kRc * per; e += kRcThreads) {
+  for (int e = threadIdx.x; e < kRc * per; e += (int)blockDim.x) {
     const int r = e / per, p = e - r * per;
     __nv_bfloat16* dst = vs + r * (vd + 8) + 8 * p;
     if (r < n) cp_async16(dst, fused + (int64_t)(row0 + r) * ld + col + 8 * p);
@@ -378,24 +378,19 @@ retention_chunk_state_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld
   }
 }
 
-// 2. elementwise over the state: U_c becomes the state ahead of chunk c as bf16 pairs (hi, lo) in place; the last state into the slot
+// 2. elementwise over the state: U_c becomes, in place, the state ahead of chunk c as bf16 (blocks of 8 hi, then their 8 lo); the last
+// state goes into the slot.  Two neighbouring threads share a block: both have read it before either writes.
 __global__ void __launch_bounds__(128)
 retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __restrict__ positions, const int32_t* __restrict__ seq_start,
                             const int32_t* __restrict__ seq_slots, int min_rows, float* __restrict__ ws, float* __restrict__ state, int64_t slot_stride,
                             int heads, int elems) {
   pdl_wait();
   pdl_launch_dependents();
-  const int s = blockIdx.x, h = blockIdx.y, e = (blockIdx.z * 128 + threadIdx.x) * 8;
+  const int s = blockIdx.x, h = blockIdx.y, e = (blockIdx.z * 128 + threadIdx.x) * 4;
   const int start = seq_start[s], rows = seq_start[s + 1] - start;
   if (rows <= min_rows || e >= elems) return;
   float* st = state + (int64_t)seq_slots[s] * slot_stride + (int64_t)h * elems + e;
-  float S[8];
-  if (positions[start] == 0) {
-#pragma unroll
-    for (int v = 0; v < 8; ++v) S[v] = 0.f;
-  } else {
-    load8(st, S);
-  }
+  float4 S = positions[start] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
   const int chunks = (rows + kRc - 1) / kRc;
   float* U = ws + ((int64_t)(start / kRc + s) * heads + h) * elems + e;
   const int64_t stride = (int64_t)heads * elems;
@@ -403,12 +398,13 @@ retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __re
 #pragma unroll
   for (int i = 0; i < 6; ++i) full *= full;   // decay^64
   const float gf = (float)full;
-  constexpr int kAhead = 4;   // chunk loads in flight
+  constexpr int kAhead = 8;   // chunk loads in flight
   for (int c0 = 0; c0 < chunks; c0 += kAhead) {
-    float u[kAhead][8];
+    float4 u[kAhead];
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
-      if (c0 + i < chunks) load8(U + (c0 + i) * stride, u[i]);
+      if (c0 + i < chunks) u[i] = *reinterpret_cast<const float4*>(U + (c0 + i) * stride);
+    __syncwarp();   // the blocks are shared with a neighbouring thread (whole warps are in range: elems is a multiple of 256)
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
       const int c = c0 + i;
@@ -421,24 +417,29 @@ retention_chunk_scan_kernel(const float* __restrict__ decay, const int32_t* __re
           if (x & 1) r *= b;
         g = (float)r;
       }
-      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(U + c * stride);
-      split8(S, dst, dst + 8);   // 8 x hi, then 8 x lo
-#pragma unroll
-      for (int v = 0; v < 8; ++v) S[v] = fmaf(g, S[v], u[i][v]);
+      uint32_t h0, l0, h1, l1;
+      split2(S.x, S.y, h0, l0);
+      split2(S.z, S.w, h1, l1);
+      // U points at element e: back to the block of 8, then this thread's half of its hi and of its lo
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(U - (e & 4) + c * stride) + (e & 4);
+      *reinterpret_cast<uint2*>(dst) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(dst + 8) = make_uint2(l0, l1);
+      S = make_float4(fmaf(g, S.x, u[i].x), fmaf(g, S.y, u[i].y), fmaf(g, S.z, u[i].z), fmaf(g, S.w, u[i].w));
     }
   }
-  *reinterpret_cast<float4*>(st) = make_float4(S[0], S[1], S[2], S[3]);
-  *reinterpret_cast<float4*>(st + 4) = make_float4(S[4], S[5], S[6], S[7]);
+  *reinterpret_cast<float4*>(st) = S;
 }
 
-// 3. outputs of a chunk.  Warp w: rows 16 (w & 3) .., half w >> 2 of the keys (scores) and of the value columns (outputs).
-__global__ void __launch_bounds__(kRcThreads)
+// 3. outputs of a chunk.  Warp w: rows 16 (w & 3) ..; quarter w >> 2 takes 16 of the 64 keys (scores) and every fourth group of 16 value
+// columns (outputs).
+constexpr int kRoThreads = 512;
+__global__ void __launch_bounds__(kRoThreads)
 retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, RetRot rot, const float* __restrict__ decay,
                            const int32_t* __restrict__ positions, const int32_t* __restrict__ seq_start, int n_seqs, int min_rows,
                            const float* __restrict__ ws, __nv_bfloat16* __restrict__ out, int heads, int dim, int vd, float eps) {
   extern __shared__ __align__(16) unsigned char smraw[];
   __shared__ float pw[kRc + 1];
-  __shared__ float ssq[2][kRc];
+  __shared__ float ssq[4][kRc];
   pdl_wait();
   pdl_launch_dependents();
   const int item = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -454,10 +455,9 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
   __nv_bfloat16* Sl = Sh + vd * ks;
   __nv_bfloat16* Ph = Sl + vd * ks;                              // [64][ps]
   __nv_bfloat16* Pl = Ph + kRc * ps;
-  fill_powers(pw, decay[h]);
   const __nv_bfloat16* U = reinterpret_cast<const __nv_bfloat16*>(ws + ((int64_t)item * heads + h) * vd * dim);
   const int per_s = dim / 8;
-  for (int e = threadIdx.x; e < vd * per_s; e += kRcThreads) {
+  for (int e = threadIdx.x; e < vd * per_s; e += kRoThreads) {
     const int j = e / per_s, d = (e - j * per_s) * 8;
     cp_async16(Sh + j * ks + d, U + (int64_t)e * 16);
     cp_async16(Sl + j * ks + d, U + (int64_t)e * 16 + 8);
@@ -465,108 +465,113 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
   stage_values(fused, ld, (int64_t)2 * heads * dim + (int64_t)h * vd, row0, n, vd, Vs);
   stage_rotated(fused, ld, (int64_t)h * dim, rot, positions, row0, n, dim, 1.0f, pw, false, Qh, Ql);
   stage_rotated(fused, ld, (int64_t)(heads + h) * dim, rot, positions, row0, n, dim, 1.0f / sqrtf((float)dim), pw, false, Kh, Kl);
+  fill_powers(pw, decay[h]);
   __syncthreads();
-  const int r0 = (warp & 3) * 16, half = warp >> 2;
+  const int r0 = (warp & 3) * 16, quarter = warp >> 2;
   const int rl = r0 + (lane >> 2);   // this lane's rows: rl and rl + 8
   const int qoff = (r0 + (lane & 15)) * ks + (lane >> 4) * 8;
   const int boff = (lane & 7) + (lane >> 4) * 8, bcol = ((lane >> 3) & 1) * 8;   // two 8-row groups of a B operand stored [n][k]
   {
-    // scores of 16 rows against keys 32 half .. + 31
-    float c[4][4];
+    // scores of 16 rows against keys 16 quarter .. + 15; the three split products have accumulators of their own
+    float c[3][2][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int x = 0; x < 3; ++x)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) c[i][j] = 0.f;
-    const int key0 = half * 32;
-    if (key0 <= r0 + 15) {
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) c[x][i][j] = 0.f;
+    const int key0 = quarter * 16;
+    if (key0 <= r0) {
+#pragma unroll 2
       for (int k0 = 0; k0 < dim; k0 += 16) {
-        uint32_t ah[4], al[4];
+        uint32_t ah[4], al[4], bh[4], bl[4];
         ldsm_x4(ah, Qh + qoff + k0);
+        ldsm_x4(bh, Kh + (key0 + boff) * ks + k0 + bcol);
         ldsm_x4(al, Ql + qoff + k0);
-#pragma unroll
-        for (int p = 0; p < 2; ++p) {
-          uint32_t bh[4], bl[4];
-          ldsm_x4(bh, Kh + (key0 + p * 16 + boff) * ks + k0 + bcol);
-          ldsm_x4(bl, Kl + (key0 + p * 16 + boff) * ks + k0 + bcol);
-          mma_bf16(c[2 * p], al, bh[0], bh[1]);
-          mma_bf16(c[2 * p], ah, bl[0], bl[1]);
-          mma_bf16(c[2 * p], ah, bh[0], bh[1]);
-          mma_bf16(c[2 * p + 1], al, bh[2], bh[3]);
-          mma_bf16(c[2 * p + 1], ah, bl[2], bl[3]);
-          mma_bf16(c[2 * p + 1], ah, bh[2], bh[3]);
-        }
+        ldsm_x4(bl, Kl + (key0 + boff) * ks + k0 + bcol);
+        mma_bf16(c[0][0], ah, bh[0], bh[1]);
+        mma_bf16(c[0][1], ah, bh[2], bh[3]);
+        mma_bf16(c[1][0], al, bh[0], bh[1]);
+        mma_bf16(c[1][1], al, bh[2], bh[3]);
+        mma_bf16(c[2][0], ah, bl[0], bl[1]);
+        mma_bf16(c[2][1], ah, bl[2], bl[3]);
       }
     }
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 2; ++i) {
       const int key = key0 + i * 8 + (lane & 3) * 2;
 #pragma unroll
       for (int hr = 0; hr < 2; ++hr) {
         const int r = rl + hr * 8;
-        const float p0 = key <= r ? c[i][2 * hr] * pw[r - key] : 0.f, p1 = key + 1 <= r ? c[i][2 * hr + 1] * pw[r - key - 1] : 0.f;
+        const float s0 = c[0][i][2 * hr] + (c[1][i][2 * hr] + c[2][i][2 * hr]);
+        const float s1 = c[0][i][2 * hr + 1] + (c[1][i][2 * hr + 1] + c[2][i][2 * hr + 1]);
         uint32_t h2, l2;
-        split2(p0, p1, h2, l2);
+        split2(key <= r ? s0 * pw[r - key] : 0.f, key + 1 <= r ? s1 * pw[r - key - 1] : 0.f, h2, l2);
         *reinterpret_cast<uint32_t*>(Ph + r * ps + key) = h2;
         *reinterpret_cast<uint32_t*>(Pl + r * ps + key) = l2;
       }
     }
   }
   cp_async_wait_all();
-  __syncthreads();   // both halves' scores, the values and the state are in place
-  // the state's part: 16 rows x this half's value columns (up to 64)
-  const int cols = vd / 2, j0 = half * cols;   // multiple of 8
-  float o[8][4];
+  __syncthreads();   // every quarter's scores, the values and the state are in place
+  // up to two groups of 16 value columns: the state's part first
+  float o[2][2][4];
 #pragma unroll
-  for (int i = 0; i < 8; ++i)
+  for (int u = 0; u < 2; ++u)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[u][i][j] = 0.f;
+  const int n_units = vd / 16;
+#pragma unroll 2
   for (int k0 = 0; k0 < dim; k0 += 16) {
     uint32_t ah[4], al[4];
     ldsm_x4(ah, Qh + qoff + k0);
     ldsm_x4(al, Ql + qoff + k0);
 #pragma unroll
-    for (int p = 0; p < 4; ++p)
-      if (p * 16 < cols) {
+    for (int u = 0; u < 2; ++u)
+      if (quarter + 4 * u < n_units) {
         uint32_t bh[4], bl[4];
-        // a half whose column count is an odd multiple of 8 reads 8 rows of the other half, whose products are not kept
-        const int jr = min(j0 + p * 16 + boff, vd - 1);
+        const int jr = (quarter + 4 * u) * 16 + boff;
         ldsm_x4(bh, Sh + jr * ks + k0 + bcol);
         ldsm_x4(bl, Sl + jr * ks + k0 + bcol);
-        mma_bf16(o[2 * p], al, bh[0], bh[1]);
-        mma_bf16(o[2 * p], ah, bl[0], bl[1]);
-        mma_bf16(o[2 * p], ah, bh[0], bh[1]);
-        mma_bf16(o[2 * p + 1], al, bh[2], bh[3]);
-        mma_bf16(o[2 * p + 1], ah, bl[2], bl[3]);
-        mma_bf16(o[2 * p + 1], ah, bh[2], bh[3]);
+        mma_bf16(o[u][0], al, bh[0], bh[1]);
+        mma_bf16(o[u][1], al, bh[2], bh[3]);
+        mma_bf16(o[u][0], ah, bl[0], bl[1]);
+        mma_bf16(o[u][1], ah, bl[2], bl[3]);
+        mma_bf16(o[u][0], ah, bh[0], bh[1]);
+        mma_bf16(o[u][1], ah, bh[2], bh[3]);
       }
   }
   {
     const float d0 = pw[rl + 1], d1 = pw[rl + 9];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) o[i][0] *= d0, o[i][1] *= d0, o[i][2] *= d1, o[i][3] *= d1;
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) o[u][i][0] *= d0, o[u][i][1] *= d0, o[u][i][2] *= d1, o[u][i][3] *= d1;
   }
   for (int k0 = 0; k0 <= r0; k0 += 16) {   // keys past the warp's rows carry zero weight
     uint32_t ah[4], al[4];
     ldsm_x4(ah, Ph + (r0 + (lane & 15)) * ps + k0 + (lane >> 4) * 8);
     ldsm_x4(al, Pl + (r0 + (lane & 15)) * ps + k0 + (lane >> 4) * 8);
 #pragma unroll
-    for (int p = 0; p < 4; ++p)
-      if (p * 16 < cols) {
+    for (int u = 0; u < 2; ++u)
+      if (quarter + 4 * u < n_units) {
         uint32_t b[4];
-        // columns past the half: inside the row's padding at most
-        ldsm_x4_t(b, Vs + (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + j0 + p * 16 + (lane >> 4) * 8);
-        mma_bf16(o[2 * p], al, b[0], b[1]);
-        mma_bf16(o[2 * p], ah, b[0], b[1]);
-        mma_bf16(o[2 * p + 1], al, b[2], b[3]);
-        mma_bf16(o[2 * p + 1], ah, b[2], b[3]);
+        ldsm_x4_t(b, Vs + (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + (quarter + 4 * u) * 16 + (lane >> 4) * 8);
+        mma_bf16(o[u][0], al, b[0], b[1]);
+        mma_bf16(o[u][1], al, b[2], b[3]);
+        mma_bf16(o[u][0], ah, b[0], b[1]);
+        mma_bf16(o[u][1], ah, b[2], b[3]);
       }
   }
   float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i)
-    if (i * 8 < cols) {
-      s0 = fmaf(o[i][0], o[i][0], fmaf(o[i][1], o[i][1], s0));
-      s1 = fmaf(o[i][2], o[i][2], fmaf(o[i][3], o[i][3], s1));
+  for (int u = 0; u < 2; ++u)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {   // a group that is not there holds zeros
+      s0 = fmaf(o[u][i][0], o[u][i][0], fmaf(o[u][i][1], o[u][i][1], s0));
+      s1 = fmaf(o[u][i][2], o[u][i][2], fmaf(o[u][i][3], o[u][i][3], s1));
     }
 #pragma unroll
   for (int x = 1; x < 4; x <<= 1) {
@@ -574,8 +579,8 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
     s1 += __shfl_xor_sync(0xffffffffu, s1, x);
   }
   if ((lane & 3) == 0) {
-    ssq[half][rl] = s0;
-    ssq[half][rl + 8] = s1;
+    ssq[quarter][rl] = s0;
+    ssq[quarter][rl + 8] = s1;
   }
   __syncthreads();
   const int64_t hv = (int64_t)heads * vd;
@@ -583,16 +588,20 @@ retention_chunk_out_kernel(const __nv_bfloat16* __restrict__ fused, int64_t ld, 
   for (int hr = 0; hr < 2; ++hr) {
     const int r = rl + hr * 8;
     if (r >= n) continue;
-    const float inv = 1.0f / sqrtf((ssq[0][r] + ssq[1][r]) / (float)vd + eps);
+    const float inv = 1.0f / sqrtf(((ssq[0][r] + ssq[1][r]) + (ssq[2][r] + ssq[3][r])) / (float)vd + eps);
     const __nv_bfloat16* gate = fused + (int64_t)(row0 + r) * ld + (int64_t)2 * heads * dim + hv + (int64_t)h * vd;
     __nv_bfloat16* dst = out + (int64_t)(row0 + r) * hv + (int64_t)h * vd;
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-      if (i * 8 < cols) {
-        const int j = j0 + i * 8 + (lane & 3) * 2;
-        const uint32_t z2 = *reinterpret_cast<const uint32_t*>(gate + j);
-        const float za = bf16lo(z2), zb = bf16hi(z2);
-        *reinterpret_cast<uint32_t*>(dst + j) = pack_bf16(o[i][2 * hr] * inv * (za / (1.0f + expf(-za))), o[i][2 * hr + 1] * inv * (zb / (1.0f + expf(-zb))));
+    for (int u = 0; u < 2; ++u)
+      if (quarter + 4 * u < n_units) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int j = (quarter + 4 * u) * 16 + i * 8 + (lane & 3) * 2;
+          const uint32_t z2 = *reinterpret_cast<const uint32_t*>(gate + j);
+          const float za = bf16lo(z2), zb = bf16hi(z2);
+          *reinterpret_cast<uint32_t*>(dst + j) =
+              pack_bf16(o[u][i][2 * hr] * inv * (za / (1.0f + expf(-za))), o[u][i][2 * hr + 1] * inv * (zb / (1.0f + expf(-zb))));
+        }
       }
   }
 }
@@ -667,9 +676,9 @@ int retention_chunk(const void* fused, int64_t ld, const float* rot, int rot_dim
   B200_CUDA(launch(retention_chunk_state_kernel, dim3(items, heads), dim3(kRcThreads), sm1, s, f, ld, rr, decay, positions, seq_start, S, min_rows,
                    (float*)ws, heads, dim, vdim));
   const int elems = dim * vdim;
-  B200_CUDA(launch(retention_chunk_scan_kernel, dim3(S, heads, (elems / 8 + 127) / 128), dim3(128), (size_t)0, s, decay, positions, seq_start, seq_slots,
+  B200_CUDA(launch(retention_chunk_scan_kernel, dim3(S, heads, (elems / 4 + 127) / 128), dim3(128), (size_t)0, s, decay, positions, seq_start, seq_slots,
                    min_rows, (float*)ws, state, slot_stride, heads, elems));
-  B200_CUDA(launch(retention_chunk_out_kernel, dim3(items, heads), dim3(kRcThreads), sm3, s, f, ld, rr, decay, positions, seq_start, S, min_rows,
+  B200_CUDA(launch(retention_chunk_out_kernel, dim3(items, heads), dim3(kRoThreads), sm3, s, f, ld, rr, decay, positions, seq_start, S, min_rows,
                    (const float*)ws, (__nv_bfloat16*)out, heads, dim, vdim, eps));
   return B200_OK;
 }

@@ -247,11 +247,10 @@ struct SelArgs {
   int inner, n_state;
 };
 
-// ONE: every sequence of the step brings one row (decode)
-template <typename AT, int L, int NS, bool ONE>
+template <typename AT, int L, int NS>
 __global__ void __launch_bounds__(kSelThreads)
 selective_scan_kernel(const SelArgs<AT> a) {
-  constexpr int kSelStage = ONE ? 4 : (L >= 2 && L * NS <= 32 ? 32 : 16);                                // rows staged at a time
+  constexpr int kSelStage = L >= 2 && L * NS <= 32 ? 32 : 16;                                            // rows staged at a time
   constexpr int CH = kSelThreads / L, NP = L * NS;                                       // channels of the CTA, padded states
   constexpr int EX = (kSelStage * CH + kSelThreads - 1) / kSelThreads;                    // staged elements per thread: channel rows ..
   constexpr int EB = (kSelStage * NP + kSelThreads - 1) / kSelThreads;                    // .. B and C rows
@@ -383,14 +382,103 @@ selective_scan_kernel(const SelArgs<AT> a) {
     if (c < inner && n0 + i < N) st[n0 + i] = S[i];
 }
 
+// Every sequence of the step brings one row (decode): sequence s is row s.  No staging and no barrier: a thread takes KB groups of
+// channels, 128 / L apart, with all their states and inputs in flight at once.
+template <typename AT, int L, int NS, int KB>
+__global__ void __launch_bounds__(kSelThreads)
+selective_step_kernel(const SelArgs<AT> a, int vec) {
+  constexpr int CH = kSelThreads / L;
+  const int64_t t = blockIdx.x;
+  const int c0 = blockIdx.y * CH * KB + threadIdx.x / L, n0 = (threadIdx.x % L) * NS, N = a.n_state, inner = a.inner;
+  const bool fresh = a.positions[t] == 0;
+  float* st = a.state + (int64_t)a.seq_slots[t] * a.slot_stride;
+  float A[KB][NS], S[KB][NS];
+#pragma unroll
+  for (int k = 0; k < KB; ++k) {
+    const int c = min(c0 + k * CH, inner - 1);
+    if (vec) {   // N a multiple of 4, rows 16-byte aligned: a lane's states are there in fours
+#pragma unroll
+      for (int i = 0; i < NS; i += 4) {
+        const int64_t o = (int64_t)c * N + min(n0 + i, N - 4);
+        ldv<float, 4>(a.A, o, &A[k][i]);
+        ldv<float, 4>(st, o, &S[k][i]);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < NS; ++i) {
+        const int64_t o = (int64_t)c * N + min(n0 + i, N - 1);
+        A[k][i] = a.A[o];
+        S[k][i] = st[o];
+      }
+    }
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  AT x[KB], z[KB];
+  float dt[KB], dtb[KB], skip[KB], B[NS], C[NS];
+#pragma unroll
+  for (int k = 0; k < KB; ++k) {
+    const int c = min(c0 + k * CH, inner - 1);
+    x[k] = a.xc[t * inner + c];
+    dt[k] = a.dt_pre[t * inner + c];
+    z[k] = a.z[t * a.ldz + c];
+    dtb[k] = a.dt_bias[c];
+    skip[k] = a.D[c];
+  }
+  {
+    AT b[NS], q[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      const AT* p = a.bc + t * a.ldbc + a.b_off + min(n0 + i, N - 1);
+      b[i] = p[0];
+      q[i] = p[N];
+    }
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      B[i] = n0 + i < N ? ldf(b[i]) : 0.f;   // states past N stay out of the sums and are not stored
+      C[i] = n0 + i < N ? ldf(q[i]) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < KB; ++k) {
+    const int c = c0 + k * CH;
+    const float d = softplus_f(dt[k] + dtb[k]), xv = ldf(x[k]), dx = d * xv;
+    float y = 0.f;
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      const float s0 = fresh ? 0.f : S[k][i];
+      S[k][i] = fmaf(decay_exp2<AT>(d * (A[k][i] * 1.4426950408889634f)), s0, dx * B[i]);
+      y = fmaf(S[k][i], C[i], y);
+    }
+#pragma unroll
+    for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (c < inner) {
+      if (threadIdx.x % L == 0) {
+        float o1[1] = {fmaf(skip[k], xv, y) * silu_f(ldf(z[k]))};
+        stv<AT, 1>(a.out, t * inner + c, o1);
+      }
+      if (vec) {
+#pragma unroll
+        for (int i = 0; i < NS; i += 4)
+          if (n0 + i < N) stv<float, 4>(st, (int64_t)c * N + n0 + i, &S[k][i]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < NS; ++i)
+          if (n0 + i < N) st[(int64_t)c * N + n0 + i] = S[k][i];
+      }
+    }
+  }
+}
+
 template <typename AT>
 int selective_scan_t(const SelArgs<AT>& a, int S, bool one, cudaStream_t s) {
   const int N = a.n_state;
+  const int vec = N % 4 == 0 && a.slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state) | reinterpret_cast<uintptr_t>(a.A)) % 16 == 0;
 #define SEL(LV, NV)                                                                                                                              \
   do {                                                                                                                                           \
-    const dim3 grid(S, (a.inner + kSelThreads / LV - 1) / (kSelThreads / LV));                                                                    \
-    if (one) B200_CUDA(launch(selective_scan_kernel<AT, LV, NV, true>, grid, dim3(kSelThreads), (size_t)0, s, a));                                \
-    else B200_CUDA(launch(selective_scan_kernel<AT, LV, NV, false>, grid, dim3(kSelThreads), (size_t)0, s, a));                                   \
+    constexpr int CH = kSelThreads / LV, KB = 16 / NV;                                                                                            \
+    if (one) B200_CUDA(launch(selective_step_kernel<AT, LV, NV, KB>, dim3(S, (a.inner + CH * KB - 1) / (CH * KB)), dim3(kSelThreads), (size_t)0, s, a, vec)); \
+    else B200_CUDA(launch(selective_scan_kernel<AT, LV, NV>, dim3(S, (a.inner + CH - 1) / CH), dim3(kSelThreads), (size_t)0, s, a));              \
   } while (0)
   if (N <= 4) SEL(1, 4);
   else if (N <= 8) SEL(2, 4);
