@@ -598,6 +598,28 @@ def test_bf16_mode_within_bf16_noise_and_equal_across_schedules(model_a):
     r.close()
 
 
+def test_bf16_batches_of_long_portions_beside_single_tokens_equal_each_request_alone():
+    """Sizes that take the tensor-core kernels: steps that carry portions of many rows (chunks), of a few rows and single decoded
+    tokens of different sequences; every request gets what it gets alone, and the oracle's logits within bf16 noise."""
+    cfg = B.make_cfg(width=128, vocab=150, loop=(0, 1, 2), layers=[
+        B.retention(heads=2, dim=64, vdim=48, rot_dims=32, decay=[0.999, 0.9]),
+        B.parallel(heads=4, kv_heads=2, dim=32, vdim=32, window=50, conv=3, inner=128, state=16, dt_rank=8, conv2=4, mlp=B.dense(128))])
+    w = B.make_weights(cfg, 15)
+    prompts = {"a": _prompt(cfg, 230, 1), "b": _prompt(cfg, 90, 2), "c": _prompt(cfg, 40, 3), "d": _prompt(cfg, 75, 4)}
+    r = B.make_runner(cfg, w, "bfloat16", block_size=64, n_blocks=12, n_state_slots=5)
+    eng = U.make_engine(r)
+    mixed = U.replay(eng, [[("a", 70), ("c", 1)], [("b", 9), ("a", 1), ("c", 8)], [("c", 1), ("a", 130), ("b", 2), ("d", 64)],
+                           [("a", 1), ("b", 64), ("d", 2), ("c", 1)]] + [[("a", 1), ("b", 1), ("c", 1), ("d", 1)]] * 9 + [[("a", 19), ("c", 20)], [("b", 6)]],
+                     prompts)
+    for n, p in prompts.items():
+        alone = U.replay(eng, [[(n, len(p))]], prompts)[n]
+        e, d = U.rel_rms(alone, O.forward(cfg, w, p).numpy()), U.rel_rms(mixed[n], alone)
+        assert np.median(e) < 0.02 and (e < 0.08).mean() > 0.95, (n, float(np.median(e)), float(e.max()))
+        assert np.median(d) < 0.02 and (d < 0.08).mean() > 0.95, (n, float(np.median(d)), float(d.max()))
+    assert len(eng.blocks.free) == 12
+    r.close()
+
+
 def test_greedy_generation_through_the_engines_own_scheduler(model_a, tmp_path):
     """A checkpoint directory goes through the registry, the weight loader, LLMEngine.generate and the scheduler (which hands out
     blocks and state slots and overlaps steps); prompts of unequal length decode side by side."""
