@@ -874,8 +874,8 @@ B200_API int b200_retention_step(int32_t f32, const void* fused, int64_t ld, con
                                  int64_t max_pos, const float* decay, const int32_t* positions, const int32_t* seq_start,
                                  const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int32_t n_seqs, int32_t heads,
                                  int32_t dim, int32_t vdim, float eps, int32_t max_rows, void* stream);
-/* The same over portions longer than min_rows rows in chunks of 64 rows on the tensor cores (bf16 rows; dim and vdim multiples of 16 up to
- * 128 and rot_dims even: b200_retention_chunk_supported).  workspace: b200_retention_chunk_workspace_bytes. */
+/* The same over portions longer than min_rows rows in chunks of 64 rows on the tensor cores (bf16 rows; vdim <= 128, dim and vdim multiples of 16 whose tiles
+ * fit 200 KB, half layout with rot_dims a multiple of 4, ld a multiple of 8, 16-byte aligned rows, table and state: b200_retention_chunk_supported).  workspace: b200_retention_chunk_workspace_bytes. */
 B200_API int b200_retention_chunk_supported(int32_t dim, int32_t vdim);
 B200_API int64_t b200_retention_chunk_workspace_bytes(int32_t n_tokens, int32_t n_seqs, int32_t heads, int32_t dim, int32_t vdim);
 B200_API int b200_retention_chunk(const void* fused, int64_t ld, const float* rot, int32_t rot_dims, int32_t half_layout, int64_t max_pos,
