@@ -31,7 +31,9 @@ class StackLayer(C.Structure):
                [(n, C.c_int32) for n in ("act", "ungated", "sigmoid_scores", "weight_input", "shared_ff")] + \
                [(n, C.c_int32) for n in ("window", "q_rank", "kv_share", "conv_taps", "decay_rank", "gate_rank", "norm_groups")] + \
                [("act_limit", C.c_float), ("route_chosen", C.c_int32), ("softcap", C.c_float)] + \
-               [(n, C.c_int32) for n in ("bias_dist", "side", "side_inner", "side_state", "side_rank", "side_taps", "loop_add", "loop_step")]
+               [(n, C.c_int32) for n in ("bias_dist", "side", "side_inner", "side_state", "side_rank", "side_taps", "loop_add", "loop_step")] + \
+               [(n, C.c_int32) for n in ("keep_first", "side_blocks")] + [("mix_main", C.c_float), ("mix_side", C.c_float)] + \
+               [(n, C.c_int32) for n in ("group_best", "route_renorm", "shared_gate")]
 
 
 class StackCfg(C.Structure):
@@ -40,15 +42,16 @@ class StackCfg(C.Structure):
                [(n, C.c_int32) for n in ("f32", "block_size", "max_tokens", "max_blocks_per_seq", "max_logit_rows")] + \
                [(n, C.c_int32) for n in ("form", "canon_taps", "depth_avg", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur")] + \
                [("logit_softcap", C.c_float), ("n_state_slots", C.c_int32), ("residual_alpha", C.c_float), ("streams", C.c_int32),
-                ("residual_mult", C.c_float)]
+                ("residual_mult", C.c_float), ("norm_kind", C.c_int32)]
 
 
-MIXER_ATTENTION, MIXER_LATENT, MIXER_MLSTM, MIXER_DELTA, MIXER_SSD, MIXER_RETENTION, MIXER_SELECTIVE = 1, 2, 3, 4, 5, 6, 7
+MIXER_ATTENTION, MIXER_LATENT, MIXER_MLSTM, MIXER_DELTA, MIXER_SSD, MIXER_RETENTION, MIXER_SELECTIVE, MIXER_LRU = 1, 2, 3, 4, 5, 6, 7, 8
 MLP_NONE, MLP_MOE, MLP_DENSE = 0, 1, 2
-ACT_SILU, ACT_GELU_TANH, ACT_RELU2, ACT_RELU, ACT_SWIGLU_CLAMP, ACT_POLYNORM = 0, 1, 2, 3, 4, 5
+ACT_SILU, ACT_GELU_TANH, ACT_RELU2, ACT_RELU, ACT_SWIGLU_CLAMP, ACT_POLYNORM, ACT_GELU_ERF = 0, 1, 2, 3, 4, 5, 6
 ACTS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "relu2": ACT_RELU2, "relu": ACT_RELU, "swiglu_clamp": ACT_SWIGLU_CLAMP,
-        "polynorm": ACT_POLYNORM}
+        "polynorm": ACT_POLYNORM, "gelu_erf": ACT_GELU_ERF}
 FORM_SANDWICH, FORM_PARALLEL, FORM_POSTNORM, FORM_HYPER, FORM_LOOPED = 0, 1, 2, 3, 4
+NORM_RMS, NORM_TANH = 0, 1
 MIXF_SINK, MIXF_GATE, MIXF_HEAD_NORM, MIXF_VALUE_IS_KEY, MIXF_SINK_ONE, MIXF_HEAD_GATE = 1, 2, 4, 8, 16, 32
 MIXF_ROT_HALF, MIXF_NO_QK_NORM, MIXF_HEAD_DECAY, MIXF_QKV_BIAS = 64, 128, 256, 512
 MAX_STREAMS = 8
@@ -59,13 +62,13 @@ MAX_STREAMS = 8
  SW_GATE_UP, SW_MLP_GATE_UP_INTERLEAVED, SW_NORM_MIX_PRE_BIAS, SW_NORM_MLP_PRE_BIAS, SW_SCALE_MIX, SW_SCALE_MLP, SW_HC_MIX, SW_HC_MLP,
  SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT, SW_EMBED_NORM, SW_LOOP_STEP, SW_QKV_BIAS, SW_DIST_BIAS, SW_DECAY, SW_SIDE_CONV,
  SW_SIDE_CONV_BIAS, SW_SIDE_PROJ, SW_SIDE_DT, SW_SIDE_DT_BIAS, SW_SIDE_A, SW_SIDE_SKIP, SW_SIDE_O, SW_OUT_MAIN, SW_OUT_SIDE,
- SW_MLP_UP_BIAS, SW_MLP_DOWN_BIAS) = range(66)
+ SW_MLP_UP_BIAS, SW_MLP_DOWN_BIAS, SW_NORM_ALPHA, SW_FINAL_NORM_ALPHA, SW_SIDE_GATES, SW_SIDE_GATES_BIAS, SW_SIDE_DECAY) = range(71)
 SW_F32 = {SW_FINAL_NORM, SW_NORM_MIX_PRE, SW_NORM_MIX_POST, SW_NORM_MLP_PRE, SW_NORM_MLP_POST, SW_Q_NORM, SW_K_NORM, SW_ROUTER_BIAS,
           SW_CANON, SW_DEPTH_AVG, SW_SINK, SW_GATES_BIAS, SW_HEAD_NORM, SW_NORM_MIX_POST_BIAS, SW_NORM_MLP_POST_BIAS,
           SW_FINAL_NORM_BIAS, SW_Q_LATENT_NORM, SW_CONV, SW_DECAY_BIAS, SW_DECAY_LOG, SW_NORM_MIX_PRE_BIAS, SW_NORM_MLP_PRE_BIAS,
           SW_SCALE_MIX, SW_SCALE_MLP, SW_HC_MIX, SW_HC_MLP, SW_CANON_MLP, SW_CONV_BIAS, SW_SKIP, SW_MLP_ACT,
           SW_EMBED_NORM, SW_LOOP_STEP, SW_DIST_BIAS, SW_DECAY, SW_SIDE_CONV, SW_SIDE_CONV_BIAS, SW_SIDE_DT_BIAS, SW_SIDE_A, SW_SIDE_SKIP,
-          SW_OUT_MAIN, SW_OUT_SIDE}
+          SW_OUT_MAIN, SW_OUT_SIDE, SW_NORM_ALPHA, SW_FINAL_NORM_ALPHA, SW_SIDE_GATES_BIAS, SW_SIDE_DECAY}
 
 W_EMBED, W_LN1, W_QKV, W_QKV_BIAS, W_O, W_LN2, W_GATE_UP, W_DOWN, W_FINAL_NORM, W_LM_HEAD, W_GATE_UP_INTERLEAVED = range(11)
 
@@ -208,6 +211,14 @@ SIGNATURES = {
     "b200_paged_attn_biased": (C.c_int, [_i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32,
                                          _f32, _vp, _i32, _vp, _i64, _vp, _i32, _vp, _vp]),
     "b200_linear_bias_act": (C.c_int, [_i32, _i32, _vp, _i64, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _i64, _vp]),
+    "b200_tanh_close": (C.c_int, [_i32, _vp, _vp, _f32, _vp, _f32, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _vp]),
+    "b200_qk_norm_cache": (C.c_int, [_i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
+    "b200_side_conv": (C.c_int, [_i32, _vp, _i64, _vp, _vp, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp]),
+    "b200_gated_lru": (C.c_int, [_i32, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _vp]),
+    "b200_latent_prep_half": (C.c_int, [_i32, _vp, _i64, _vp, _vp, _vp, _vp, _i32, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
+    "b200_moe_route_form": (C.c_int, [_i32, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp]),
+    "b200_paged_attn_kept": (C.c_int, [_i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32,
+                                       _vp, _vp, _i32, _vp, _i32, _vp, _vp]),
     "b200_ssd_prep": (C.c_int, [_i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32,
                                 _i32, _i32, _i32, _vp]),
     "b200_ssd_gate_norm": (C.c_int, [_i32, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp]),

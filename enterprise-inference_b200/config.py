@@ -209,6 +209,7 @@ class AttentionSpec:
     bias_max: float = 0.0                  # > 0: a learned bias by distance joins the score, one table row from this distance on
     head_gate: bool = False                # one sigmoid gate per head, read from the mixer's input
     sink: bool = False                     # a learned per-head term exp(sink) in the softmax denominator
+    keep_first: int = 0                    # with a window: the first positions that every query sees besides it
 
 
 @dataclass
@@ -224,7 +225,9 @@ class MoESpec:
 class StackLayerSpec:
     mixer: object                     # AttentionSpec | LatentAttentionSpec | ChannelDeltaSpec | HeadDeltaSpec | StateSpaceSpec | RetentionSpec
     mlp: Optional[object] = None      # MoESpec | FeedForwardSpec
-    side: Optional[object] = None     # SelectiveScanSpec: a second mixer that reads the same input; the results are normed and averaged
+    side: Optional[object] = None     # a second mixer that reads the same input.  SelectiveScanSpec: the results are normed and averaged;
+                                      # GatedLRUSpec: their sum, weighted by side_mix
+    side_mix: Tuple[float, float] = (1.0, 1.0)
 
 
 @dataclass
@@ -328,6 +331,7 @@ class LatentAttentionSpec:
     window: int = 0                        # positions a query sees, its own included (0: all)
     head_gate: bool = False                # one sigmoid gate per head (instead of one per output)
     kv_from: Optional[int] = None          # the layer whose cached latent rows this layer reads (None: its own)
+    rot_half: bool = False                 # rotated dimension i pairs with i + rot.dims / 2 (else 2i with 2i + 1)
 
 
 @dataclass
@@ -355,6 +359,12 @@ class FeedForwardSpec:
     limit: float = 0.0                     # act "swiglu_clamp": min(gate, limit) * sigmoid(1.702 gate) * (clamp(up, +-limit) + 1)
     router: str = ""                       # "chosen_softmax": bias inside the logits, weights = softmax over the chosen logits
     bias: bool = False                     # dense: both projections have biases
+    groups: int = 1                        # moe: equal groups of neighbouring experts, of which only the `keep` best stay eligible
+    keep: int = 1
+    group_best: int = 1                    # a group counts by the sum of this many of its largest choice scores
+    renorm: bool = False                   # mixing weights are divided by their sum
+    weight_input: bool = True              # the mixing weight scales the expert's input (else its output)
+    shared_gate: bool = False              # the shared expert's result is scaled by a sigmoid read from the input
 
 
 @dataclass
@@ -797,11 +807,7 @@ class BofusunConfig:
 
     def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
         """(layer, pass) in the order they run; pass is None outside the loop."""
-        n = len(self.layers)
-        if self.loop_times <= 0:
-            return [(i, None) for i in range(n)]
-        a, b = self.loop_start, self.loop_stop
-        return [(i, None) for i in range(a)] + [(i, t) for t in range(self.loop_times) for i in range(a, b)] + [(i, None) for i in range(b, n)]
+        return unrolled_runs(len(self.layers), self.loop_start, self.loop_stop, self.loop_times)
 
     @property
     def n_layers(self) -> int:
@@ -885,6 +891,165 @@ class BofusunConfig:
                              loop_start=start, loop_stop=stop, loop_times=times, layers=layers)
 
 
+# ---- Rirusun ----------------------------------------------------------------------------------------------------------------
+@dataclass
+class GatedLRUSpec:
+    """Real-gated linear recurrent unit: `inner` channels in `blocks` equal parts with gate matrices of their own, a causal
+    convolution of `conv` taps with bias ahead of it, the result times gelu of a second branch of the same size."""
+    inner: int
+    blocks: int
+    conv: int
+    kind: str = "lru"
+
+
+@dataclass
+class RirusunConfig:
+    """Rirusun: decoder-only, one elementwise norm per layer (tanh of the scaled stream, weight, bias) whose output the mixer and
+    the routed experts both read, x += mixer(h) + experts(h), and a run of layers that is passed several times with the same weights
+    (each pass with its own cache and state).  Mixers: latent attention (half-layout rotation with YaRN scaling, plain softmax), the
+    mLSTM recurrence, and windowed attention with kept first positions, distance bias and sink beside a gated linear recurrent unit.
+    Experts: ungated, exact gelu; sigmoid scores with a choice bias, group-limited by the sum of a group's two best, weights that sum
+    to one; one gated shared expert."""
+    name: str = "rirusun"
+    width: int = 256
+    vocab: int = 1024
+    embed_scale: float = 1.0
+    norm_eps: float = 1e-6
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0                    # 0: no loop
+    layers: List[StackLayerSpec] = field(default_factory=list)
+    architecture: str = "Rirusun"
+    # what the parallel form of other designs has and this one does not
+    canon_taps: int = 0
+    bigram_buckets: int = 0
+    bigram_mul_prev: int = 0
+    bigram_mul_cur: int = 0
+    logit_softcap: float = 0.0
+    depth_avg: bool = False
+
+    @property
+    def hidden(self) -> int:
+        return self.width
+
+    def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
+        """(layer, pass) in the order they run; pass is None outside the loop."""
+        return unrolled_runs(len(self.layers), self.loop_start, self.loop_stop, self.loop_times)
+
+    @property
+    def n_layers(self) -> int:
+        """Layer runs: every pass of a looped layer counts, with a cache and a state of its own."""
+        return len(self.layer_runs())
+
+    @property
+    def needs_state(self) -> bool:
+        return any(isinstance(L.mixer, MLSTMSpec) or L.side is not None for L in self.layers)
+
+    def to_dict(self):
+        return asdict(self)
+
+    def _layer_params(self, L, active_only: bool) -> int:
+        W, a, s, f = self.width, L.mixer, L.side, L.mlp
+        if isinstance(a, MLSTMSpec):
+            n = W * (2 * a.heads * a.dim + 2 * a.heads * a.vdim + 2 * a.heads) + a.heads * a.vdim * W
+        elif isinstance(a, LatentAttentionSpec):
+            n = W * (a.heads * (a.dim + a.rot_dim) + a.kv_rank + a.rot_dim) + a.heads * a.kv_rank * (a.dim + a.vdim) + a.heads * a.vdim * W
+        else:
+            n = W * (a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)) + a.heads * a.vdim * W
+        if s is not None:
+            n += 3 * W * s.inner + 2 * s.inner * (s.inner // s.blocks)
+        if f is not None:
+            n += (f.experts + int(f.shared_gate)) * W + (f.top if active_only else f.experts) * 2 * f.ff * W + 2 * f.shared_ff * W
+        return n
+
+    def decode_params(self) -> int:
+        """Weights one decode row multiplies (chosen experts only; a looped layer counts in every pass)."""
+        return self.vocab * self.width + sum(self._layer_params(self.layers[i], True) for i, _ in self.layer_runs())
+
+    def weight_bytes(self) -> int:
+        return 2 * (2 * self.vocab * self.width + sum(self._layer_params(L, False) for L in self.layers))
+
+    def kv_bytes_per_token(self, f32: bool = False) -> int:
+        n = 0
+        for i, _ in self.layer_runs():
+            a = self.layers[i].mixer
+            if isinstance(a, LatentAttentionSpec):
+                n += a.kv_rank + a.rot_dim
+            elif isinstance(a, AttentionSpec):
+                n += a.kv_heads * (a.dim + a.vdim)
+        return n * (4 if f32 else 2)
+
+    @staticmethod
+    def _latent(m: dict, where: str) -> LatentAttentionSpec:
+        rot, r, rd = None, m.get("rot"), int(m.get("rot_dim") or 0)
+        if r and int(r.get("dims") or 0) > 0 and rd > 0:
+            sc = r.get("scaling")
+            extra = dict(factor=float(sc["factor"]), original=int(sc["original"]), fast=float(sc["fast"]), slow=float(sc["slow"]), scaled=True) if sc else {}
+            rot = RotarySpec(base=float(r["base"]), dims=int(r["dims"]), **extra)
+            if rot.dims % 2 or rot.dims > rd:
+                raise ValueError(f"{where}: {rot.dims} rotated dimensions in a part of {rd}")
+        return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=rd, vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                                   scale=float(m["scale"]), rot=rot, rot_half=True)
+
+    @staticmethod
+    def _attention(m: dict, where: str) -> AttentionSpec:
+        mask = m.get("mask") or {}
+        a = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]),
+                          scale=float(m["scale"]), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                          bias_max=float(m.get("bias_max") or 0.0), sink=True)
+        if a.heads % a.kv_heads:
+            raise ValueError(f"{where}: {a.heads} heads over {a.kv_heads} key heads")
+        return a
+
+    @staticmethod
+    def _experts(f: dict, where: str) -> FeedForwardSpec:
+        if f.get("kind", "moe") != "moe":
+            raise ValueError(f"{where}: unsupported feed-forward kind {f.get('kind')!r}")
+        r = f["router"]
+        g, sh = r.get("groups") or {}, f.get("shared") or {}
+        groups = int(g.get("count") or 1)
+        out = FeedForwardSpec(kind="moe", ff=int(f["expert"]["ff"]), act="gelu_erf", experts=int(r["experts"]), top=int(r["top"]), gated=False,
+                              groups=groups, keep=int(g.get("keep") or groups), group_best=2, renorm=True, weight_input=False,
+                              shared_ff=int(sh.get("ff") or 0), shared_gate=int(sh.get("ff") or 0) > 0)
+        if out.experts % groups or not 0 < out.keep <= groups or not 0 < out.top <= out.keep * (out.experts // groups):
+            raise ValueError(f"{where}: top {out.top} of {out.experts} experts in {groups} groups, {out.keep} kept")
+        return out
+
+    @staticmethod
+    def from_dict(c: dict, name: str = "rirusun") -> "RirusunConfig":
+        layers = []
+        for i, l in enumerate(c["layers"]):
+            kind, m, where = l.get("type"), l["mixer"], f"layer {i}"
+            side, mix = None, (1.0, 1.0)
+            if kind == "latent_attention":
+                mixer = RirusunConfig._latent(m, where)
+            elif kind == "mlstm":
+                mixer = MLSTMSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]), gate_cap=float(m["gate_cap"]))
+            elif kind == "parallel":
+                mixer, b = RirusunConfig._attention(m["left"], where), m["right"]
+                side = GatedLRUSpec(inner=int(b["width"]), blocks=int(b.get("blocks") or 1), conv=int(b.get("conv") or 1))
+                mix = (float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0)))
+                if side.inner % side.blocks:
+                    raise ValueError(f"{where}: {side.inner} channels in {side.blocks} blocks")
+            else:
+                raise ValueError(f"{where}: unsupported mixer type {kind!r} (this design has latent_attention, parallel, mlstm)")
+            f = l.get("mlp")
+            layers.append(StackLayerSpec(mixer=mixer, mlp=RirusunConfig._experts(f, where) if f else None, side=side, side_mix=mix))
+        loop = c.get("loop") or {}
+        start, stop, times = int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 0))
+        if loop and not (0 <= start < stop <= len(layers) and times >= 1):
+            raise ValueError(f"loop over layers {start} .. {stop - 1} of {len(layers)}, {times} times")
+        return RirusunConfig(name=name, width=int(c["width"]), vocab=int(c["vocab"]), embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)),
+                             norm_eps=float((c.get("norm") or {}).get("eps", 1e-6)), loop_start=start, loop_stop=stop, loop_times=times, layers=layers)
+
+
+def unrolled_runs(n: int, start: int, stop: int, times: int) -> List[Tuple[int, Optional[int]]]:
+    """(layer, pass) of n layers in the order they run: layers start .. stop - 1 `times` times in a row (times 0: no loop, pass None)."""
+    if times <= 0:
+        return [(i, None) for i in range(n)]
+    return [(i, None) for i in range(start)] + [(i, t) for t in range(times) for i in range(start, stop)] + [(i, None) for i in range(stop, n)]
+
+
 def distance_bucket(n: int, rows: int, far: float) -> int:
     """Row of a learned distance table: the distance itself below rows / 2, then logarithmic, the last row from `far` on."""
     half = rows // 2
@@ -893,10 +1058,11 @@ def distance_bucket(n: int, rows: int, far: float) -> int:
     return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
 
 
-def distance_entries(window: int, far: float) -> int:
-    """Distances that need an entry of their own: what the window shows, and no further than the distance the last row starts at."""
+def distance_entries(window: int, far: float, keep_first: int = 0) -> int:
+    """Distances that need an entry of their own: what the window shows (any distance, where it keeps first positions), and no
+    further than the distance the last row starts at."""
     n = math.ceil(far) + 1
-    return min(n, window) if window > 0 else n
+    return min(n, window) if window > 0 and keep_first <= 0 else n
 
 
 def checkpoint_shapes(path: str) -> Dict[str, list]:
@@ -917,7 +1083,7 @@ def checkpoint_shapes(path: str) -> Dict[str, list]:
 
 # config.json "architecture" -> reader.  HF-style configs (model_type) go through from_hf_config.
 ARCHITECTURES = {"Bopilorn": BopilornConfig.from_dict, "Dupolorn": DupolornConfig.from_dict, "Futidra": FutidraConfig.from_dict,
-                 "Rudolix": RudolixConfig.from_dict, "Bofusun": BofusunConfig.from_dict}
+                 "Rudolix": RudolixConfig.from_dict, "Bofusun": BofusunConfig.from_dict, "Rirusun": RirusunConfig.from_dict}
 NEEDS_SHAPES = {"Futidra"}   # readers that take the checkpoint's tensor shapes for sizes config.json does not name
 
 

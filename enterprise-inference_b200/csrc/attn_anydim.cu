@@ -1,6 +1,6 @@
 // Paged causal softmax attention (optionally over a sliding window of the last `window` keys) for heads of any size
 // (query/key size `dim`, value size `vdim`, dim != vdim allowed),
-// any block size, a caller-given score scale (with an optional cap and a bias by distance: AttnExtra), fp32 queries and a bf16 or fp32 cache.  The tcgen05 kernels of attn_tc.cu /
+// any block size, a caller-given score scale (with an optional cap, a bias by distance and first keys that a window keeps: AttnExtra), fp32 queries and a bf16 or fp32 cache.  The tcgen05 kernels of attn_tc.cu /
 // attn_prefill.cu are built for 128-wide heads; this file serves every other head shape on CUDA cores with fp32 scores,
 // fp32 softmax weights and fp32 accumulation.
 //
@@ -46,6 +46,12 @@ __device__ __forceinline__ float block_sum128(float v, float* red) {
   return (red[0] + red[1]) + (red[2] + red[3]);
 }
 
+// the tile after `base`: past the kept first keys the walk goes on at the window's first tile
+__device__ __forceinline__ int next_tile(int base, int tile, int keep, int lo_tile) {
+  const int n = base + tile;
+  return n >= keep ? max(n, lo_tile) : n;
+}
+
 template <typename CT, typename AT>
 __global__ void __launch_bounds__(kAdThreads)
 paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, const CT* __restrict__ vc,
@@ -73,13 +79,14 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
 #pragma unroll
   for (int i = 0; i < kAdMaxVPer; ++i) acc[i] = 0.f;
   __syncthreads();
-  const int lo = window > 0 ? max(ctx - window, 0) : 0;   // the first key the row sees; the tile that holds it is the first walked
-  for (int base = lo - lo % kAdThreads; base < ctx; base += kAdThreads) {
+  const int lo = window > 0 ? max(ctx - window, 0) : 0;   // the window's first key; the tile that holds it is the first walked,
+  const int keep = ex.keep_first, lo_tile = lo - lo % kAdThreads;   // after those of the kept first keys
+  for (int base = keep > 0 ? 0 : lo_tile; base < ctx; base = next_tile(base, kAdThreads, keep, lo_tile)) {
     const int j = base + tid;
     float sc = -INFINITY;
-    int blk = 0;
-    if (j < ctx && j >= lo) {
-      blk = bt[j / block_size];
+    const int blk = j < ctx ? bt[j / block_size] : 0;
+    const bool see = j < ctx && (j >= lo || j < keep);
+    if (see) {
       const CT* kp = kc + (((int64_t)blk * kv_heads + g) * block_size + j % block_size) * kst;
       float a = 0.f;
       for (int d = 0; d < dim; ++d) a = fmaf(qs[d], cache_load<CT>(kp, d), a);
@@ -87,7 +94,7 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
     }
     const float tm = block_max128(sc, red);
     const float mn = fmaxf(m, tm);
-    const float p = (j < ctx && j >= lo) ? expf(sc - mn) : 0.f;
+    const float p = see ? expf(sc - mn) : 0.f;
     const float corr = expf(m - mn);      // first tile: exp(-inf) = 0
     const float ts = block_sum128(p, red);
     l = l * corr + ts;
@@ -101,7 +108,7 @@ paged_attn_rows_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
       const int d = tid + i * kAdThreads;
       if (d < vdim) {
         float a = acc[i] * corr;
-        for (int jj = max(lo - base, 0); jj < n; ++jj) {
+        for (int jj = base < keep ? 0 : max(lo - base, 0); jj < n; ++jj) {   // (a tile of kept keys: weights of the others are zero)
           const CT* vp = vc + (((int64_t)blk_of[jj] * kv_heads + g) * block_size + (base + jj) % block_size) * vst;
           a = fmaf(ps[jj], cache_load<CT>(vp, d), a);
         }
@@ -245,7 +252,8 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
   __syncthreads();
   // with a window the run's first row sees the oldest key of all: the walk starts at the tile that holds it
   const int lo_run = window > 0 ? max(ctx_lens[t0] - window, 0) : 0;
-  for (int base = lo_run - lo_run % kTileKeys; base < ctx_max; base += kTileKeys) {
+  const int keep = ex.keep_first, lo_tile = lo_run - lo_run % kTileKeys;
+  for (int base = keep > 0 ? 0 : lo_tile; base < ctx_max; base = next_tile(base, kTileKeys, keep, lo_tile)) {
     const int n = min(kTileKeys, ctx_max - base);
     for (int i = threadIdx.x; i < n * dim; i += kTcThreads) {
       const int jj = i / dim, d = i % dim, j = base + jj;
@@ -263,10 +271,11 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
         const int r = qi / G;
         const int ctx = ctx_lens[t0 + r];
         const int lo = window > 0 ? max(ctx - window, 0) : 0;
-        if (base < ctx && base + n > lo) {
+        if (base < ctx && (base + n > lo || base < keep)) {
           const int j = base + lane;
           float sc = -INFINITY;
-          if (j < ctx && j >= lo) {
+          const bool see = j < ctx && (j >= lo || j < keep);
+          if (see) {
             const float* qp = Qs + qi * dim;
             const float* kp = Ks + lane * kst;
             float a = 0.f;
@@ -275,7 +284,7 @@ paged_attn_runs_kernel(const float* __restrict__ q, const CT* __restrict__ kc, c
             sc = score_shape(a * scale, ex.softcap, brow, ctx - 1 - j, ex.bias_dist);
           }
           const float mn = fmaxf(m[k], warp_max(sc));
-          const float p = (j < ctx && j >= lo) ? expf(sc - mn) : 0.f;
+          const float p = see ? expf(sc - mn) : 0.f;
           const float corr = expf(m[k] - mn);
           l[k] = l[k] * corr + warp_sum(p);
           m[k] = mn;

@@ -51,7 +51,7 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// NG: 16-column output groups per warp (rank <= 128 NG).  EX: score cap, distance bias and per-head gate of AttnExtra.
+// NG: 16-column output groups per warp (rank <= 128 NG).  EX: score cap, distance bias, per-head gate and kept first keys of AttnExtra.
 template <int NG, bool EX>
 __global__ void __launch_bounds__(kLaThreads)
 latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
@@ -109,9 +109,12 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
   // with n_splits > 1 this CTA walks only its share of the tiles and leaves unnormalised sums for the merge kernel
   // (with a window the walk starts at the tile that holds the oldest key the group's first row sees)
   const int tile0 = window > 0 ? max(ctx_lens[t0 + i0 / G] - window, 0) / kLaKeys : 0;
-  const int tiles = (ctx_max + kLaKeys - 1) / kLaKeys - tile0, per = (tiles + n_splits - 1) / n_splits;
-  const int base_lo = (tile0 + blockIdx.z * per) * kLaKeys, base_hi = min(ctx_max, (tile0 + (int)(blockIdx.z + 1) * per) * kLaKeys);
-  for (int base = base_lo; base < base_hi; base += kLaKeys) {
+  // first keys that the window keeps: their tiles lead the walk, those between them and the window are skipped
+  const int keep = EX ? ex.keep_first : 0, lead = EX ? min((keep + kLaKeys - 1) / kLaKeys, tile0) : 0;
+  const int tiles = (ctx_max + kLaKeys - 1) / kLaKeys - tile0 + lead, per = (tiles + n_splits - 1) / n_splits;
+  const int walk_lo = blockIdx.z * per, walk_hi = min(tiles, (int)(blockIdx.z + 1) * per);
+  for (int w = walk_lo; w < walk_hi; ++w) {
+    const int base = (w < lead ? w : w - lead + tile0) * kLaKeys;
     const int n = min(kLaKeys, ctx_max - base);
     {
       // four threads per key row, alternate 16-byte chunks: one block-table lookup per thread and tile
@@ -160,7 +163,7 @@ latent_attn_mma_kernel(const float* __restrict__ q, const __nv_bfloat16* __restr
     for (int rr = 0; rr < kLaPairs / kLaWarps; ++rr) {
       const int row = warp * (kLaPairs / kLaWarps) + rr, c = ctxp[row], lo = lop[row];
       const int j0 = base + lane, j1 = j0 + 32;
-      const bool see0 = j0 < c && j0 >= lo, see1 = j1 < c && j1 >= lo;
+      const bool see0 = j0 < c && (j0 >= lo || (EX && j0 < keep)), see1 = j1 < c && (j1 >= lo || (EX && j1 < keep));
       float s0 = see0 ? Ss[row * kSsStride + lane] * scale : -INFINITY;
       float s1 = see1 ? Ss[row * kSsStride + lane + 32] * scale : -INFINITY;
       if constexpr (EX) {

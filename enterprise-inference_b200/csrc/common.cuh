@@ -82,6 +82,7 @@ __device__ __forceinline__ float warp_max(float v) {
 // activations of the feed-forwards (b200_act_kind), fp32
 __device__ __forceinline__ float act_apply(float z, int kind) {
   if (kind == B200_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (kind == B200_ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
   if (kind == B200_ACT_RELU) return fmaxf(z, 0.f);
   if (kind == B200_ACT_RELU2) {
     const float r = fmaxf(z, 0.f);
@@ -243,7 +244,7 @@ int linear_tc(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, const
 int linear_tc_grouped_tile(int pairs, int experts);
 int linear_tc_grouped(const __nv_bfloat16* x, int64_t ldx, int N, int n_tiles, const __nv_bfloat16* w, int experts, int n_out, int k,
                       const int32_t* tile_expert, __nv_bfloat16* y, int64_t ldy, const int32_t* row_pair, const float* wts,
-                      float* out, cudaStream_t s);
+                      float* out, cudaStream_t s, int act = -1);   // act: b200_act_kind applied to y's fp32 sums (-1: none)
 int linear_tc_grouped_gate_up(const __nv_bfloat16* x, int64_t ldx, int N, int n_tiles, const __nv_bfloat16* w, int experts, int ff,
                               int k, const int32_t* tile_expert, __nv_bfloat16* y, cudaStream_t s, int act = 0, float act_limit = 0.f);
 // act: b200_act_kind of the gate in the epilogue (0: silu; B200_ACT_SWIGLU_CLAMP with act_limit)
@@ -324,14 +325,16 @@ int rotate_back_rows(const __nv_bfloat16* in, int in_stride, __nv_bfloat16* out,
                      int heads, int vdim, int64_t max_pos, cudaStream_t s);
 int convert_f32_to_bf16(const float* in, __nv_bfloat16* out, int64_t n, cudaStream_t s);
 int convert_bf16_to_f32(const __nv_bfloat16* in, float* out, int64_t n, cudaStream_t s);
-// What a score and an output row may take besides scale, window and sink: score cap, bias by distance, one sigmoid gate per head
+// What a score and an output row may take besides scale, window and sink: score cap, bias by distance, one sigmoid gate per head,
+// first keys that a window keeps
 struct AttnExtra {
   float softcap = 0.f;               // > 0: s = softcap tanh(s / softcap)
   const float* dist_bias = nullptr;  // [heads][bias_dist] fp32, added after the cap: entry min(i - j, bias_dist - 1)
   int bias_dist = 0;
   const void* gate = nullptr;        // gate[t * ldg + h], activation type
   int64_t ldg = 0;
-  bool any() const { return softcap > 0.f || dist_bias != nullptr || gate != nullptr; }
+  int keep_first = 0;                // with a window: keys 0 .. keep_first - 1 stay visible besides it
+  bool any() const { return softcap > 0.f || dist_bias != nullptr || gate != nullptr || keep_first > 0; }
 };
 // paged softmax attention for any head sizes (attn_anydim.cu)
 int64_t paged_attn_anydim_workspace_bytes(int T);
@@ -363,9 +366,16 @@ bool moe_tc_supported(int width, int ff);
 // logits_ws ([T][experts] fp32) given and bf16 rows: the logits come from the tcgen05 linear (lin_ws: its split-K workspace)
 // score_mode 0: softmax over all experts, the bias joins the choice only; 1: every expert's score is the sigmoid of its logit;
 // 2: the bias joins the logits, the largest logits are chosen, weights = softmax over the chosen logits
+// RouteForm: what else a router may do; gate_out given: w_router has one more row, and sigmoid of its logit goes to gate_out[t]
+// (logits_ws then holds [T][experts + 1])
+struct RouteForm {
+  int group_best = 1;      // a group's score: the sum of this many of its largest choice scores (1 or 2)
+  bool renorm = false;     // the chosen experts' weights are divided by their sum
+  float* gate_out = nullptr;
+};
 int moe_route(bool f32, const void* x, const __nv_bfloat16* w_router, const float* bias, int T, int width, int experts, int top,
               int groups, int keep, int32_t* out_ids, float* out_w, cudaStream_t s, float* logits_ws = nullptr,
-              void* lin_ws = nullptr, int64_t lin_ws_bytes = 0, int score_mode = 0);
+              void* lin_ws = nullptr, int64_t lin_ws_bytes = 0, int score_mode = 0, RouteForm rf = RouteForm());
 // The shape of an expert: gated = down(act(gate x) * (up x)) over [expert][2 ff][width], else down(act(up x)) over
 // [expert][ff][width]; weight_input: the mixing weight scales the expert's input row instead of its output row.
 struct ExpertForm {
@@ -396,7 +406,7 @@ int ff_act(bool f32, const void* in, void* out, int T, int ff, bool gated, int k
 int logit_cap(const float* in, float* out_f32, __nv_bfloat16* out_bf16, int R, int vocab, int ld, float cap, cudaStream_t s);
 int latent_prep(bool f32, const void* qkv, int64_t ld, const float* norm_w, const int32_t* positions, const int32_t* slots,
                 const float* rot, int rot_dims, int64_t max_pos, float* qfull, void* cache, int T, int heads, int dim, int rot_dim,
-                int kv_rank, float eps, cudaStream_t s);
+                int kv_rank, float eps, cudaStream_t s, bool half_layout = false);
 int head_linear(bool f32, bool y_f32, const void* x, int64_t ldx, int x_hs, const __nv_bfloat16* w, void* y, int64_t ldy, int y_hs,
                 const void* gate, int64_t ldg, int g_hs, int T, int heads, int n_out, int k, cudaStream_t s, int g_es = 1);
 int mlstm_gates(bool f32, const void* x, const __nv_bfloat16* w, const float* bias, float* out, int T, int width, int heads, float cap,
@@ -473,11 +483,24 @@ int retention_chunk(const void* fused, int64_t ld, const float* rot, int rot_dim
 int conv_inputs(bool f32, const void* fused, int64_t ld, const float* conv_a, int taps_a, float* tails_a, const float* conv_x, const float* bias_x,
                 int taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
                 const int32_t* seq_slots, const int32_t* slots, float* qout, void* kc, void* vc, void* xc, int T, int heads, int kv_heads,
-                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s);
+                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s, bool silu_x = true);
 int selective_dt_pad(int rank);
 int selective_rows(int rank, int state);
 int selective_scan(bool f32, const void* xc, const void* bc, int64_t ldbc, int b_off, const float* dt_pre, const float* dt_bias, const float* A,
                    const float* D, const void* z, int64_t ldz, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots,
                    float* state, int64_t slot_stride, void* out, int S, int inner, int n_state, bool one_row, cudaStream_t s);
+
+// parallel form with the elementwise norm (tanh_stream.cu): x[t] += sa ya + sb yb + sum of parts + sh_gate[t] y_sh, then
+// out = tanh(alpha x) w + b.  With `rows` only those rows are read and x is left as it is.
+int tanh_close(bool f32, float* x, const void* ya, float sa, const void* yb, float sb, const float* parts, int n_parts, const void* y_sh,
+               const float* sh_gate, const float* alpha, const float* w, const float* b, void* out, const int32_t* rows, int R, int width,
+               cudaStream_t s);
+// q and k RMS-normalised over the whole projection, v as it is: fp32 queries, k and v into the paged cache; ld: elements per fused row
+int qk_norm_cache(bool f32, const void* fused, int64_t ld, const float* qw, const float* kw, const int32_t* slots, float* qout, void* kc, void* vc,
+                  int T, int heads, int kv_heads, int dim, int vdim, int block_size, float eps, cudaStream_t s);
+// gated linear recurrent unit (lru.cu): gates [T][blocks][2 block] are the gate products before bias, y the other branch (gelu here)
+int gated_lru(bool f32, const void* u, const float* gates, const float* gate_bias, const float* decay, const void* y, int64_t ldy,
+              const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int S,
+              int width, int blocks, bool one_row, cudaStream_t s);
 
 }  // namespace b200

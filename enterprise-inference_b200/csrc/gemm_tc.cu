@@ -1206,7 +1206,7 @@ static int launch_grouped(bool scatter, const CUtensorMap& mw, const CUtensorMap
 
 int linear_tc_grouped(const __nv_bfloat16* x, int64_t ldx, int N, int n_tiles, const __nv_bfloat16* w, int experts, int n_out, int k,
                       const int32_t* tile_expert, __nv_bfloat16* y, int64_t ldy, const int32_t* row_pair, const float* wts,
-                      float* out, cudaStream_t s) {
+                      float* out, cudaStream_t s, int act) {
   B200_REQUIRE(linear_tc_grouped_supported(n_out, k), B200_ERR_UNSUPPORTED, "linear_tc_grouped: k=%d must be a multiple of 8", k);
   B200_REQUIRE(x && w && tile_expert && reinterpret_cast<uintptr_t>(x) % 16 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0 &&
                    ldx % 8 == 0,
@@ -1236,6 +1236,7 @@ int linear_tc_grouped(const __nv_bfloat16* x, int64_t ldx, int N, int n_tiles, c
   p.grp_wt = wts;
   p.grp_out = out;
   p.tile_n = N;
+  p.post_act = act < 0 ? 0 : act + 1;
   CUtensorMap mw, mx;
   int rc = get_map(w, (uint64_t)experts * n_out, (uint64_t)k, (uint64_t)k, kBlockM, &mw);
   if (rc) return rc;

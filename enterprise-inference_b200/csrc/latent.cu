@@ -7,7 +7,7 @@
 // latents (the row's first kv_rank entries are the "values") is expanded by W_uv afterwards.
 //
 //  * latent_prep: RMS norm of the latent with its weight, rotation of the shared key part and of every head's rotated query
-//    part (interleaved pairs, fp32 cos|sin table), cache append, rotated query parts into the fp32 query rows;
+//    part (interleaved pairs or the half layout, fp32 cos|sin table), cache append, rotated query parts into the fp32 query rows;
 //  * head_linear: y[t][h] = W[h] x[t][h] for every head at once, strided rows in and out, fp32 accumulation, optional
 //    sigmoid gate on the output (the output gate of the mixer reads the same input as the projections).
 #include <stdlib.h>
@@ -29,7 +29,7 @@ template <typename AT>
 __global__ void __launch_bounds__(128)
 latent_prep_kernel(const AT* __restrict__ qkv, int64_t ld, const float* __restrict__ norm_w, const int32_t* __restrict__ positions,
                    const int32_t* __restrict__ slots, const float* __restrict__ rot, int rot_dims, int64_t max_pos,
-                   float* __restrict__ qfull, AT* __restrict__ cache, int heads, int dim, int rot_dim, int kv_rank, float eps) {
+                   float* __restrict__ qfull, AT* __restrict__ cache, int heads, int dim, int rot_dim, int kv_rank, float eps, int half_layout) {
   __shared__ float red[4];
   pdl_wait();
   pdl_launch_dependents();
@@ -58,8 +58,11 @@ latent_prep_kernel(const AT* __restrict__ qkv, int64_t ld, const float* __restri
     const AT* src = hv < heads ? row + (int64_t)hv * qh + dim : dkv + kv_rank;
     float v = ldx<AT>(src, i);
     if (cs && i < 2 * half) {
-      const float o = ldx<AT>(src, i ^ 1), c = cs[i >> 1], s = cs[half + (i >> 1)];
-      v = (i & 1) ? fmaf(v, c, o * s) : fmaf(v, c, -o * s);
+      // interleaved: i turns with i ^ 1; half layout: i with i + half
+      const int pr = half_layout ? (i < half ? i : i - half) : i >> 1;
+      const bool second = half_layout ? i >= half : (i & 1);
+      const float o = ldx<AT>(src, half_layout ? (second ? i - half : i + half) : i ^ 1), c = cs[pr], s = cs[half + pr];
+      v = second ? fmaf(v, c, o * s) : fmaf(v, c, -o * s);
     }
     if (hv < heads) qfull[(t * heads + hv) * krow + kv_rank + i] = v;
     else stx<AT>(dst, kv_rank + i, v);
@@ -204,16 +207,16 @@ head_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx_, int x_
 
 int latent_prep(bool f32, const void* qkv, int64_t ld, const float* norm_w, const int32_t* positions, const int32_t* slots,
                 const float* rot, int rot_dims, int64_t max_pos, float* qfull, void* cache, int T, int heads, int dim, int rot_dim,
-                int kv_rank, float eps, cudaStream_t s) {
+                int kv_rank, float eps, cudaStream_t s, bool half_layout) {
   if (T == 0) return B200_OK;
   B200_REQUIRE(rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0, B200_ERR_INVALID, "latent_prep: %d of %d dimensions rotate",
                rot_dims, rot_dim);
   if (f32)
     B200_CUDA(launch(latent_prep_kernel<float>, dim3(T), dim3(128), (size_t)0, s, (const float*)qkv, ld, norm_w, positions, slots, rot,
-                     rot ? rot_dims : 0, max_pos, qfull, (float*)cache, heads, dim, rot_dim, kv_rank, eps));
+                     rot ? rot_dims : 0, max_pos, qfull, (float*)cache, heads, dim, rot_dim, kv_rank, eps, half_layout ? 1 : 0));
   else
     B200_CUDA(launch(latent_prep_kernel<__nv_bfloat16>, dim3(T), dim3(128), (size_t)0, s, (const __nv_bfloat16*)qkv, ld, norm_w, positions,
-                     slots, rot, rot ? rot_dims : 0, max_pos, qfull, (__nv_bfloat16*)cache, heads, dim, rot_dim, kv_rank, eps));
+                     slots, rot, rot ? rot_dims : 0, max_pos, qfull, (__nv_bfloat16*)cache, heads, dim, rot_dim, kv_rank, eps, half_layout ? 1 : 0));
   return B200_OK;
 }
 

@@ -1,0 +1,186 @@
+// Real-gated linear recurrent unit (B200_MIXER_LRU), per channel c of one sequence:
+//   r = sigmoid(R u + br)_c,  i = sigmoid(I u + bi)_c              (R, I block-diagonal: head_linear gives the products in fp32)
+//   a = exp(-r d_c),   S_t = a S_(t-1) + sqrt(1 - a^2) i u_t,   out_t = S_t gelu_tanh(y_t)
+// u: convolved inputs, y: the other branch's projection, both of the activation type; gates, decays and S fp32.
+//
+//  * step kernel (every sequence brings one row): a thread per channel; the state is read ahead of the dependency wait.
+//  * scan kernel: the recurrence is linear, so a run of rows acts on the state as S -> A S + B.  A CTA takes 16 channels of one
+//    sequence and walks it in tiles of 32 segments x kLruRows rows: a thread folds its segment of one channel into (A, B), one warp
+//    per channel scans the 32 pairs with shuffles and hands every segment the state ahead of it, and the threads run their rows once
+//    more from there.  The next tile's inputs are requested before the barriers of this one.
+// A sequence whose first row of the step is at position 0 starts from zeros, whatever the slot held.
+#include <algorithm>
+
+#include "common.cuh"
+
+namespace b200 {
+namespace {
+
+__device__ __forceinline__ float ldf(float v) { return v; }
+__device__ __forceinline__ float ldf(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void stf(float* p, int64_t i, float v) { p[i] = v; }
+__device__ __forceinline__ void stf(__nv_bfloat16* p, int64_t i, float v) { p[i] = __float2bfloat16_rn(v); }
+
+// One row of one channel, with z the decay gate's and g the input gate's logit: m = 1 - a and b = sqrt(1 - a^2) i u, 1 - a^2 = m (2 - m).
+// The decays of a long memory are close to one; they are carried as m = 1 - e^-h, which keeps its relative precision there, and the
+// state moves by S += b - m S: a decay that is off by a rounding would be off the same way at every row of the context.
+// 32-bit mode: the library's functions.  Serving mode: the hardware's exponential and reciprocal (fp32, a few units in the last
+// place), and for small h the Taylor series of 1 - e^-h.
+template <typename AT>
+__device__ __forceinline__ void lru_terms(float z, float g, float d, float u, float& m, float& b) {
+  if constexpr (sizeof(AT) == 4) {
+    const float r = 1.0f / (1.0f + expf(-z)), i = 1.0f / (1.0f + expf(-g));
+    m = -expm1f(-r * d);
+    b = sqrtf(m * (2.0f - m)) * i * u;
+  } else {
+    const float r = __fdividef(1.0f, 1.0f + __expf(-z)), i = __fdividef(1.0f, 1.0f + __expf(-g)), h = r * d;
+    const float series = h * fmaf(h, fmaf(h, fmaf(h, fmaf(h, fmaf(h, -1.0f / 720.0f, 1.0f / 120.0f), -1.0f / 24.0f), 1.0f / 6.0f), -0.5f), 1.0f);
+    m = h < 0.25f ? series : 1.0f - __expf(-h);
+    b = sqrtf(m * (2.0f - m)) * i * u;
+  }
+}
+__device__ __forceinline__ float lru_move(float S, float m, float b) { return S + fmaf(-m, S, b); }
+
+// gelu_tanh(y); 0.5 (1 + tanh(w)) = 1 / (1 + e^-2w)
+template <typename AT>
+__device__ __forceinline__ float branch_gelu(float y) {
+  if constexpr (sizeof(AT) == 4) return act_apply(y, B200_ACT_GELU_TANH);
+  else return __fdividef(y, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * y * y, y, y)));
+}
+
+template <typename AT>
+struct LruArgs {
+  const AT* u;
+  const float *gates, *gate_bias, *decay;
+  const AT* y;
+  int64_t ldy;
+  const int32_t *positions, *seq_start, *seq_slots;
+  float* state;
+  int64_t slot_stride;
+  AT* out;
+  int width, block;
+};
+
+constexpr int kStepThreads = 128;
+template <typename AT>
+__global__ void __launch_bounds__(kStepThreads)
+lru_step_kernel(const LruArgs<AT> p) {
+  const int64_t t = blockIdx.x;
+  const int c = blockIdx.y * kStepThreads + threadIdx.x;
+  if (c >= p.width) {
+    pdl_wait();
+    return;
+  }
+  const int ir = 2 * (c / p.block) * p.block + c % p.block, ii = ir + p.block;   // this channel's rows among the gates
+  float* st = p.state + (int64_t)p.seq_slots[t] * p.slot_stride + c;
+  const float S0 = p.positions[t] == 0 ? 0.f : *st, d = p.decay[c], br = p.gate_bias[ir], bi = p.gate_bias[ii];
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* g = p.gates + t * 2 * p.width;
+  float m, b;
+  lru_terms<AT>(g[ir] + br, g[ii] + bi, d, ldf(p.u[t * p.width + c]), m, b);
+  const float S = lru_move(S0, m, b);
+  *st = S;
+  stf(p.out, t * p.width + c, S * branch_gelu<AT>(ldf(p.y[t * p.ldy + c])));
+}
+
+constexpr int kLruCh = 16, kLruSegs = 32, kLruRows = 4, kLruThreads = kLruCh * kLruSegs;
+template <typename AT>
+__global__ void __launch_bounds__(kLruThreads)
+lru_scan_kernel(const LruArgs<AT> p) {
+  __shared__ float2 ab[kLruCh][kLruSegs + 1];
+  __shared__ float sin_[kLruCh][kLruSegs + 1];
+  const int s = blockIdx.x, ch = threadIdx.x % kLruCh, seg = threadIdx.x / kLruCh, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.y * kLruCh + ch, cc = min(c, p.width - 1);
+  const bool live = c < p.width;
+  const int start = p.seq_start[s], n_rows = p.seq_start[s + 1] - start;
+  if (n_rows <= 0) {
+    pdl_wait();
+    return;
+  }
+  const int ir = 2 * (cc / p.block) * p.block + cc % p.block, ii = ir + p.block;
+  const float d = p.decay[cc], br = p.gate_bias[ir], bi = p.gate_bias[ii];
+  // warp w carries channel w of the tile from tile to tile
+  const int wc = blockIdx.y * kLruCh + warp;
+  float* st = p.state + (int64_t)p.seq_slots[s] * p.slot_stride + min(wc, p.width - 1);
+  float carry = p.positions[start] == 0 ? 0.f : *st;
+  pdl_wait();
+  pdl_launch_dependents();
+  constexpr int kTile = kLruSegs * kLruRows;
+  float zr[kLruRows], zi[kLruRows];
+  AT ur[kLruRows], yr[kLruRows];
+  auto fetch = [&](int b0) {   // rows past the end are read at the last one and dropped below
+#pragma unroll
+    for (int k = 0; k < kLruRows; ++k) {
+      const int64_t t = start + min(b0 + seg * kLruRows + k, n_rows - 1);
+      zr[k] = p.gates[t * 2 * p.width + ir];
+      zi[k] = p.gates[t * 2 * p.width + ii];
+      ur[k] = p.u[t * p.width + cc];
+      yr[k] = p.y[t * p.ldy + cc];
+    }
+  };
+  fetch(0);
+  for (int b0 = 0; b0 < n_rows; b0 += kTile) {
+    float m[kLruRows], b[kLruRows], y[kLruRows], A = 1.0f, B = 0.f;
+    const int r0 = b0 + seg * kLruRows;
+#pragma unroll
+    for (int k = 0; k < kLruRows; ++k) {
+      lru_terms<AT>(zr[k] + br, zi[k] + bi, d, ldf(ur[k]), m[k], b[k]);
+      if (r0 + k >= n_rows) m[k] = b[k] = 0.f;
+      y[k] = ldf(yr[k]);
+      A = fmaf(-m[k], A, A);
+      B = lru_move(B, m[k], b[k]);
+    }
+    if (b0 + kTile < n_rows) fetch(b0 + kTile);
+    ab[ch][seg] = make_float2(A, B);
+    __syncthreads();
+    {
+      float2 f = ab[warp][lane];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {   // inclusive: the map of segments 0 .. lane
+        const float pa = __shfl_up_sync(0xffffffffu, f.x, o), pb = __shfl_up_sync(0xffffffffu, f.y, o);
+        if (lane >= o) {
+          f.y = fmaf(f.x, pb, f.y);
+          f.x *= pa;
+        }
+      }
+      const float after = fmaf(f.x, carry, f.y), before = __shfl_up_sync(0xffffffffu, after, 1);
+      sin_[warp][lane] = lane == 0 ? carry : before;
+      carry = __shfl_sync(0xffffffffu, after, 31);
+    }
+    __syncthreads();
+    float S = sin_[ch][seg];
+#pragma unroll
+    for (int k = 0; k < kLruRows; ++k) {
+      S = lru_move(S, m[k], b[k]);
+      if (live && r0 + k < n_rows) stf(p.out, (int64_t)(start + r0 + k) * p.width + c, S * branch_gelu<AT>(y[k]));
+    }
+  }
+  if (lane == 0 && wc < p.width) *st = carry;
+}
+
+template <typename AT>
+int gated_lru_t(const LruArgs<AT>& a, int S, bool one_row, cudaStream_t s) {
+  if (one_row) B200_CUDA(launch(lru_step_kernel<AT>, dim3(S, (a.width + kStepThreads - 1) / kStepThreads), dim3(kStepThreads), (size_t)0, s, a));
+  else B200_CUDA(launch(lru_scan_kernel<AT>, dim3(S, (a.width + kLruCh - 1) / kLruCh), dim3(kLruThreads), (size_t)0, s, a));
+  return B200_OK;
+}
+
+}  // namespace
+
+int gated_lru(bool f32, const void* u, const float* gates, const float* gate_bias, const float* decay, const void* y, int64_t ldy,
+              const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state, int64_t slot_stride, void* out, int S,
+              int width, int blocks, bool one_row, cudaStream_t s) {
+  if (S == 0) return B200_OK;
+  B200_REQUIRE(width > 0 && blocks > 0 && width % blocks == 0, B200_ERR_INVALID, "gated_lru: %d channels in %d parts", width, blocks);
+  if (f32) {
+    LruArgs<float> a = {(const float*)u, gates, gate_bias, decay, (const float*)y, ldy, positions, seq_start, seq_slots, state, slot_stride, (float*)out,
+                        width, width / blocks};
+    return gated_lru_t<float>(a, S, one_row, s);
+  }
+  LruArgs<__nv_bfloat16> a = {(const __nv_bfloat16*)u, gates, gate_bias, decay, (const __nv_bfloat16*)y, ldy, positions, seq_start, seq_slots, state,
+                              slot_stride, (__nv_bfloat16*)out, width, width / blocks};
+  return gated_lru_t<__nv_bfloat16>(a, S, one_row, s);
+}
+
+}  // namespace b200

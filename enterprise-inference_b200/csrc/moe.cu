@@ -14,6 +14,8 @@
 //  * tensor-core form (bf16 serving mode, width and ff multiples of 8; every step size): the (token, slot) pairs are
 //    grouped by expert into whole token tiles, the token rows gathered, and two launches of the grouped tcgen05 linear
 //    (gemm_tc.cu) run gate|up and down for all experts at once; the second one scatters the weighted fp32 rows.
+// Score mode 1 scores every expert with the sigmoid of its logit.  RouteForm: a group may count by the sum of its two largest choice
+// scores, the chosen weights may be divided by their sum, and one more router row may gate a shared expert (its sigmoid per token).
 // Score mode 2 (chosen-softmax router): the bias is part of the logits, the `top` largest logits win and the mixing weights are
 // the softmax over those `top` logits alone.  Experts may also be gated by B200_ACT_SWIGLU_CLAMP (gate_combine, common.cuh).
 // All write one fp32 partial row per (token, slot), already multiplied by the mixing weight; the consumer (the norm that
@@ -50,7 +52,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 // One warp: softmax over the logits in sc[experts] (replaced by the scores), choice scores in ch, the group limit, top-k.
 __device__ __forceinline__ void route_select(float* sc, float* ch, float* gs, const float* __restrict__ bias, int lane, int t,
                                              int experts, int top, int groups, int keep, int32_t* __restrict__ out_ids,
-                                             float* __restrict__ out_w, int sigmoid_scores) {
+                                             float* __restrict__ out_w, int sigmoid_scores, const RouteForm& rf) {
   if (sigmoid_scores == 2) {   // the logits themselves compete; the weights follow the choice
     for (int e = lane; e < experts; e += 32) {
       const float z = sc[e] + (bias ? bias[e] : 0.f);
@@ -81,9 +83,12 @@ __device__ __forceinline__ void route_select(float* sc, float* ch, float* gs, co
   if (groups > 1 && keep < groups) {
     const int per = experts / groups;
     for (int g = lane; g < groups; g += 32) {
-      float b = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, ch[e]);
-      gs[g] = b;
+      float b = -INFINITY, b2 = -INFINITY;   // the largest and the next
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        b2 = fmaxf(b2, fminf(b, ch[e]));
+        b = fmaxf(b, ch[e]);
+      }
+      gs[g] = rf.group_best >= 2 && per > 1 ? b + b2 : b;
     }
     __syncwarp();
     // drop the groups - keep worst groups: pick the keep best, mark them, then mask the rest
@@ -140,13 +145,23 @@ __device__ __forceinline__ void route_select(float* sc, float* ch, float* gs, co
     const float inv = 1.0f / sum;
     for (int k = 0; k < top; ++k) w[k] *= inv;
   }
+  if (rf.renorm) {
+    // lane 0 wrote the chosen weights itself
+    if (lane == 0) {
+      float* w = out_w + (int64_t)t * top;
+      float sum = 0.f;
+      for (int k = 0; k < top; ++k) sum += w[k];
+      const float inv = 1.0f / (sum + 1e-20f);
+      for (int k = 0; k < top; ++k) w[k] *= inv;
+    }
+  }
 }
 
 // Selection over logits that a linear already produced ([T][experts] fp32): one warp per token.
 constexpr int kSelWarps = 4;
 __global__ void __launch_bounds__(kSelWarps * 32)
 moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int experts, int top, int groups,
-                  int keep, int32_t* __restrict__ out_ids, float* __restrict__ out_w, int sigmoid_scores) {
+                  int keep, int32_t* __restrict__ out_ids, float* __restrict__ out_w, int sigmoid_scores, RouteForm rf) {
   extern __shared__ float sm[];
   pdl_wait();
   pdl_launch_dependents();
@@ -156,16 +171,18 @@ moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ bi
   float* sc = sm + (size_t)warp * (2 * experts + groups);
   float* ch = sc + experts;
   float* gs = ch + experts;
-  for (int e = lane; e < experts; e += 32) sc[e] = logits[(int64_t)t * experts + e];
+  const int ld = experts + (rf.gate_out ? 1 : 0);
+  for (int e = lane; e < experts; e += 32) sc[e] = logits[(int64_t)t * ld + e];
+  if (rf.gate_out && lane == 0) rf.gate_out[t] = 1.0f / (1.0f + expf(-logits[(int64_t)t * ld + experts]));
   __syncwarp();
-  route_select(sc, ch, gs, bias, lane, t, experts, top, groups, keep, out_ids, out_w, sigmoid_scores);
+  route_select(sc, ch, gs, bias, lane, t, experts, top, groups, keep, out_ids, out_w, sigmoid_scores, rf);
 }
 
 template <typename AT>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(const AT* __restrict__ x, const __nv_bfloat16* __restrict__ wr, const float* __restrict__ bias, int width,
                  int experts, int top, int groups, int keep, int32_t* __restrict__ out_ids, float* __restrict__ out_w,
-                 int sigmoid_scores) {
+                 int sigmoid_scores, RouteForm rf) {
   extern __shared__ float sm[];
   float* xs = sm;                 // [width]
   float* sc = xs + width;         // [experts] scores
@@ -176,16 +193,19 @@ moe_route_kernel(const AT* __restrict__ x, const __nv_bfloat16* __restrict__ wr,
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = kRouteThreads / 32;
   for (int c = threadIdx.x; c < width; c += kRouteThreads) xs[c] = ld_act<AT>(x, (int64_t)t * width + c);
   __syncthreads();
-  for (int e = warp; e < experts; e += nw) {
+  for (int e = warp; e < experts + (rf.gate_out ? 1 : 0); e += nw) {
     const __nv_bfloat16* w = wr + (int64_t)e * width;
     float a = 0.f;
     for (int c = lane; c < width; c += 32) a = fmaf(__bfloat162float(w[c]), xs[c], a);
     a = warp_sum(a);
-    if (lane == 0) sc[e] = a;
+    if (lane == 0) {
+      if (e < experts) sc[e] = a;
+      else rf.gate_out[t] = 1.0f / (1.0f + expf(-a));
+    }
   }
   __syncthreads();
   if (warp != 0) return;
-  route_select(sc, ch, gs, bias, lane, t, experts, top, groups, keep, out_ids, out_w, sigmoid_scores);
+  route_select(sc, ch, gs, bias, lane, t, experts, top, groups, keep, out_ids, out_w, sigmoid_scores, rf);
 }
 
 // ---- token form ---------------------------------------------------------------------------------------------------------
@@ -509,10 +529,8 @@ static int moe_experts_tc(const __nv_bfloat16* x, const __nv_bfloat16* w_gu, con
   int rc;
   static const int fuse_env = getenv("B200_MOE_FUSE_SILU") ? atoi(getenv("B200_MOE_FUSE_SILU")) : 1;
   if (!form.gated) {
-    // one projection, activated in place
-    rc = linear_tc_grouped(xg, width, N, n_tiles, w_gu, experts, ff, width, tile_expert, act, ff, nullptr, nullptr, nullptr, s);
-    if (rc) return rc;
-    rc = ff_act(false, act, act, (int)rows, ff, false, form.act, s);
+    // one projection, activated in the epilogue (on the fp32 sums)
+    rc = linear_tc_grouped(xg, width, N, n_tiles, w_gu, experts, ff, width, tile_expert, act, ff, nullptr, nullptr, nullptr, s, form.act);
     if (rc) return rc;
   } else if (form.act == B200_ACT_SWIGLU_CLAMP && fuse_env && ff % 64 == 0 && (N <= 64 || fuse_env > 1)) {
     // the clamped gate in the same epilogue (it sees the bf16-rounded gate and up values the separate kernel would read)
@@ -540,8 +558,8 @@ static int moe_experts_tc(const __nv_bfloat16* x, const __nv_bfloat16* w_gu, con
 
 int moe_route(bool f32, const void* x, const __nv_bfloat16* w_router, const float* bias, int T, int width, int experts, int top,
               int groups, int keep, int32_t* out_ids, float* out_w, cudaStream_t s, float* logits_ws, void* lin_ws,
-              int64_t lin_ws_bytes, int score_mode) {
-  const int sg = score_mode;
+              int64_t lin_ws_bytes, int score_mode, RouteForm rf) {
+  const int sg = score_mode, n_rows = experts + (rf.gate_out ? 1 : 0);   // rows of the router's matrix
   if (T == 0) return B200_OK;
   B200_REQUIRE(experts > 0 && top > 0 && top <= experts, B200_ERR_INVALID, "router: top %d of %d experts", top, experts);
   if (groups < 1) groups = 1;
@@ -550,17 +568,17 @@ int moe_route(bool f32, const void* x, const __nv_bfloat16* w_router, const floa
   static const int tc_env = getenv("B200_STACK_TC") ? atoi(getenv("B200_STACK_TC")) : 1;
   const size_t smem_sel = (size_t)kSelWarps * (2 * experts + groups) * 4;
   if (!f32 && tc_env && logits_ws && width % 8 == 0 && reinterpret_cast<uintptr_t>(w_router) % 16 == 0 && smem_sel <= 48 * 1024 &&
-      linear_tc_supported(T, experts, width) && (lin_ws == nullptr || linear_tc_workspace_bytes(T, experts, width) <= lin_ws_bytes)) {
+      linear_tc_supported(T, n_rows, width) && (lin_ws == nullptr || linear_tc_workspace_bytes(T, n_rows, width) <= lin_ws_bytes)) {
     // bf16 rows: the logits are a tcgen05 linear with unrounded fp32 output (bf16 products are exact in fp32, the sum is
     // fp32), then one warp per token selects
     LinearExtra ex;
     ex.mode = 4;
     ex.out_f32 = logits_ws;
-    const int rc = linear_tc((const __nv_bfloat16*)x, width, w_router, nullptr, nullptr, experts, T, experts, width, lin_ws,
+    const int rc = linear_tc((const __nv_bfloat16*)x, width, w_router, nullptr, nullptr, n_rows, T, n_rows, width, lin_ws,
                              lin_ws_bytes, &ex, s);
     if (rc) return rc;
     B200_CUDA(launch(moe_select_kernel, dim3((T + kSelWarps - 1) / kSelWarps), dim3(kSelWarps * 32), smem_sel, s,
-                     (const float*)logits_ws, bias, T, experts, top, groups, keep, out_ids, out_w, sg));
+                     (const float*)logits_ws, bias, T, experts, top, groups, keep, out_ids, out_w, sg, rf));
     return B200_OK;
   }
   const size_t smem = ((size_t)width + 2 * experts + groups) * 4;
@@ -569,11 +587,11 @@ int moe_route(bool f32, const void* x, const __nv_bfloat16* w_router, const floa
   if (f32) {
     if (smem > 48 * 1024) B200_CUDA(ensure_dynamic_smem(moe_route_kernel<float>, 200 * 1024, done[0]));
     B200_CUDA(launch(moe_route_kernel<float>, dim3(T), dim3(kRouteThreads), smem, s, (const float*)x, w_router, bias, width, experts,
-                     top, groups, keep, out_ids, out_w, sg));
+                     top, groups, keep, out_ids, out_w, sg, rf));
   } else {
     if (smem > 48 * 1024) B200_CUDA(ensure_dynamic_smem(moe_route_kernel<__nv_bfloat16>, 200 * 1024, done[1]));
     B200_CUDA(launch(moe_route_kernel<__nv_bfloat16>, dim3(T), dim3(kRouteThreads), smem, s, (const __nv_bfloat16*)x, w_router,
-                     bias, width, experts, top, groups, keep, out_ids, out_w, sg));
+                     bias, width, experts, top, groups, keep, out_ids, out_w, sg, rf));
   }
   return B200_OK;
 }

@@ -4,7 +4,7 @@
 //  * conv_inputs: causal per-channel convolutions over the fused projection rows q | k | v | x.  A thread owns V channels and walks a
 //    run of rows with the earlier inputs in registers, so every input is fetched once; ahead of a portion's first row they come from
 //    the sequence's tails in its state slot.  q, k, v: no activation; q leaves as fp32 rows, k and v go to the paged caches.
-//    x: bias and silu, rows of the activation type (they are also the input of the scan's projection).  In a step whose
+//    x: bias and silu (or no activation), rows of the activation type (they are also the input of the scan's projection).  In a step whose
 //    sequences bring one row each (decode) the thread that read a channel's tail also shifts it.
 //  * selective_scan: per channel c and state n   S = exp(dt_c A[c][n]) S + dt_c x_c B_n;   y_c = sum_n S[c][n] C_n + D_c x_c;
 //    out_c = y_c silu(z_c), dt = softplus(dt_pre + bias).  Channels and states do not interact except through the sum over n, so a
@@ -57,7 +57,7 @@ struct ConvArgs {
   const int32_t *positions, *row_to_seq, *seq_start, *seq_slots, *slots;
   float* qout;
   AT *kc, *vc, *xc;
-  int T, heads, kv_heads, dim, vdim, inner, block_size, one_row, run, blocks_a;
+  int T, heads, kv_heads, dim, vdim, inner, block_size, one_row, run, blocks_a, silu_x;
 };
 
 // TAPS > 0: known at compile time, earlier inputs in registers; 0: any count, earlier inputs re-read
@@ -143,8 +143,10 @@ __device__ __forceinline__ void conv_walk(const ConvArgs<AT>& a, bool is_x, int 
       }
     }
     if (is_x) {
+      if (a.silu_x) {
 #pragma unroll
-      for (int v = 0; v < V; ++v) acc[v] = silu_f(acc[v]);
+        for (int v = 0; v < V; ++v) acc[v] = silu_f(acc[v]);
+      }
       stv<AT, V>(a.xc, (int64_t)t * a.inner + c, acc);
     } else if (c < nq) {
       stv<float, V>(a.qout, (int64_t)t * nq + c, acc);
@@ -496,7 +498,7 @@ int selective_scan_t(const SelArgs<AT>& a, int S, bool one, cudaStream_t s) {
 int conv_inputs(bool f32, const void* fused, int64_t ld, const float* conv_a, int taps_a, float* tails_a, const float* conv_x, const float* bias_x,
                 int taps_x, float* tails_x, int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
                 const int32_t* seq_slots, const int32_t* slots, float* qout, void* kc, void* vc, void* xc, int T, int heads, int kv_heads,
-                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s) {
+                int dim, int vdim, int inner, int block_size, bool one_row, cudaStream_t s, bool silu_x) {
   if (T == 0) return B200_OK;
   B200_REQUIRE(taps_a <= 1 || (conv_a && tails_a && seq_slots), B200_ERR_INVALID, "conv_inputs: the q/k/v convolution needs its weights and tails");
   B200_REQUIRE(inner == 0 || (taps_x >= 1 && conv_x && xc && (taps_x == 1 || (tails_x && seq_slots))), B200_ERR_INVALID,
@@ -505,12 +507,12 @@ int conv_inputs(bool f32, const void* fused, int64_t ld, const float* conv_a, in
   if (f32) {
     ConvArgs<float> a = {(const float*)fused, ld, conv_a, conv_x, bias_x, tails_a, tails_x, taps_a, taps_x, slot_stride, positions, row_to_seq, seq_start,
                          seq_slots, slots, qout, (float*)kc, (float*)vc, (float*)xc, T, heads, kv_heads, dim, vdim, inner, block_size,
-                         one_row ? 1 : 0, 1, 0};
+                         one_row ? 1 : 0, 1, 0, silu_x ? 1 : 0};
     return conv_inputs_t<float>(a, s);
   }
   ConvArgs<__nv_bfloat16> a = {(const __nv_bfloat16*)fused, ld, conv_a, conv_x, bias_x, tails_a, tails_x, taps_a, taps_x, slot_stride, positions, row_to_seq,
                                seq_start, seq_slots, slots, qout, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, (__nv_bfloat16*)xc, T, heads, kv_heads, dim,
-                               vdim, inner, block_size, one_row ? 1 : 0, 1, 0};
+                               vdim, inner, block_size, one_row ? 1 : 0, 1, 0, silu_x ? 1 : 0};
   return conv_inputs_t<__nv_bfloat16>(a, s);
 }
 

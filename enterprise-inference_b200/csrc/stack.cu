@@ -18,6 +18,10 @@
 //               recurrence over the state slot;  ff(h2): dense gated, or routed experts + shared expert
 //               X_{i+1} = u + (mixer + ff);  u = sum_j dwa[j] X_j;  norms of the next layer      one kernel
 //   logit rows: u[rows] / rms * g -> W_head -> fp32 logits -> soft cap -> fp32 and bf16 copies -> argmax
+//   norm_kind B200_NORM_TANH: h = tanh(alpha x) w + b feeds both sublayers; the closing sum and the next layer's h are one elementwise
+//   launch (tanh_close).  Attention mixer of this kind: fused q | k | v (| x | y of the recurrent unit) with biases -> whole-projection
+//   norms, k and v into the paged cache -> windowed attention with kept first keys, distance bias and sink -> W_o; beside it
+//   x -> convolution -> block-diagonal gates -> recurrence over the state slot, times gelu(y) -> W_o'
 //
 // Post-norm form (b200_stack_cfg.form = B200_FORM_POSTNORM), same step entry, cache, state slots and graph replay:
 //   x = table[id]                                                         fp32 residual stream (bf16 copy for the linears)
@@ -85,6 +89,9 @@ struct StackLayerW {
   // looped form (tail2_off: the convolution tail of the second mixer, rec_off: the state of the retention or of the selective scan)
   const float *loop_step = nullptr, *dist_bias = nullptr, *decay = nullptr, *side_conv = nullptr, *side_conv_b = nullptr, *side_dt_b = nullptr,
               *side_a = nullptr, *side_skip = nullptr, *out_main = nullptr, *out_side = nullptr;
+  // parallel form with the elementwise norm
+  const float *norm_alpha = nullptr, *side_gates_b = nullptr, *side_decay = nullptr;
+  const __nv_bfloat16* side_gates = nullptr;
   const __nv_bfloat16 *qkv_b = nullptr, *side_proj = nullptr, *side_dt = nullptr, *side_o = nullptr, *mlp_up_b = nullptr, *mlp_down_b = nullptr;
 };
 
@@ -132,6 +139,9 @@ struct StackModel {
   const float* embed_norm = nullptr;
   float *eout = nullptr, *dtp = nullptr;                   // embedding output; step sizes ahead of bias and softplus
   void *xc = nullptr, *xp = nullptr, *ssy = nullptr;       // convolved channels, dt | B | C, gated scan output
+  // parallel form with the elementwise norm
+  const float* final_alpha = nullptr;
+  float *lru_gates = nullptr, *shared_gate = nullptr;      // gate products of the recurrent unit; the shared expert's gate per row
   void* ret_ws = nullptr;                                  // chunk states of the retention
   int64_t ret_ws_bytes = 0;
 };
@@ -143,7 +153,9 @@ static bool is_mlstm(const b200_stack_layer& L) { return L.mixer == B200_MIXER_M
 static bool is_delta(const b200_stack_layer& L) { return L.mixer == B200_MIXER_DELTA; }
 static bool is_ssd(const b200_stack_layer& L) { return L.mixer == B200_MIXER_SSD; }
 static bool is_retention(const b200_stack_layer& L) { return L.mixer == B200_MIXER_RETENTION; }
-static bool has_side(const b200_stack_layer& L) { return L.side == B200_MIXER_SELECTIVE; }
+static bool has_scan(const b200_stack_layer& L) { return L.side == B200_MIXER_SELECTIVE; }
+static bool has_lru(const b200_stack_layer& L) { return L.side == B200_MIXER_LRU; }
+static bool has_side(const b200_stack_layer& L) { return has_scan(L) || has_lru(L); }
 static bool head_decay(const b200_stack_layer& L) { return (L.mixer_flags & B200_MIXF_HEAD_DECAY) != 0; }
 
 // bf16 mode, keys and values of 64 to 128 dimensions in blocks of 128 tokens: the tcgen05 attention kernels of the fixed
@@ -172,7 +184,7 @@ static int64_t up(int64_t v, int64_t a) { return (v + a - 1) / a * a; }
 static int attn_channels(const b200_stack_layer& L) { return L.heads * L.dim + L.kv_heads * (L.dim + L.vdim); }
 static int qkv_rows(const b200_stack_layer& L) {
   if (is_retention(L)) return 2 * L.heads * (L.dim + L.vdim);                                  // q | k | v | gate
-  if (has_side(L))                                                                             // q | k | v | x | z | head gates
+  if (has_side(L))                                                                             // q | k | v | x | z (or y) | head gates
     return attn_channels(L) + 2 * L.side_inner + ((L.mixer_flags & B200_MIXF_HEAD_GATE) ? L.heads : 0);
   if (is_ssd(L)) return 2 * L.heads * L.vdim + 2 * L.kv_heads * L.dim + L.heads;             // z | x | B | C | dt
   if (is_delta(L) && head_decay(L)) return 2 * L.kv_heads * L.dim + 2 * L.heads * L.vdim + 2 * L.heads;   // q | k | v | gate | b | a
@@ -244,6 +256,8 @@ static int stack_gate_up(b200_ctx* c, const void* x, const StackLayerW& W, const
 static int stack_ready_parallel(const b200_ctx* c) {
   const StackModel* M = c->stack;
   const b200_stack_cfg& m = M->cfg;
+  const bool tn = m.norm_kind == B200_NORM_TANH;
+  B200_REQUIRE(!tn || (M->final_norm_b && M->final_alpha), B200_ERR_STATE, "step: the output norm is not complete");
   B200_REQUIRE(m.bigram_buckets <= 0 || M->bigram, B200_ERR_STATE, "step: bigram table not set");
   B200_REQUIRE(m.n_state_slots <= 0 || M->state, B200_ERR_STATE, "step: state slots not set");
   for (size_t l = 0; l < M->layers.size(); ++l) {
@@ -258,10 +272,17 @@ static int stack_ready_parallel(const b200_ctx* c) {
       B200_REQUIRE(!(L.mixer_flags & B200_MIXF_SINK) || W.sink, B200_ERR_STATE, "step: layer %d sink missing", li);
       B200_REQUIRE(L.rot_dims == 0 || (L.rot_table >= 0 && M->rot[L.rot_table] && M->rot_half[L.rot_table] * 2 == L.rot_dims),
                    B200_ERR_STATE, "step: layer %d rotation table missing or of another size", li);
+    } else if (L.mixer == B200_MIXER_ATTENTION) {
+      B200_REQUIRE(W.q_norm && W.k_norm && W.kc && W.vc && (!(L.mixer_flags & B200_MIXF_QKV_BIAS) || W.qkv_b) && (L.bias_dist <= 0 || W.dist_bias) &&
+                       (!(L.mixer_flags & B200_MIXF_SINK) || W.sink),
+                   B200_ERR_STATE, "step: layer %d attention weights / cache incomplete", li);
+      B200_REQUIRE(!has_lru(L) || (W.side_conv && W.side_conv_b && W.side_gates && W.side_gates_b && W.side_decay && W.side_o), B200_ERR_STATE,
+                   "step: layer %d weights of its second mixer incomplete", li);
     } else {
       B200_REQUIRE(W.gates && W.head_norm, B200_ERR_STATE, "step: layer %d recurrent weights incomplete", li);
     }
-    if (L.mlp != B200_MLP_NONE) B200_REQUIRE(W.n_mlp_pre, B200_ERR_STATE, "step: layer %d second norm missing", li);
+    B200_REQUIRE(!tn || (W.n_mix_pre_b && W.norm_alpha), B200_ERR_STATE, "step: layer %d norm incomplete", li);
+    if (L.mlp != B200_MLP_NONE && !tn) B200_REQUIRE(W.n_mlp_pre, B200_ERR_STATE, "step: layer %d second norm missing", li);
     if (L.mlp == B200_MLP_DENSE) B200_REQUIRE(W.mlp_gate_up && W.mlp_down, B200_ERR_STATE, "step: layer %d feed-forward weights incomplete", li);
     if (L.mlp == B200_MLP_MOE) {
       B200_REQUIRE(W.router && W.e_gate_up && W.e_down, B200_ERR_STATE, "step: layer %d expert weights incomplete", li);
@@ -579,7 +600,14 @@ static int stack_enqueue_step_parallel(b200_ctx* c, const StepArgs& a, cudaStrea
   if (stateful && m.bigram_buckets > 0)
     STEP(prev_token_commit(a.ids, m.vocab, a.prev_tokens, a.n_prev, M->seq_start, seq_slots, S, st_prev, M->slot_floats, s));
   const bool conv = m.canon_taps >= 1;
+  const bool tn = m.norm_kind == B200_NORM_TANH;   // one elementwise norm per layer, read by both sublayers
+  const bool one_row_each = (a.n_seqs > 0 && a.n_seqs == T) || a.row_to_seq == nullptr;   // known, not assumed
+  void* hm = tn ? M->hn : M->hc;                   // the mixers' input
   // X_0 and the first layer's norms
+  if (tn)
+    STEP(tanh_close(f32, u, nullptr, 0.f, nullptr, 0.f, nullptr, 0, nullptr, nullptr, M->w[0].norm_alpha, M->w[0].n_mix_pre, M->w[0].n_mix_pre_b, M->hn,
+                    nullptr, T, Wd, s));
+  else
   STEP(parallel_close(f32, u, nullptr, nullptr, nullptr, 0, nullptr, m.depth_avg ? M->results : nullptr, rstride, 1, nullptr,
                       M->w[0].n_mix_pre, M->w[0].n_mlp_pre, conv ? M->h1f : nullptr, conv ? nullptr : M->hc, M->hn, T, Wd, m.norm_eps, s));
   for (int l = 0; l < nL; ++l) {
@@ -589,14 +617,55 @@ static int stack_enqueue_step_parallel(b200_ctx* c, const StepArgs& a, cudaStrea
     if (conv)
       STEP(canon_conv(f32, M->h1f, W.canon, M->hc, T, Wd, m.canon_taps, a.positions, a.row_to_seq, M->seq_start, seq_slots,
                       M->state ? M->state + W.tail_off : nullptr, M->slot_floats, s));
-    STEP(stack_linear(c, M->hc, Wd, W.qkv, M->qkv, qr, T, qr, Wd, s));
     const int av = L.heads * L.vdim;
-    if (is_latent(L)) {
+    const void* y_side = nullptr;
+    if (L.mixer_flags & B200_MIXF_QKV_BIAS)
+      STEP(linear_ex(f32, f32, hm, Wd, W.qkv, W.qkv_b, M->qkv, qr, T, qr, Wd, -1, c->lin_ws, c->lin_ws_bytes, s));
+    else
+      STEP(stack_linear(c, hm, Wd, W.qkv, M->qkv, qr, T, qr, Wd, s));
+    if (L.mixer == B200_MIXER_ATTENTION) {
+      const int ch = attn_channels(L), inner = has_lru(L) ? L.side_inner : 0;
+      STEP(qk_norm_cache(f32, M->qkv, qr, W.q_norm, W.k_norm, a.slots, M->q, W.kc, W.vc, T, L.heads, L.kv_heads, L.dim, L.vdim, m.block_size, m.norm_eps,
+                         s));
+      AttnExtra ex;
+      ex.dist_bias = L.bias_dist > 0 ? W.dist_bias : nullptr;
+      ex.bias_dist = L.bias_dist;
+      ex.keep_first = L.window > 0 ? L.keep_first : 0;
+      const float* sink = (L.mixer_flags & B200_MIXF_SINK) ? W.sink : nullptr;
+      if (!f32 && paged_attn_mma_supported(L.heads, L.kv_heads, L.dim, L.vdim)) {
+        STEP(step_runs(runs_built));
+        const int seen = L.window > 0 ? std::min(a.max_ctx, L.window + ex.keep_first + 64) : a.max_ctx;
+        STEP(paged_attn_mma(M->q, (const __nv_bfloat16*)W.kc, (const __nv_bfloat16*)W.vc, a.block_table, a.bt_stride, a.row_to_seq, a.ctx_lens,
+                            (__nv_bfloat16*)M->attn, static_cast<const int32_t*>(M->attn_ws) + 8, static_cast<const int32_t*>(M->attn_ws), T,
+                            L.heads, L.kv_heads, L.dim, L.vdim, m.block_size, L.scale, sink, s,
+                            latent_attn_splits(T, L.heads, L.vdim, seen, M->lat_ws_bytes), M->lat_ws, L.window, ex));
+      } else {
+        if (attn_plan) STEP(step_runs(runs_built));
+        STEP(paged_attn_anydim(f32, M->q, W.kc, W.vc, a.block_table, a.bt_stride, a.row_to_seq, a.ctx_lens, a.positions, nullptr, 1ll << 40,
+                               M->attn, T, L.heads, L.kv_heads, L.dim, L.vdim, m.block_size, L.scale, attn_plan ? 2 : 0, M->attn_ws, s, 0, 0, sink,
+                               L.window, ex));
+      }
+      if (inner) {
+        const char* x_in = static_cast<const char*>(M->qkv) + (int64_t)ch * es;
+        const int blk = inner / L.side_blocks;
+        float* tails = L.side_taps > 1 ? M->state + W.tail2_off : nullptr;
+        STEP(conv_inputs(f32, x_in, qr, nullptr, 0, nullptr, W.side_conv, W.side_conv_b, L.side_taps, tails, M->slot_floats, a.positions, a.row_to_seq,
+                         M->seq_start, seq_slots, nullptr, nullptr, nullptr, nullptr, M->xc, T, 0, 0, 0, 0, inner, m.block_size, one_row_each, s, false));
+        if (!one_row_each && tails)
+          STEP(delta_tails(f32, x_in, qr, a.positions, M->seq_start, seq_slots, tails, M->slot_floats, S, inner, L.side_taps, s));
+        STEP(head_linear(f32, true, M->xc, inner, blk, W.side_gates, M->lru_gates, 2 * (int64_t)inner, 2 * blk, nullptr, 0, 0, T, L.side_blocks, 2 * blk,
+                         blk, s));
+        STEP(gated_lru(f32, M->xc, M->lru_gates, W.side_gates_b, W.side_decay, x_in + (int64_t)inner * es, qr, a.positions, M->seq_start, seq_slots,
+                       M->state + W.rec_off, M->slot_floats, M->ssy, S, inner, L.side_blocks, one_row_each, s));
+        STEP(stack_linear(c, M->ssy, inner, W.side_o, M->y2, Wd, T, Wd, inner, s));
+        y_side = M->y2;
+      }
+    } else if (is_latent(L)) {
       const int qh = L.dim + L.rot_dim, krow = L.kv_rank + L.rot_dim;
       const float* rot = L.rot_dims > 0 ? M->rot[L.rot_table] : nullptr;
       const int64_t max_pos = rot ? M->rot_pos[L.rot_table] : (1ll << 40);
       STEP(latent_prep(f32, M->qkv, qr, W.k_norm, a.positions, a.slots, rot, L.rot_dims, max_pos, M->q, W.kc, T, L.heads, L.dim,
-                       L.rot_dim, L.kv_rank, m.norm_eps, s));
+                       L.rot_dim, L.kv_rank, m.norm_eps, s, (L.mixer_flags & B200_MIXF_ROT_HALF) != 0));
       // q' = W_uk^T q_plain into the leading kv_rank entries of every query row
       STEP(head_linear(f32, true, M->qkv, qr, qh, W.uk_t, M->q, (int64_t)L.heads * krow, krow, nullptr, 0, 0, T, L.heads, L.kv_rank,
                        L.dim, s));
@@ -618,7 +687,7 @@ static int stack_enqueue_step_parallel(b200_ctx* c, const StepArgs& a, cudaStrea
                        L.vdim, T, L.heads, L.vdim, L.kv_rank, s));
     } else {
       const int hd = L.heads * L.dim;
-      STEP(mlstm_gates(f32, M->hc, W.gates, W.gates_bias, M->gates_buf, T, Wd, L.heads, L.gate_cap, s));
+      STEP(mlstm_gates(f32, hm, W.gates, W.gates_bias, M->gates_buf, T, Wd, L.heads, L.gate_cap, s));
       STEP(mlstm_scan(f32, M->qkv, qr, 0, hd, 2 * hd, M->gates_buf, a.positions, M->seq_start, seq_slots, M->state + W.rec_off,
                       M->slot_floats, M->oraw, S, L.heads, L.dim, L.vdim, s, S == T));
       const char* gptr = static_cast<const char*>(M->qkv) + (int64_t)(2 * hd + av) * es;
@@ -633,8 +702,12 @@ static int stack_enqueue_step_parallel(b200_ctx* c, const StepArgs& a, cudaStrea
       STEP(stack_linear(c, M->ffa, L.ff, W.mlp_down, M->y2, Wd, T, Wd, L.ff, s));
       y_ff = M->y2;
     } else if (L.mlp == B200_MLP_MOE) {
+      RouteForm rf;
+      rf.group_best = L.group_best;
+      rf.renorm = L.route_renorm != 0;
+      rf.gate_out = L.shared_gate ? M->shared_gate : nullptr;
       STEP(moe_route(f32, M->hn, W.router, W.router_bias, T, Wd, L.experts, L.top, L.groups, L.keep, M->route_ids, M->route_w, s,
-                     M->route_logits, c->lin_ws, c->lin_ws_bytes, L.sigmoid_scores != 0));
+                     M->route_logits, c->lin_ws, c->lin_ws_bytes, L.sigmoid_scores != 0, rf));
       ExpertForm form;
       form.gated = !L.ungated;
       form.act = L.act;
@@ -644,20 +717,37 @@ static int stack_enqueue_step_parallel(b200_ctx* c, const StepArgs& a, cudaStrea
       parts = M->parts;
       n_parts = L.top;
       if (L.shared_ff > 0) {
-        const int sr = (L.ungated ? 1 : 2) * L.shared_ff;
-        STEP(stack_linear(c, M->hn, Wd, W.shared_up, M->gu, sr, T, sr, Wd, s));
-        STEP(ff_act(f32, M->gu, M->ffa, T, L.shared_ff, !L.ungated, L.act, s));
+        if (L.ungated) {   // activated in the epilogue
+          STEP(linear_ex(f32, f32, M->hn, Wd, W.shared_up, nullptr, M->ffa, L.shared_ff, T, L.shared_ff, Wd, L.act, c->lin_ws, c->lin_ws_bytes, s));
+        } else {
+          STEP(stack_linear(c, M->hn, Wd, W.shared_up, M->gu, 2 * L.shared_ff, T, 2 * L.shared_ff, Wd, s));
+          STEP(ff_act(f32, M->gu, M->ffa, T, L.shared_ff, true, L.act, s));
+        }
         STEP(stack_linear(c, M->ffa, L.shared_ff, W.shared_down, M->y3, Wd, T, Wd, L.shared_ff, s));
         y_sh = M->y3;
       }
     }
     const bool last = l + 1 == nL;
+    if (tn) {
+      const float sa = y_side ? L.mix_main : 1.0f;
+      const float* gate = L.shared_gate ? M->shared_gate : nullptr;
+      if (!last || M->tap)
+        STEP(tanh_close(f32, u, M->y, sa, y_side, L.mix_side, parts, n_parts, y_sh, gate, last ? nullptr : M->w[l + 1].norm_alpha,
+                        last ? nullptr : M->w[l + 1].n_mix_pre, last ? nullptr : M->w[l + 1].n_mix_pre_b, last ? nullptr : M->hn, nullptr, T, Wd, s));
+      // logit rows: the last close and the output norm over those rows only
+      if (last && M->tap)
+        STEP(tanh_close(f32, u, nullptr, 0.f, nullptr, 0.f, nullptr, 0, nullptr, nullptr, M->final_alpha, M->final_norm, M->final_norm_b, M->lm_in,
+                        a.logit_rows, a.R, Wd, s));
+      else if (last)
+        STEP(tanh_close(f32, u, M->y, sa, y_side, L.mix_side, parts, n_parts, y_sh, gate, M->final_alpha, M->final_norm, M->final_norm_b, M->lm_in,
+                        a.logit_rows, a.R, Wd, s));
+    } else
     STEP(parallel_close(f32, u, M->y, y_ff, parts, n_parts, y_sh, m.depth_avg ? M->results : nullptr, rstride, l + 2,
                         m.depth_avg ? W.dwa : nullptr, last ? nullptr : M->w[l + 1].n_mix_pre, last ? nullptr : M->w[l + 1].n_mlp_pre,
                         conv ? M->h1f : nullptr, conv ? nullptr : M->hc, M->hn, T, Wd, m.norm_eps, s));
     if (M->tap) B200_CUDA(cudaMemcpyAsync(M->tap + (int64_t)l * T * Wd, u, (size_t)T * Wd * 4, cudaMemcpyDeviceToDevice, s));
   }
-  STEP(rms_rows(f32, u, a.logit_rows, M->final_norm, M->lm_in, a.R, Wd, m.norm_eps, s));
+  if (!tn) STEP(rms_rows(f32, u, a.logit_rows, M->final_norm, M->lm_in, a.R, Wd, m.norm_eps, s));
   STEP(stack_logits_f32(c, a, m.logit_softcap, s));
 #undef STEP
   return B200_OK;
@@ -1041,25 +1131,43 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
                    cfg->max_blocks_per_seq > 0 && cfg->max_logit_rows > 0,
                B200_ERR_INVALID, "stack_create: bad sizes");
   int max_qkv = 0, max_q = 0, max_a = 0, max_top = 0, max_exp = 0, max_ff = 0, max_lat = 0, max_gates = 0, max_gu = 0, max_ffa = 0;
-  int max_qrank = 0, max_qh = 0, max_dhd = 0, max_dqk = 0, max_dav = 0, max_dh = 0, max_heads = 0, max_inner = 0, max_proj = 0;
+  int max_qrank = 0, max_qh = 0, max_dhd = 0, max_dqk = 0, max_dav = 0, max_dh = 0, max_heads = 0, max_inner = 0, max_proj = 0, max_lru = 0;
   int64_t moe_ws_bytes = 16;
   for (int l = 0; l < cfg->n_layers; ++l) {
     const b200_stack_layer& L = layers[l];
     if (cfg->form == B200_FORM_PARALLEL) {
-      B200_REQUIRE(L.mixer == B200_MIXER_LATENT || L.mixer == B200_MIXER_MLSTM, B200_ERR_UNSUPPORTED,
+      const bool tn = cfg->norm_kind == B200_NORM_TANH;
+      B200_REQUIRE(L.mixer == B200_MIXER_LATENT || L.mixer == B200_MIXER_MLSTM || (tn && L.mixer == B200_MIXER_ATTENTION), B200_ERR_UNSUPPORTED,
                    "stack_create: layer %d: mixer %d is not served in the parallel form", l, L.mixer);
+      B200_REQUIRE(!tn || (!cfg->canon_taps && !cfg->depth_avg && !cfg->bigram_buckets), B200_ERR_UNSUPPORTED,
+                   "stack_create: input convolution, depth average and bigram rows come with RMS norms");
+      B200_REQUIRE(!tn || L.mlp != B200_MLP_DENSE, B200_ERR_UNSUPPORTED, "stack_create: layer %d: dense feed-forwards come with RMS norms", l);
+      B200_REQUIRE(tn || (!L.side && !L.group_best && !L.route_renorm && !L.shared_gate), B200_ERR_UNSUPPORTED,
+                   "stack_create: layer %d: a second mixer and these router options come with the elementwise norm", l);
+      if (L.mixer == B200_MIXER_ATTENTION) {
+        B200_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0 && L.rot_dims == 0 && L.vrot_table < 0 && L.window >= 0 && L.keep_first >= 0 &&
+                         L.bias_dist >= 0 && L.softcap == 0.f &&
+                         !(L.mixer_flags & ~(B200_MIXF_SINK | B200_MIXF_QKV_BIAS)),
+                     B200_ERR_INVALID, "stack_create: layer %d: bad attention sizes or flags", l);
+        B200_REQUIRE(L.side == 0 || has_lru(L), B200_ERR_UNSUPPORTED, "stack_create: layer %d: second mixer %d", l, L.side);
+        B200_REQUIRE(!has_lru(L) || (L.side_inner > 0 && L.side_blocks > 0 && L.side_inner % L.side_blocks == 0 && L.side_taps >= 1 && L.side_taps <= 64 &&
+                                     cfg->n_state_slots > 0),
+                     B200_ERR_INVALID, "stack_create: layer %d: bad sizes of the recurrent unit (or no state slots)", l);
+        if (has_lru(L)) max_inner = std::max(max_inner, L.side_inner), max_lru = std::max(max_lru, L.side_inner);
+      }
       B200_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0, B200_ERR_INVALID, "stack_create: layer %d: bad mixer sizes", l);
       if (L.mixer == B200_MIXER_LATENT)
         B200_REQUIRE(L.kv_rank > 0 && L.rot_dim >= 0 && L.rot_dims >= 0 && L.rot_dims <= L.rot_dim && L.rot_dims % 2 == 0 &&
                          L.rot_table < 16 && L.kv_rank <= 512,
                      B200_ERR_INVALID, "stack_create: layer %d: bad latent sizes", l);
-      else
+      else if (L.mixer == B200_MIXER_MLSTM)
         B200_REQUIRE(L.gate_cap > 0.f && L.dim <= 256 && cfg->n_state_slots > 0, B200_ERR_INVALID,
                      "stack_create: layer %d: bad recurrent sizes (or no state slots)", l);
       B200_REQUIRE(L.mlp == B200_MLP_NONE || L.mlp == B200_MLP_MOE || L.mlp == B200_MLP_DENSE, B200_ERR_UNSUPPORTED,
                    "stack_create: layer %d: unknown feed-forward %d", l, L.mlp);
-      B200_REQUIRE(L.mlp == B200_MLP_NONE || (L.ff > 0 && L.act >= 0 && L.act <= B200_ACT_RELU && L.shared_ff >= 0), B200_ERR_INVALID,
-                   "stack_create: layer %d: bad feed-forward sizes", l);
+      B200_REQUIRE(L.mlp == B200_MLP_NONE || (L.ff > 0 && L.act >= 0 && (L.act <= B200_ACT_RELU || L.act == B200_ACT_GELU_ERF) && L.shared_ff >= 0),
+                   B200_ERR_INVALID, "stack_create: layer %d: bad feed-forward sizes", l);
+      B200_REQUIRE(!L.shared_gate || (L.mlp == B200_MLP_MOE && L.shared_ff > 0), B200_ERR_INVALID, "stack_create: layer %d: no shared expert to gate", l);
     } else if (cfg->form == B200_FORM_POSTNORM) {
       B200_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0 && L.window >= 0, B200_ERR_INVALID, "stack_create: layer %d: bad mixer sizes", l);
       if (L.mixer == B200_MIXER_ATTENTION) {
@@ -1123,7 +1231,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
                      B200_ERR_UNSUPPORTED, "stack_create: layer %d: mixer %d is not served in the looped form", l, L.mixer);
         B200_REQUIRE(L.rot_dims == 0 && L.conv_taps >= 0 && L.conv_taps <= 64 && L.softcap >= 0.f && L.bias_dist >= 0, B200_ERR_INVALID,
                      "stack_create: layer %d: bad attention sizes", l);
-        B200_REQUIRE(L.side == 0 || has_side(L), B200_ERR_UNSUPPORTED, "stack_create: layer %d: second mixer %d", l, L.side);
+        B200_REQUIRE(L.side == 0 || has_scan(L), B200_ERR_UNSUPPORTED, "stack_create: layer %d: second mixer %d", l, L.side);
         B200_REQUIRE(!has_side(L) || (L.side_inner > 0 && L.side_state > 0 && L.side_state <= 256 && L.side_rank > 0 && L.side_taps >= 1 && L.side_taps <= 64),
                      B200_ERR_INVALID, "stack_create: layer %d: bad sizes of the selective scan", l);
       }
@@ -1184,7 +1292,8 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
   M->w.resize(cfg->n_layers);
   M->esz = cfg->f32 ? 4 : 2;
   if (par && cfg->n_state_slots > 0) {
-    // one slot: [previous token (int32) + padding to 4 floats | per layer: convolution tail [taps - 1][width], recurrent state]
+    // one slot: [previous token (int32) + padding to 4 floats | per layer: convolution tail [taps - 1][width], recurrent state (a second mixer's
+    // tail and state likewise)]
     int64_t off = 4;
     for (int l = 0; l < cfg->n_layers; ++l) {
       if (cfg->canon_taps > 1) {
@@ -1194,6 +1303,12 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       if (is_mlstm(layers[l])) {
         M->w[l].rec_off = off;
         off += mlstm_state_floats(layers[l].heads, layers[l].dim, layers[l].vdim);
+      }
+      if (has_lru(layers[l])) {   // the convolution's tail, then the recurrence's state
+        M->w[l].tail2_off = off = up(off, 4);
+        off = up(off + (int64_t)(layers[l].side_taps - 1) * layers[l].side_inner, 4);
+        M->w[l].rec_off = off;
+        off += layers[l].side_inner;
       }
       off = up(off, 4);
     }
@@ -1290,7 +1405,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
     for (int l = 0; l < cfg->n_layers; ++l) {
       shapes.push_back({qkv_rows(layers[l]), (int)Wd});
       shapes.push_back({(int)Wd, layers[l].heads * layers[l].vdim});
-      if (layers[l].mlp == B200_MLP_MOE) shapes.push_back({layers[l].experts, (int)Wd});
+      if (layers[l].mlp == B200_MLP_MOE) shapes.push_back({layers[l].experts + (layers[l].shared_gate ? 1 : 0), (int)Wd});
       if (layers[l].mlp == B200_MLP_DENSE) {
         shapes.push_back({(layers[l].ungated ? 1 : 2) * layers[l].ff, (int)Wd});
         shapes.push_back({(int)Wd, layers[l].ff});
@@ -1299,7 +1414,8 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
         shapes.push_back({(layers[l].ungated ? 1 : 2) * layers[l].shared_ff, (int)Wd});
         shapes.push_back({(int)Wd, layers[l].shared_ff});
       }
-      if (has_side(layers[l])) {
+      if (has_lru(layers[l])) shapes.push_back({(int)Wd, layers[l].side_inner});
+      if (has_scan(layers[l])) {
         shapes.push_back({selective_rows(layers[l].side_rank, layers[l].side_state), layers[l].side_inner});
         shapes.push_back({layers[l].side_inner, selective_dt_pad(layers[l].side_rank)});
         shapes.push_back({(int)Wd, layers[l].side_inner});
@@ -1352,7 +1468,7 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       if (is_retention(layers[l]) && retention_chunk_supported(layers[l].dim, layers[l].vdim))
         M->ret_ws_bytes = std::max<int64_t>(M->ret_ws_bytes, retention_chunk_workspace_bytes((int)T, (int)std::min<int64_t>(T, cfg->n_state_slots), layers[l].heads,
                                                                                              layers[l].dim, layers[l].vdim));
-  if ((post || hyp || loop) && !cfg->f32)
+  if ((par || post || hyp || loop) && !cfg->f32)
     for (int l = 0; l < cfg->n_layers; ++l)
       if (layers[l].mixer == B200_MIXER_ATTENTION && paged_attn_mma_supported(layers[l].heads, layers[l].kv_heads, layers[l].dim, layers[l].vdim))
         M->lat_ws_bytes = std::max<int64_t>(M->lat_ws_bytes, std::min<int64_t>(T * layers[l].heads, 148 * 16) * 16 * (layers[l].vdim + 2) * 4);
@@ -1370,7 +1486,9 @@ extern "C" int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_lay
       {(void**)&M->route_ids, T * std::max(max_top, 1) * 4},
       {(void**)&M->route_w, T * std::max(max_top, 1) * 4},
       {(void**)&M->parts, T * std::max(max_top, 1) * Wd * 4},
-      {(void**)&M->route_logits, T * std::max(max_exp, 1) * 4},
+      {(void**)&M->route_logits, T * (max_exp + 1) * 4},
+      {(void**)&M->shared_gate, T * 4},
+      {(void**)&M->lru_gates, T * 2 * (int64_t)max_lru * 4},
       {(void**)&M->lm_in, R * Wd * es},
       {(void**)&M->attn_ws, attn_ws_bytes},
       {(void**)&M->moe_ws, moe_ws_bytes},
@@ -1444,18 +1562,18 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
   StackModel* M = c->stack;
   const int64_t Wd = M->cfg.width, V = M->cfg.vocab;
   int64_t er = 0, ec = 1;
-  const bool par = M->cfg.form == B200_FORM_PARALLEL;
+  const bool par = M->cfg.form == B200_FORM_PARALLEL, tn = par && M->cfg.norm_kind == B200_NORM_TANH;
   const bool post = M->cfg.form == B200_FORM_POSTNORM;
   const bool hyp = M->cfg.form == B200_FORM_HYPER;
   const bool global = kind == B200_SW_EMBED || kind == B200_SW_FINAL_NORM || kind == B200_SW_HEAD || kind == B200_SW_BIGRAM ||
-                      kind == B200_SW_FINAL_NORM_BIAS || kind == B200_SW_EMBED_NORM;
+                      kind == B200_SW_FINAL_NORM_BIAS || kind == B200_SW_EMBED_NORM || kind == B200_SW_FINAL_NORM_ALPHA;
   const bool loop = M->cfg.form == B200_FORM_LOOPED;
   if (!global) B200_REQUIRE(layer >= 0 && layer < M->cfg.n_layers, B200_ERR_INVALID, "stack_set_weight: layer %d out of range", layer);
   const b200_stack_layer L = global ? b200_stack_layer{} : M->layers[layer];
   switch (kind) {
     case B200_SW_EMBED: case B200_SW_HEAD: er = V; ec = Wd; break;
     case B200_SW_FINAL_NORM: case B200_SW_NORM_MIX_PRE: case B200_SW_NORM_MIX_POST: case B200_SW_NORM_MLP_PRE:
-    case B200_SW_NORM_MLP_POST: er = par ? 1 : Wd; break;
+    case B200_SW_NORM_MLP_POST: er = par && !tn ? 1 : Wd; break;
     case B200_SW_QKV: er = qkv_rows(L); ec = Wd; break;
     case B200_SW_Q_NORM: er = (L.mixer_flags & B200_MIXF_HEAD_NORM) ? L.dim : (int64_t)L.heads * L.dim; break;
     case B200_SW_K_NORM: er = is_latent(L) ? L.kv_rank : ((L.mixer_flags & B200_MIXF_HEAD_NORM) ? L.dim : (int64_t)L.kv_heads * L.dim); break;
@@ -1473,6 +1591,10 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_SIDE_A: er = L.side_inner; ec = L.side_state; break;
     case B200_SW_SIDE_O: er = Wd; ec = L.side_inner; break;
     case B200_SW_MLP_UP_BIAS: er = L.ff; break;
+    case B200_SW_NORM_ALPHA: case B200_SW_FINAL_NORM_ALPHA: er = 1; break;
+    case B200_SW_SIDE_GATES: er = 2 * (int64_t)L.side_inner; ec = L.side_blocks > 0 ? L.side_inner / L.side_blocks : 0; break;
+    case B200_SW_SIDE_GATES_BIAS: er = 2 * (int64_t)L.side_inner; break;
+    case B200_SW_SIDE_DECAY: er = L.side_inner; break;
     case B200_SW_CONV:
       if (L.mixer == B200_MIXER_ATTENTION) {
         er = attn_channels(L), ec = L.conv_taps;
@@ -1490,7 +1612,7 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_DECAY_LOG: er = L.heads; break;
     case B200_SW_GATE_UP: er = (int64_t)L.heads * L.vdim; ec = L.gate_rank; break;
     case B200_SW_O: er = Wd; ec = (int64_t)L.heads * L.vdim; break;
-    case B200_SW_ROUTER: er = L.experts; ec = Wd; break;
+    case B200_SW_ROUTER: er = L.experts + (L.shared_gate ? 1 : 0); ec = Wd; break;
     case B200_SW_ROUTER_BIAS: er = L.experts; break;
     case B200_SW_EXPERT_GATE_UP: er = (int64_t)L.experts * (L.ungated ? 1 : 2) * L.ff; ec = Wd; break;
     case B200_SW_EXPERT_DOWN: er = (int64_t)L.experts * Wd; ec = L.ff; break;
@@ -1510,8 +1632,18 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_SHARED_DOWN: er = Wd; ec = L.shared_ff; break;
     default: B200_REQUIRE(false, B200_ERR_INVALID, "stack_set_weight: unknown kind %d", kind);
   }
-  B200_REQUIRE(kind < B200_SW_EMBED_NORM || loop, B200_ERR_INVALID, "stack_set_weight: kind %d belongs to the looped form", kind);
-  if (loop) {
+  // the elementwise norm's form takes kinds of several others
+  const bool tn_side = kind == B200_SW_SIDE_CONV || kind == B200_SW_SIDE_CONV_BIAS || kind == B200_SW_SIDE_O ||
+                       (kind >= B200_SW_SIDE_GATES && kind <= B200_SW_SIDE_DECAY);
+  const bool tn_attn = kind == B200_SW_QKV_BIAS || kind == B200_SW_DIST_BIAS || kind == B200_SW_Q_NORM;
+  const bool tn_kind = tn && (tn_side || tn_attn || kind == B200_SW_NORM_MIX_PRE_BIAS || kind == B200_SW_FINAL_NORM_BIAS || kind == B200_SW_NORM_ALPHA ||
+                              kind == B200_SW_FINAL_NORM_ALPHA);
+  B200_REQUIRE(kind < B200_SW_NORM_ALPHA || tn, B200_ERR_INVALID, "stack_set_weight: kind %d belongs to the parallel form with the elementwise norm", kind);
+  B200_REQUIRE(kind < B200_SW_EMBED_NORM || loop || tn_kind, B200_ERR_INVALID, "stack_set_weight: kind %d belongs to the looped form", kind);
+  if (tn_kind) {
+    B200_REQUIRE(!tn_side || has_lru(L), B200_ERR_INVALID, "stack_set_weight: layer %d has no second mixer", layer);
+    B200_REQUIRE(!tn_attn || L.mixer == B200_MIXER_ATTENTION, B200_ERR_INVALID, "stack_set_weight: layer %d has no attention", layer);
+  } else if (loop) {
     const bool dense = kind == B200_SW_MLP_GATE_UP || kind == B200_SW_MLP_DOWN || kind == B200_SW_MLP_UP_BIAS || kind == B200_SW_MLP_DOWN_BIAS;
     const bool side = (kind >= B200_SW_SIDE_CONV && kind <= B200_SW_OUT_SIDE);
     B200_REQUIRE(kind <= B200_SW_QKV || kind == B200_SW_O || kind >= B200_SW_EMBED_NORM || dense || kind == B200_SW_CONV, B200_ERR_INVALID,
@@ -1624,6 +1756,11 @@ extern "C" int b200_stack_set_weight(b200_ctx* c, int32_t layer, int32_t kind, c
     case B200_SW_OUT_SIDE: M->w[layer].out_side = f; break;
     case B200_SW_MLP_UP_BIAS: M->w[layer].mlp_up_b = b; break;
     case B200_SW_MLP_DOWN_BIAS: M->w[layer].mlp_down_b = b; break;
+    case B200_SW_NORM_ALPHA: M->w[layer].norm_alpha = f; break;
+    case B200_SW_FINAL_NORM_ALPHA: M->final_alpha = f; break;
+    case B200_SW_SIDE_GATES: M->w[layer].side_gates = b; break;
+    case B200_SW_SIDE_GATES_BIAS: M->w[layer].side_gates_b = f; break;
+    case B200_SW_SIDE_DECAY: M->w[layer].side_decay = f; break;
   }
   return B200_OK;
 }
@@ -2188,8 +2325,88 @@ extern "C" int b200_paged_attn_biased(int32_t f32, int32_t form, const float* q,
 
 extern "C" int b200_linear_bias_act(int32_t f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy, int32_t T,
                                     int32_t n_out, int32_t k, int32_t act, void* ws, int64_t ws_bytes, void* stream) {
-  B200_REQUIRE(x && w && y && T >= 0 && n_out > 0 && k > 0 && act <= B200_ACT_RELU, B200_ERR_INVALID, "linear_bias_act: bad argument");
+  B200_REQUIRE(x && w && y && T >= 0 && n_out > 0 && k > 0 && (act <= B200_ACT_RELU || act == B200_ACT_GELU_ERF), B200_ERR_INVALID, "linear_bias_act: bad argument");
   if (T == 0) return B200_OK;
   return linear_ex(f32 != 0, y_f32 != 0 || f32 != 0, x, ldx, (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias, y, ldy, T, n_out, k, act, ws, ws_bytes,
                    (cudaStream_t)stream);
+}
+
+// ---- per-kernel entry points of the parallel form with the elementwise norm ------------------------------------------------------
+extern "C" int b200_tanh_close(int32_t f32, float* x, const void* ya, float sa, const void* yb, float sb, const float* parts, int32_t n_parts,
+                               const void* y_sh, const float* sh_gate, const float* alpha, const float* w, const float* b, void* out,
+                               const int32_t* rows, int32_t R, int32_t width, void* stream) {
+  B200_REQUIRE(x && width > 0 && R >= 0 && n_parts >= 0, B200_ERR_INVALID, "tanh_close: bad argument");
+  return tanh_close(f32 != 0, x, ya, sa, yb, sb, parts, n_parts, y_sh, sh_gate, alpha, w, b, out, rows, R, width, (cudaStream_t)stream);
+}
+
+extern "C" int b200_qk_norm_cache(int32_t f32, const void* fused, int64_t ld, const float* qw, const float* kw, const int32_t* slots, float* q_out,
+                                  void* kc, void* vc, int32_t T, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t block_size,
+                                  float eps, void* stream) {
+  B200_REQUIRE(fused && qw && kw && slots && q_out && kc && vc && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && block_size > 0, B200_ERR_INVALID,
+               "qk_norm_cache: bad argument");
+  return qk_norm_cache(f32 != 0, fused, ld, qw, kw, slots, q_out, kc, vc, T, heads, kv_heads, dim, vdim, block_size, eps, (cudaStream_t)stream);
+}
+
+extern "C" int b200_side_conv(int32_t f32, const void* x, int64_t ld, const float* conv, const float* bias, int32_t taps, float* tails,
+                              int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
+                              const int32_t* seq_slots, void* out, int32_t T, int32_t S, int32_t width, int32_t one_row, void* stream) {
+  B200_REQUIRE(x && conv && out && positions && seq_start && seq_slots && width > 0 && taps >= 1 && (taps == 1 || tails), B200_ERR_INVALID,
+               "side_conv: bad argument");
+  cudaStream_t s = (cudaStream_t)stream;
+  int rc = conv_inputs(f32 != 0, x, ld, nullptr, 0, nullptr, conv, bias, taps, tails, slot_stride, positions, row_to_seq, seq_start, seq_slots, nullptr,
+                       nullptr, nullptr, nullptr, out, T, 0, 0, 0, 0, width, 1, one_row != 0, s, false);
+  if (rc || one_row || taps == 1) return rc;
+  return delta_tails(f32 != 0, x, ld, positions, seq_start, seq_slots, tails, slot_stride, S, width, taps, s);
+}
+
+extern "C" int b200_gated_lru(int32_t f32, const void* u, const float* gates, const float* gate_bias, const float* decay, const void* y, int64_t ldy,
+                              const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state, int64_t slot_stride,
+                              void* out, int32_t S, int32_t width, int32_t blocks, int32_t one_row, void* stream) {
+  B200_REQUIRE(u && gates && gate_bias && decay && y && positions && seq_start && seq_slots && state && out, B200_ERR_INVALID, "gated_lru: null argument");
+  return gated_lru(f32 != 0, u, gates, gate_bias, decay, y, ldy, positions, seq_start, seq_slots, state, slot_stride, out, S, width, blocks, one_row != 0,
+                   (cudaStream_t)stream);
+}
+
+extern "C" int b200_latent_prep_half(int32_t f32, const void* qkv, int64_t ld, const float* norm_w, const int32_t* positions, const int32_t* slots,
+                                     const float* rot, int32_t rot_dims, int64_t max_pos, float* qfull, void* cache, int32_t T, int32_t heads,
+                                     int32_t dim, int32_t rot_dim, int32_t kv_rank, float eps, void* stream) {
+  B200_REQUIRE(qkv && norm_w && positions && slots && qfull && cache && heads > 0 && kv_rank > 0 && max_pos > 0, B200_ERR_INVALID,
+               "latent_prep_half: bad argument");
+  return latent_prep(f32 != 0, qkv, ld, norm_w, positions, slots, rot, rot_dims, max_pos, qfull, cache, T, heads, dim, rot_dim, kv_rank, eps,
+                     (cudaStream_t)stream, true);
+}
+
+extern "C" int b200_moe_route_form(int32_t f32, const void* x, const void* w_router, const float* bias, int32_t T, int32_t width, int32_t experts,
+                                   int32_t top, int32_t groups, int32_t keep, int32_t group_best, int32_t renorm, float* gate_out, float* logits,
+                                   int32_t* out_ids, float* out_w, void* stream) {
+  B200_REQUIRE(x && w_router && out_ids && out_w && width > 0, B200_ERR_INVALID, "moe_route_form: bad argument");
+  RouteForm rf;
+  rf.group_best = group_best;
+  rf.renorm = renorm != 0;
+  rf.gate_out = gate_out;
+  return moe_route(f32 != 0, x, (const __nv_bfloat16*)w_router, bias, T, width, experts, top, groups, keep, out_ids, out_w, (cudaStream_t)stream, logits,
+                   nullptr, 0, 1, rf);
+}
+
+extern "C" int b200_paged_attn_kept(int32_t f32, int32_t form, const float* q, const void* kc, const void* vc, const int32_t* block_table,
+                                    int32_t bt_stride, const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, void* out,
+                                    int32_t T, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t block_size, float scale,
+                                    int32_t window, int32_t keep_first, const float* sink, const float* dist_bias, int32_t bias_dist, void* ws,
+                                    int32_t n_splits, float* part, void* stream) {
+  B200_REQUIRE(q && kc && vc && block_table && ctx_lens && positions && out && block_size > 0 && window >= 0 && keep_first >= 0 &&
+                   (!dist_bias || bias_dist > 0) && (form == 0 || ws) && form >= 0 && form <= 2,
+               B200_ERR_INVALID, "paged_attn_kept: bad argument");
+  AttnExtra ex;
+  ex.dist_bias = dist_bias, ex.bias_dist = bias_dist, ex.keep_first = window > 0 ? keep_first : 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (form == 2) {
+    B200_REQUIRE(!f32, B200_ERR_UNSUPPORTED, "paged_attn_kept: the tensor-core form takes bf16 caches");
+    int rc = paged_attn_runs_plan(row_to_seq, ctx_lens, T, ws, s);
+    if (rc) return rc;
+    return paged_attn_mma(q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, block_table, bt_stride, row_to_seq, ctx_lens, (__nv_bfloat16*)out,
+                          static_cast<const int32_t*>(ws) + 8, static_cast<const int32_t*>(ws), T, heads, kv_heads, dim, vdim, block_size, scale, sink, s,
+                          n_splits, part, window, ex);
+  }
+  return paged_attn_anydim(f32 != 0, q, kc, vc, block_table, bt_stride, row_to_seq, ctx_lens, positions, nullptr, 1ll << 40, out, T, heads, kv_heads, dim,
+                           vdim, block_size, scale, form, ws, s, 0, 0, sink, window, ex);
 }

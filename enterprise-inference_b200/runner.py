@@ -440,13 +440,15 @@ class StackRunner(ModelRunner):
             return keys[k]
 
         from .config import (AttentionSpec, BofusunConfig, ChannelDeltaSpec, DupolornConfig, FutidraConfig, HeadDeltaSpec, MLSTMSpec, RetentionSpec,
-                             RudolixConfig, StateSpaceSpec, distance_entries)
-        self.parallel = isinstance(cfg, DupolornConfig)
+                             RirusunConfig, RudolixConfig, StateSpaceSpec, distance_entries)
+        self.tanh_norm = isinstance(cfg, RirusunConfig)   # the parallel form with one elementwise norm per layer
+        self.parallel = isinstance(cfg, DupolornConfig) or self.tanh_norm
         self.postnorm = isinstance(cfg, FutidraConfig)
         self.hyper = isinstance(cfg, RudolixConfig)
         self.looped = isinstance(cfg, BofusunConfig)
         # what runs, in order: a looped layer once per pass, each run with its own cache and state
-        runs = cfg.layer_runs() if self.looped else [(i, None) for i in range(len(cfg.layers))]
+        self.unrolled = hasattr(cfg, "layer_runs")
+        runs = cfg.layer_runs() if self.unrolled else [(i, None) for i in range(len(cfg.layers))]
         self.run_layers = [cfg.layers[i] for i, _ in runs]
         # dense feed-forwards of the post-norm form in bf16: gate activation and product in the gate|up linear's epilogue
         self.fuse_gate_up = self.postnorm and not self.f32 and os.environ.get("B200_STACK_FUSE_GATE_UP", "1") != "0"
@@ -523,15 +525,25 @@ class StackRunner(ModelRunner):
             if isinstance(a, MLSTMSpec):
                 d = dict(mixer=_abi.MIXER_MLSTM, heads=a.heads, kv_heads=a.heads, dim=a.dim, vdim=a.vdim, rot_table=-1, vrot_table=-1,
                          gate_cap=a.gate_cap)
+            elif isinstance(a, AttentionSpec):
+                flags = (_abi.MIXF_SINK if a.sink else 0) | (_abi.MIXF_QKV_BIAS if L.side is not None else 0)
+                d = dict(mixer=_abi.MIXER_ATTENTION, heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, rot_table=-1, vrot_table=-1,
+                         scale=a.scale, mixer_flags=flags, window=a.window, keep_first=a.keep_first,
+                         bias_dist=distance_entries(a.window, a.bias_max, a.keep_first) if a.bias_max > 0 else 0)
+                if L.side is not None:
+                    s = L.side
+                    d.update(side=_abi.MIXER_LRU, side_inner=s.inner, side_taps=s.conv, side_blocks=s.blocks, mix_main=L.side_mix[0],
+                             mix_side=L.side_mix[1])
             else:
                 d = dict(mixer=_abi.MIXER_LATENT, heads=a.heads, kv_heads=1, dim=a.dim, vdim=a.vdim, rot_dims=a.rot.dims if a.rot else 0,
                          rot_table=table_of(a.rot), vrot_table=-1, scale=a.scale, kv_rank=a.kv_rank, rot_dim=a.rot_dim,
-                         mixer_flags=(_abi.MIXF_SINK if a.sink else 0) | (_abi.MIXF_GATE if a.gate else 0))
+                         mixer_flags=(_abi.MIXF_SINK if a.sink else 0) | (_abi.MIXF_GATE if a.gate else 0) | (_abi.MIXF_ROT_HALF if a.rot_half else 0))
             if f is not None and f.kind == "dense":
                 d.update(mlp=_abi.MLP_DENSE, ff=f.ff, act=_abi.ACTS[f.act])
             elif f is not None:
-                d.update(mlp=_abi.MLP_MOE, experts=f.experts, top=f.top, groups=1, keep=1, ff=f.ff, act=_abi.ACTS[f.act], ungated=1,
-                         sigmoid_scores=1, weight_input=1, shared_ff=f.shared_ff)
+                d.update(mlp=_abi.MLP_MOE, experts=f.experts, top=f.top, groups=f.groups, keep=f.keep, ff=f.ff, act=_abi.ACTS[f.act], ungated=1,
+                         sigmoid_scores=1, weight_input=int(f.weight_input), shared_ff=f.shared_ff, shared_gate=int(f.shared_gate),
+                         group_best=f.group_best if self.tanh_norm else 0, route_renorm=int(f.renorm))
             layers[i] = _abi.StackLayer(**d)
         sc = _abi.StackCfg(width=cfg.width, vocab=cfg.vocab, n_layers=cfg.n_layers, embed_scale=cfg.embed_scale,
                            norm_eps=cfg.norm_eps, f32=int(self.f32), block_size=block_size, max_tokens=max_tokens,
@@ -540,6 +552,7 @@ class StackRunner(ModelRunner):
             sc.form, sc.canon_taps, sc.depth_avg = _abi.FORM_PARALLEL, cfg.canon_taps, int(cfg.depth_avg)
             sc.bigram_buckets, sc.bigram_mul_prev, sc.bigram_mul_cur = cfg.bigram_buckets, cfg.bigram_mul_prev, cfg.bigram_mul_cur
             sc.logit_softcap, sc.n_state_slots = cfg.logit_softcap, self.n_state_slots
+            sc.norm_kind = _abi.NORM_TANH if self.tanh_norm else _abi.NORM_RMS
         if self.postnorm:
             sc.form, sc.residual_alpha, sc.n_state_slots = _abi.FORM_POSTNORM, cfg.postln_alpha, self.n_state_slots
         if self.hyper:
@@ -610,7 +623,7 @@ class StackRunner(ModelRunner):
 
     def load_weights(self, w: Dict[str, torch.Tensor]):
         from .weights import STACK_WEIGHT_MAPS
-        self._shared_uploads = {} if self.looped else None   # source tensor -> device tensor: the passes of a looped layer share one upload
+        self._shared_uploads = {} if self.unrolled else None   # source tensor -> device tensor: the passes of a looped layer share one upload
         for layer, kind, t in STACK_WEIGHT_MAPS[self.cfg.architecture](w, self.cfg):
             self._set(layer, kind, t)
         self._shared_uploads = None
@@ -840,6 +853,59 @@ class StackRunner(ModelRunner):
                         self._set(r, kind, t)
         self._shared_uploads = None
 
+    def _init_random_tanh(self, seed: int, std: float):
+        from .config import LatentAttentionSpec, MLSTMSpec, distance_entries
+        c, A = self.cfg, _abi
+        g = torch.Generator(device=self.device)
+        g.manual_seed(seed)
+
+        def rnd(*shape, sd=std):
+            t = torch.empty(shape, dtype=torch.bfloat16, device=self.device)
+            t.normal_(0.0, sd, generator=g)
+            return t
+
+        def full(n, v=1.0):
+            return torch.full((n,), v, device=self.device)
+
+        self._shared_uploads = {}
+        runs = c.layer_runs()
+        self._set(0, A.SW_EMBED, rnd(c.vocab, c.width, sd=1.0))
+        self._set(0, A.SW_FINAL_NORM, full(c.width))
+        self._set(0, A.SW_FINAL_NORM_BIAS, full(c.width, 0.0))
+        self._set(0, A.SW_FINAL_NORM_ALPHA, full(1, 0.5))
+        self._set(0, A.SW_HEAD, rnd(c.vocab, c.width))
+        for i, L in enumerate(c.layers):
+            a, s, f = L.mixer, L.side, L.mlp
+            out = [(A.SW_NORM_MIX_PRE, full(c.width)), (A.SW_NORM_MIX_PRE_BIAS, full(c.width, 0.0)), (A.SW_NORM_ALPHA, full(1, 0.5)),
+                   (A.SW_O, rnd(c.width, a.heads * a.vdim))]
+            if isinstance(a, MLSTMSpec):
+                out += [(A.SW_QKV, rnd(2 * a.heads * (a.dim + a.vdim), c.width)), (A.SW_GATES, rnd(2 * a.heads, c.width)),
+                        (A.SW_GATES_BIAS, torch.cat([full(a.heads, 0.0), full(a.heads, 3.0)])), (A.SW_HEAD_NORM, full(a.heads * a.vdim))]
+            elif isinstance(a, LatentAttentionSpec):
+                out += [(A.SW_QKV, rnd(a.heads * (a.dim + a.rot_dim) + a.kv_rank + a.rot_dim, c.width)), (A.SW_K_NORM, full(a.kv_rank)),
+                        (A.SW_UK_T, rnd(a.heads * a.kv_rank, a.dim, sd=a.kv_rank ** -0.5)), (A.SW_UV, rnd(a.heads * a.vdim, a.kv_rank, sd=a.kv_rank ** -0.5))]
+            else:
+                rows = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + (2 * s.inner if s else 0)
+                out += [(A.SW_QKV, rnd(rows, c.width)), (A.SW_Q_NORM, full(a.heads * a.dim)), (A.SW_K_NORM, full(a.kv_heads * a.dim)),
+                        (A.SW_SINK, full(a.heads, 0.0))]
+                if a.bias_max > 0:
+                    out.append((A.SW_DIST_BIAS, rnd(a.heads, distance_entries(a.window, a.bias_max, a.keep_first), sd=0.5).float()))
+                if s:
+                    blk = s.inner // s.blocks
+                    out += [(A.SW_QKV_BIAS, torch.zeros(rows, device=self.device, dtype=torch.bfloat16)), (A.SW_SIDE_CONV, rnd(s.inner, s.conv, sd=0.5).float()),
+                            (A.SW_SIDE_CONV_BIAS, full(s.inner, 0.0)), (A.SW_SIDE_GATES, rnd(2 * s.inner, blk)), (A.SW_SIDE_GATES_BIAS, full(2 * s.inner, 0.0)),
+                            (A.SW_SIDE_DECAY, full(s.inner, 0.2)), (A.SW_SIDE_O, rnd(c.width, s.inner))]
+            if f is not None:
+                out += [(A.SW_ROUTER, rnd(f.experts + int(f.shared_gate), c.width)), (A.SW_ROUTER_BIAS, full(f.experts, 0.0)),
+                        (A.SW_EXPERT_GATE_UP, rnd(f.experts * f.ff, c.width)), (A.SW_EXPERT_DOWN, rnd(f.experts * c.width, f.ff))]
+                if f.shared_ff > 0:
+                    out += [(A.SW_SHARED_UP, rnd(f.shared_ff, c.width)), (A.SW_SHARED_DOWN, rnd(c.width, f.shared_ff))]
+            for r, (j, _) in enumerate(runs):
+                if j == i:
+                    for kind, t in out:
+                        self._set(r, kind, t)
+        self._shared_uploads = None
+
     def set_step_slots(self, seq_slots: Optional[torch.Tensor]):
         """Device-pointer steps (step_device) of a model with state slots: int32 device tensor, one slot per sequence of the step."""
         self._step_slots = seq_slots
@@ -847,6 +913,8 @@ class StackRunner(ModelRunner):
 
     def init_random_weights(self, seed: int = 1234, std: float = 0.02):
         """Random-init weights generated on the device (benchmarks).  Norm weights are 1, the router bias 0."""
+        if self.tanh_norm:
+            return self._init_random_tanh(seed, std)
         if self.parallel:
             return self._init_random_parallel(seed, std)
         if self.postnorm:

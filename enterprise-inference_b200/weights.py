@@ -352,5 +352,59 @@ def bofusun_weights(w: Dict[str, torch.Tensor], cfg) -> Iterator[Tuple[int, int,
                     yield r, kind, tensor
 
 
+def rirusun_weights(w: Dict[str, torch.Tensor], cfg) -> Iterator[Tuple[int, int, torch.Tensor]]:
+    """(layer RUN, b200_stack_weight kind, tensor) of a Rirusun checkpoint: `embed`, `head`, the output norm `final.norm[.b|.alpha]`, and per
+    layer i the norm `l<i>.norm1[.b|.alpha]`, the mixer `l<i>.mix.*` and the experts `l<i>.mlp.*`.  A looped layer's tensors are yielded once
+    per pass, the same object every time (the runner uploads it once).  Projections of the mixer's input are fused row-wise: latent
+    q | dkv; mLSTM q | k | v | g, and i | f as the gate rows; attention beside a recurrent unit q | k | v | x | y, with biases (zeros for
+    q | k | v).  A latent head's key expansion goes over transposed ([heads][kv_rank][dim]); the distance table is expanded to one entry per
+    distance and head; the unit's gate matrices are stacked per block (decay gate, input gate) and its decays go over as
+    8 softplus(lam); the shared expert's gate row follows the router's rows; experts are stacked [E][ff][width] and [E][width][ff]."""
+    from . import _abi as A
+    from .config import LatentAttentionSpec, MLSTMSpec, distance_bucket, distance_entries
+    runs = cfg.layer_runs()
+    yield 0, A.SW_EMBED, w["embed"]
+    yield 0, A.SW_FINAL_NORM, w["final.norm"]
+    yield 0, A.SW_FINAL_NORM_BIAS, w["final.norm.b"]
+    yield 0, A.SW_FINAL_NORM_ALPHA, w["final.norm.alpha"].reshape(1)
+    yield 0, A.SW_HEAD, w["head"]
+    for i, L in enumerate(cfg.layers):
+        p, a, s, f = f"l{i}.", L.mixer, L.side, L.mlp
+        m = p + "mix."
+        out = [(A.SW_NORM_MIX_PRE, w[p + "norm1"]), (A.SW_NORM_MIX_PRE_BIAS, w[p + "norm1.b"]), (A.SW_NORM_ALPHA, w[p + "norm1.alpha"].reshape(1))]
+        if isinstance(a, MLSTMSpec):
+            out += [(A.SW_QKV, torch.cat([w[m + n] for n in "qkvg"], 0)), (A.SW_GATES, torch.cat([w[m + "i"], w[m + "f"]], 0)),
+                    (A.SW_GATES_BIAS, torch.cat([w[m + "i.b"], w[m + "f.b"]], 0)), (A.SW_HEAD_NORM, w[m + "norm"]), (A.SW_O, w[m + "o"])]
+        elif isinstance(a, LatentAttentionSpec):
+            uk_t = w[m + "uk"].reshape(a.heads, a.dim, a.kv_rank).transpose(1, 2).reshape(a.heads * a.kv_rank, a.dim)
+            out += [(A.SW_QKV, torch.cat([w[m + "q"], w[m + "dkv"]], 0)), (A.SW_K_NORM, w[m + "dkv.norm"]), (A.SW_UK_T, uk_t), (A.SW_UV, w[m + "uv"]),
+                    (A.SW_O, w[m + "o"])]
+        else:
+            l, r = m + "left.", m + "right."
+            rows = [w[l + n] for n in "qkv"] + [w[r + "x"], w[r + "y"]]
+            zeros = torch.zeros(sum(x.shape[0] for x in rows[:3]), dtype=w[r + "x.b"].dtype)
+            rel = w[l + "rel"].float()
+            idx = torch.tensor([distance_bucket(d, rel.shape[0], a.bias_max) for d in range(distance_entries(a.window, a.bias_max, a.keep_first))])
+            blk = s.inner // s.blocks
+            gates = torch.stack([w[r + n].reshape(s.blocks, blk, blk) for n in ("ra", "ri")], 1).reshape(2 * s.inner, blk)
+            gates_b = torch.stack([w[r + n + ".b"].reshape(s.blocks, blk) for n in ("ra", "ri")], 1).reshape(2 * s.inner)
+            out += [(A.SW_QKV, torch.cat(rows, 0)), (A.SW_QKV_BIAS, torch.cat([zeros, w[r + "x.b"], w[r + "y.b"]])), (A.SW_Q_NORM, w[l + "q.norm"]),
+                    (A.SW_K_NORM, w[l + "k.norm"]), (A.SW_SINK, w[l + "sink"]), (A.SW_DIST_BIAS, rel[idx].T.contiguous()), (A.SW_O, w[l + "o"]),
+                    (A.SW_SIDE_CONV, w[r + "conv"]), (A.SW_SIDE_CONV_BIAS, w[r + "conv.b"]), (A.SW_SIDE_GATES, gates), (A.SW_SIDE_GATES_BIAS, gates_b),
+                    (A.SW_SIDE_DECAY, 8.0 * torch.nn.functional.softplus(w[r + "lam"].double())), (A.SW_SIDE_O, w[r + "o"])]
+        if f is not None:
+            e = p + "mlp."
+            out += [(A.SW_ROUTER, torch.cat([w[e + "router"]] + ([w[e + "shared.sg"]] if f.shared_gate else []), 0)),
+                    (A.SW_ROUTER_BIAS, w[e + "correction"]),
+                    (A.SW_EXPERT_GATE_UP, torch.cat([w[f"{e}e{j}.up"] for j in range(f.experts)], 0)),
+                    (A.SW_EXPERT_DOWN, torch.cat([w[f"{e}e{j}.down"] for j in range(f.experts)], 0))]
+            if f.shared_ff > 0:
+                out += [(A.SW_SHARED_UP, w[e + "shared.up"]), (A.SW_SHARED_DOWN, w[e + "shared.down"])]
+        for r, (j, _) in enumerate(runs):
+            if j == i:
+                for kind, tensor in out:
+                    yield r, kind, tensor
+
+
 STACK_WEIGHT_MAPS = {"Bopilorn": bopilorn_weights, "Dupolorn": dupolorn_weights, "Futidra": futidra_weights, "Rudolix": rudolix_weights,
-                     "Bofusun": bofusun_weights}
+                     "Bofusun": bofusun_weights, "Rirusun": rirusun_weights}

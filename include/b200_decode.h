@@ -432,6 +432,20 @@ B200_API int b200_tp_allreduce(b200_ctx* ctx, int32_t buf_idx, const void* parti
  * alone; experts with B200_ACT_SWIGLU_CLAMP: g = min(gate h, act_limit), u = clamp(up h, -act_limit, act_limit),
  * down(g * sigmoid(1.702 g) * (u + 1)).
  *
+ * With norm_kind = B200_NORM_TANH the parallel form has ONE elementwise norm per layer, D(x) = tanh(alpha x) w + b with a scalar alpha,
+ * and both sublayers read its output: x += mixer(h) + ff(h), h = D(x); no input convolution, depth average or bigram rows.  Mixers: the
+ * latent one (B200_MIXF_ROT_HALF: dimension i of the rotated part turns with i + rot_dims / 2), mLSTM, and
+ * B200_MIXER_ATTENTION without rotation: q and k RMS-normalised over the whole projection, window of `window` positions besides the
+ * first `keep_first`, bias by distance, B200_MIXF_SINK.  side = B200_MIXER_LRU: a second mixer reads the same input, and the layer
+ * takes mix_main * first + mix_side * second; the fused rows are q | k | v | x | y (B200_MIXF_QKV_BIAS: with biases).
+ *
+ * B200_MIXER_LRU (real-gated linear recurrent unit): u = conv(x) with side_taps taps and bias; per part of the channels
+ * r = sigmoid(R u + br), i = sigmoid(I u + bi); a = exp(-r d) (d: B200_SW_SIDE_DECAY); S = a S + sqrt(1 - a^2) i u (fp32, per sequence);
+ * result W (S * gelu_tanh(y)).  The last side_taps - 1 inputs of the convolution are state as well.
+ *
+ * Routed experts of this form: sigmoid scores, the bias joins the choice only, groups counted by group_best, route_renorm, weights on the
+ * output (weight_input 0), an optional shared expert with shared_gate.
+ *
  * Fifth layer form (b200_stack_cfg.form = B200_FORM_LOOPED): RMS norms on both sides of every sublayer over one fp32 stream,
  *   x += rms(sublayer(rms(x) * w_pre)) * w_post   (rms(v) = v / sqrt(mean(v^2) + eps); the weights given here are the whole factors),
  * x starting from e = rms(table[id]) * w_embed.  Layers may be run several times: a layer list is given UNROLLED, every pass an entry
@@ -455,12 +469,13 @@ B200_API int b200_tp_allreduce(b200_ctx* ctx, int32_t buf_idx, const void* parti
  *
  * Feed-forward of this form: B200_MLP_DENSE, ungated, act B200_ACT_RELU2, optional biases on both projections. */
 typedef enum b200_mixer_kind { B200_MIXER_ATTENTION = 1, B200_MIXER_LATENT = 2, B200_MIXER_MLSTM = 3, B200_MIXER_DELTA = 4, B200_MIXER_SSD = 5,
-                               B200_MIXER_RETENTION = 6, B200_MIXER_SELECTIVE = 7 } b200_mixer_kind;
+                               B200_MIXER_RETENTION = 6, B200_MIXER_SELECTIVE = 7, B200_MIXER_LRU = 8 } b200_mixer_kind;
 typedef enum b200_mlp_kind { B200_MLP_NONE = 0, B200_MLP_MOE = 1, B200_MLP_DENSE = 2 } b200_mlp_kind;
 typedef enum b200_act_kind { B200_ACT_SILU = 0, B200_ACT_GELU_TANH = 1, B200_ACT_RELU2 = 2, B200_ACT_RELU = 3, B200_ACT_SWIGLU_CLAMP = 4,
-                             B200_ACT_POLYNORM = 5 } b200_act_kind;
+                             B200_ACT_POLYNORM = 5, B200_ACT_GELU_ERF = 6 } b200_act_kind;
 typedef enum b200_stack_form { B200_FORM_SANDWICH = 0, B200_FORM_PARALLEL = 1, B200_FORM_POSTNORM = 2, B200_FORM_HYPER = 3,
                                B200_FORM_LOOPED = 4 } b200_stack_form;
+typedef enum b200_norm_kind { B200_NORM_RMS = 0, B200_NORM_TANH = 1 } b200_norm_kind;
 enum { B200_MIXF_SINK = 1, B200_MIXF_GATE = 2, B200_MIXF_HEAD_NORM = 4, B200_MIXF_VALUE_IS_KEY = 8, B200_MIXF_SINK_ONE = 16,
        B200_MIXF_HEAD_GATE = 32, B200_MIXF_ROT_HALF = 64, B200_MIXF_NO_QK_NORM = 128, B200_MIXF_HEAD_DECAY = 256,
        B200_MIXF_QKV_BIAS = 512 };
@@ -494,9 +509,15 @@ typedef struct b200_stack_layer {
   int32_t route_chosen;                /* router: bias inside the logits, mixing weights = softmax over the chosen logits */
   float softcap;                       /* attention scores: softcap * tanh(score / softcap) (0: none) */
   int32_t bias_dist;                   /* attention: entries per head of the distance bias (0: none) */
-  int32_t side;                        /* second mixer beside the first: 0 or B200_MIXER_SELECTIVE */
-  int32_t side_inner, side_state, side_rank, side_taps;   /* selective scan: channels, states per channel, dt rank, taps */
+  int32_t side;                        /* second mixer beside the first: 0, B200_MIXER_SELECTIVE or B200_MIXER_LRU */
+  int32_t side_inner, side_state, side_rank, side_taps;   /* channels and taps of the second mixer; selective scan: states per channel, dt rank */
   int32_t loop_add, loop_step;         /* looped form: what the stream takes ahead of this entry */
+  int32_t keep_first;                  /* attention with a window: the first positions every query sees besides it */
+  int32_t side_blocks;                 /* B200_MIXER_LRU: equal parts of the channels, each with gate matrices of its own */
+  float mix_main, mix_side;            /* parallel form with a second mixer: factors of the two results */
+  int32_t group_best;                  /* router: a group counts by the sum of this many of its best choice scores (0, 1: its best; 2) */
+  int32_t route_renorm;                /* router: mixing weights are divided by their sum */
+  int32_t shared_gate;                 /* the shared expert's result is scaled by the sigmoid of one more router row */
 } b200_stack_layer;
 
 typedef struct b200_stack_cfg {
@@ -516,6 +537,7 @@ typedef struct b200_stack_cfg {
   float residual_alpha;                /* post-norm form: the stream's factor inside the norm */
   int32_t streams;                     /* multi-stream form: copies of the residual (1 .. B200_MAX_STREAMS) */
   float residual_mult;                 /* multi-stream form: factor of every sublayer's result */
+  int32_t norm_kind;                   /* parallel form: b200_norm_kind */
 } b200_stack_cfg;
 
 typedef enum b200_stack_weight {
@@ -600,7 +622,16 @@ typedef enum b200_stack_weight {
   B200_SW_OUT_MAIN = 62,           /* f32 [width]: norm weights of the two results that are averaged */
   B200_SW_OUT_SIDE = 63,           /* f32 [width] */
   B200_SW_MLP_UP_BIAS = 64,        /* bf16 [ff] */
-  B200_SW_MLP_DOWN_BIAS = 65       /* bf16 [width] */
+  B200_SW_MLP_DOWN_BIAS = 65,      /* bf16 [width] */
+  /* parallel form with B200_NORM_TANH (norm weights and biases: B200_SW_NORM_MIX_PRE[_BIAS], B200_SW_FINAL_NORM[_BIAS], [width] each;
+     attention: B200_SW_Q_NORM, _K_NORM, _SINK, _DIST_BIAS, _QKV_BIAS, _SIDE_CONV[_BIAS], _SIDE_O; with shared_gate B200_SW_ROUTER has
+     experts + 1 rows, the last one the shared expert's gate) */
+  B200_SW_NORM_ALPHA = 66,         /* f32 [1] */
+  B200_SW_FINAL_NORM_ALPHA = 67,   /* f32 [1] */
+  B200_SW_SIDE_GATES = 68,         /* bf16 [side_blocks][2 * block][block], block = side_inner / side_blocks: per part the rows of the decay
+                                      gate, then those of the input gate */
+  B200_SW_SIDE_GATES_BIAS = 69,    /* f32 [2 * side_inner], in the same order */
+  B200_SW_SIDE_DECAY = 70          /* f32 [side_inner]: what a full decay gate takes from log a (>= 0) */
 } b200_stack_weight;
 
 B200_API int b200_stack_create(const b200_stack_cfg* cfg, const b200_stack_layer* layers, b200_ctx** out);
@@ -913,6 +944,45 @@ B200_API int b200_paged_attn_biased(int32_t f32, int32_t form, const float* q, c
  * y_f32: fp32 rows of n_out instead of bf16.  Shapes it cannot address and f32 take the CUDA-core linear. */
 B200_API int b200_linear_bias_act(int32_t f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy,
                                   int32_t n_tokens, int32_t n_out, int32_t k, int32_t act, void* workspace, int64_t ws_bytes, void* stream);
+/* Parallel form with the elementwise norm, between two layers: x[t] += sa ya + sb yb + sum of the n_parts expert rows + sh_gate[t] y_sh
+ * (ya NULL: nothing is added; yb, parts, y_sh, sh_gate optional), then, with out, out = tanh(alpha[0] x) w + b.  rows: row r of the launch
+ * reads stream row rows[r] and the same rows of the other inputs, the stream is not written, out is dense. */
+B200_API int b200_tanh_close(int32_t f32, float* x, const void* ya, float sa, const void* yb, float sb, const float* parts, int32_t n_parts,
+                             const void* y_sh, const float* sh_gate, const float* alpha, const float* w, const float* b, void* out,
+                             const int32_t* rows, int32_t n_rows, int32_t width, void* stream);
+/* Fused rows q | k | v of leading dimension ld -> q and k RMS-normalised over the whole projection times weights of that size, v as it is:
+ * q_out fp32 [T][heads*dim], k and v to the paged caches at slot_mapping[t]. */
+B200_API int b200_qk_norm_cache(int32_t f32, const void* fused, int64_t ld, const float* qw, const float* kw, const int32_t* slot_mapping,
+                                float* q_out, void* k_cache, void* v_cache, int32_t n_tokens, int32_t heads, int32_t kv_heads, int32_t dim,
+                                int32_t vdim, int32_t block_size, float eps, void* stream);
+/* Causal per-channel convolution with bias and without activation: rows x of leading dimension ld -> out [T][width]; tails
+ * [slot][taps - 1][width] fp32, slot_stride floats apart, are read and advanced.  one_row: every sequence brings one row. */
+B200_API int b200_side_conv(int32_t f32, const void* x, int64_t ld, const float* conv, const float* bias, int32_t taps, float* tails,
+                            int64_t slot_stride, const int32_t* positions, const int32_t* row_to_seq, const int32_t* seq_start,
+                            const int32_t* seq_slots, void* out, int32_t n_tokens, int32_t n_seqs, int32_t width, int32_t one_row, void* stream);
+/* Gated linear recurrent unit: u, out [T][width] and y (leading dimension ldy) of the activation type, gates fp32 [T][blocks][2][width / blocks]
+ * (decay gate, input gate) ahead of gate_bias (same order) and sigmoid, decay [width] (log a = -r decay); state [slot][width] fp32. */
+B200_API int b200_gated_lru(int32_t f32, const void* u, const float* gates, const float* gate_bias, const float* decay, const void* y, int64_t ldy,
+                            const int32_t* positions, const int32_t* seq_start, const int32_t* seq_slots, float* state, int64_t slot_stride,
+                            void* out, int32_t n_seqs, int32_t width, int32_t blocks, int32_t one_row, void* stream);
+/* b200_latent_prep in the half layout: dimension i of a rotated part turns with i + rot_dims / 2. */
+B200_API int b200_latent_prep_half(int32_t f32, const void* qkv, int64_t ld, const float* norm_w, const int32_t* positions,
+                                   const int32_t* slot_mapping, const float* rot, int32_t rot_dims, int64_t max_pos, float* qfull, void* cache,
+                                   int32_t n_tokens, int32_t heads, int32_t dim, int32_t rot_dim, int32_t kv_rank, float eps, void* stream);
+/* Router with sigmoid scores: the bias joins the choice only, a group counts by the sum of its group_best (1 or 2) largest choice scores, renorm
+ * divides the chosen weights by their sum; gate_out [T] (optional): sigmoid of one more router row.  logits (optional, bf16 rows):
+ * fp32 scratch [T][experts + 1] for the form whose logits come from the tcgen05 linear. */
+B200_API int b200_moe_route_form(int32_t f32, const void* x, const void* w_router, const float* bias, int32_t n_tokens, int32_t width,
+                                 int32_t experts, int32_t top, int32_t groups, int32_t keep, int32_t group_best, int32_t renorm, float* gate_out,
+                                 float* logits, int32_t* out_ids, float* out_w, void* stream);
+/* Paged attention over a window of `window` keys (0: all) besides the first keep_first, with a distance bias
+ * (dist_bias[h][min(i - j, bias_dist - 1)], NULL: none) and a sink per head (NULL: none).  form, workspace, n_splits and part as in
+ * b200_paged_attn_biased. */
+B200_API int b200_paged_attn_kept(int32_t f32, int32_t form, const float* q, const void* k_cache, const void* v_cache, const int32_t* block_table,
+                                  int32_t bt_stride, const int32_t* row_to_seq, const int32_t* ctx_lens, const int32_t* positions, void* out,
+                                  int32_t n_tokens, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t block_size, float scale,
+                                  int32_t window, int32_t keep_first, const float* sink, const float* dist_bias, int32_t bias_dist, void* workspace,
+                                  int32_t n_splits, float* part, void* stream);
 /* y[T][n_out] = x[T][k] . w[n_out][k]^T on CUDA cores in true fp32; w bf16, x / y fp32 or bf16. */
 B200_API int b200_linear_simt(int32_t x_f32, int32_t y_f32, const void* x, int64_t ldx, const void* w, void* y, int64_t ldy,
                      int32_t n_tokens, int32_t n_out, int32_t k, void* stream);
