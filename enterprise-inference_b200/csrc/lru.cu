@@ -4,8 +4,8 @@
 // u: convolved inputs, y: the other branch's projection, both of the activation type; gates, decays and S fp32.
 //
 //  * step kernel (every sequence brings one row): a thread per channel; the state is read ahead of the dependency wait.
-//  * scan kernel: the recurrence is linear, so a run of rows acts on the state as S -> A S + B.  A CTA takes 16 channels of one
-//    sequence and walks it in tiles of 32 segments x kLruRows rows: a thread folds its segment of one channel into (A, B), one warp
+//  * scan kernel: the recurrence is linear, so a run of rows acts on the state as S -> S - M S + B (M = 1 - the product of its decays).  A CTA takes 16 channels of one
+//    sequence and walks it in tiles of 32 segments x kLruRows rows: a thread folds its segment of one channel into (M, B), one warp
 //    per channel scans the 32 pairs with shuffles and hands every segment the state ahead of it, and the threads run their rows once
 //    more from there.  The next tile's inputs are requested before the barriers of this one.
 // A sequence whose first row of the step is at position 0 starts from zeros, whatever the slot held.
@@ -121,18 +121,18 @@ lru_scan_kernel(const LruArgs<AT> p) {
   };
   fetch(0);
   for (int b0 = 0; b0 < n_rows; b0 += kTile) {
-    float m[kLruRows], b[kLruRows], y[kLruRows], A = 1.0f, B = 0.f;
+    float m[kLruRows], b[kLruRows], y[kLruRows], M = 0.f, B = 0.f;   // the segment: S -> S - M S + B
     const int r0 = b0 + seg * kLruRows;
 #pragma unroll
     for (int k = 0; k < kLruRows; ++k) {
       lru_terms<AT>(zr[k] + br, zi[k] + bi, d, ldf(ur[k]), m[k], b[k]);
       if (r0 + k >= n_rows) m[k] = b[k] = 0.f;
       y[k] = ldf(yr[k]);
-      A = fmaf(-m[k], A, A);
+      M = lru_move(M, m[k], m[k]);
       B = lru_move(B, m[k], b[k]);
     }
     if (b0 + kTile < n_rows) fetch(b0 + kTile);
-    ab[ch][seg] = make_float2(A, B);
+    ab[ch][seg] = make_float2(M, B);
     __syncthreads();
     {
       float2 f = ab[warp][lane];
@@ -140,11 +140,11 @@ lru_scan_kernel(const LruArgs<AT> p) {
       for (int o = 1; o < 32; o <<= 1) {   // inclusive: the map of segments 0 .. lane
         const float pa = __shfl_up_sync(0xffffffffu, f.x, o), pb = __shfl_up_sync(0xffffffffu, f.y, o);
         if (lane >= o) {
-          f.y = fmaf(f.x, pb, f.y);
-          f.x *= pa;
+          f.y = lru_move(pb, f.x, f.y);
+          f.x = lru_move(pa, f.x, f.x);
         }
       }
-      const float after = fmaf(f.x, carry, f.y), before = __shfl_up_sync(0xffffffffu, after, 1);
+      const float after = lru_move(carry, f.x, f.y), before = __shfl_up_sync(0xffffffffu, after, 1);
       sin_[warp][lane] = lane == 0 ? carry : before;
       carry = __shfl_sync(0xffffffffu, after, 31);
     }
