@@ -762,6 +762,48 @@ def _rudolix_like_bofusun(Cf, name, z):
                             layers=layers * z["pairs"])
 
 
+# Rirusun beside Dupolorn (the closest model of the framework: the same parallel layer form, latent attention, matrix-memory
+# recurrence and routed experts with a shared one on the same kernels) at equal width, heads, head sizes, latent size, experts and
+# expert width.  Rirusun's layers cycle the matrix memory, latent attention and the pair of windowed attention and recurrent unit, all with
+# routed experts; Dupolorn's cycle the matrix memory, latent attention and latent attention with sink and gate, all with routed
+# experts.  A third arm, Bofusun's pair of attention and selective scan (dense feed-forwards of top x expert width), is the like of
+# the pair.  Windows are wider than every context of the comparison.
+RIRUSUN_SIZES = {
+    "w2048-e32": dict(width=2048, heads=16, kv=4, dim=128, rot_dim=64, vdim=128, kv_rank=512, r_heads=8, r_dim=128, r_vdim=256, lru=4096, blocks=16,
+                      conv=4, window=4096, experts=32, top=4, groups=4, keep=2, ff=1024, shared=1024, layers=3, vocab=32768),
+    "w1024-e16": dict(width=1024, heads=16, kv=4, dim=64, rot_dim=32, vdim=64, kv_rank=256, r_heads=4, r_dim=128, r_vdim=256, lru=2048, blocks=16,
+                      conv=4, window=4096, experts=16, top=2, groups=4, keep=2, ff=1024, shared=1024, layers=3, vocab=32768),
+}
+
+
+def _rirusun_config(Cf, name, z):
+    rot = Cf.RotarySpec(base=10000.0, dims=z["rot_dim"], factor=4.0, original=4096, fast=32.0, slow=1.0, scaled=True)
+    moe = Cf.FeedForwardSpec(kind="moe", ff=z["ff"], act="gelu_erf", experts=z["experts"], top=z["top"], gated=False, groups=z["groups"], keep=z["keep"],
+                             group_best=2, renorm=True, weight_input=False, shared_ff=z["shared"], shared_gate=True)
+    mixers = [dict(mixer=Cf.MLSTMSpec(heads=z["r_heads"], dim=z["r_dim"], vdim=z["r_vdim"], gate_cap=15.0)),
+              dict(mixer=Cf.LatentAttentionSpec(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"],
+                                                scale=(z["dim"] + z["rot_dim"]) ** -0.5, rot=rot, rot_half=True)),
+              dict(mixer=Cf.AttentionSpec(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["vdim"], scale=z["dim"] ** -0.5, window=z["window"],
+                                          keep_first=4, bias_max=1024.0, sink=True),
+                   side=Cf.GatedLRUSpec(inner=z["lru"], blocks=z["blocks"], conv=z["conv"]), side_mix=(0.7, 0.7))]
+    return Cf.RirusunConfig(name=name, width=z["width"], vocab=z["vocab"], layers=[Cf.StackLayerSpec(mlp=moe, **mixers[i % 3]) for i in range(z["layers"])])
+
+
+def _dupolorn_like_rirusun(Cf, name, z):
+    rot = Cf.RotarySpec(base=10000.0, dims=z["rot_dim"])
+    la = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"], scale=(z["dim"] + z["rot_dim"]) ** -0.5, rot=rot)
+    mixers = [Cf.MLSTMSpec(heads=z["r_heads"], dim=z["r_dim"], vdim=z["r_vdim"], gate_cap=15.0), Cf.LatentAttentionSpec(**la),
+              Cf.LatentAttentionSpec(sink=True, gate=True, **la)]
+    moe = Cf.FeedForwardSpec(kind="moe", ff=z["ff"], act="relu2", experts=z["experts"], top=z["top"], shared_ff=z["shared"])
+    return Cf.DupolornConfig(name=name, width=z["width"], vocab=z["vocab"], embed_scale=1.0, canon_taps=4, bigram_buckets=0, logit_softcap=0.0,
+                             layers=[Cf.ParallelLayerSpec(mixer=mixers[i % 3], mlp=moe) for i in range(z["layers"])])
+
+
+def _bofusun_like_rirusun(Cf, name, z):
+    return _bofusun_config(Cf, name, dict(width=z["width"], heads=z["heads"], kv=z["kv"], dim=z["dim"], r_heads=z["heads"], r_dim=128, r_vdim=128, inner=z["lru"],
+                                          state=16, dt_rank=z["width"] // 16, conv=z["conv"], window=z["window"], ff=z["top"] * z["ff"], pairs=1, vocab=z["vocab"]))
+
+
 def _design_batch(R, n_seqs, ctx, n_new, bs, vocab):
     """n_seqs sequences that already hold ctx tokens and bring n_new rows each; the last row of each is a logit row."""
     import numpy as np
@@ -811,8 +853,8 @@ def run_design(args):
     sampler.start()
     t0 = time.monotonic()
     out = []
-    dup, fut, rud, bof = (args.design == n for n in ("dupolorn", "futidra", "rudolix", "bofusun"))
-    sizes = BOFUSUN_SIZES if bof else RUDOLIX_SIZES if rud else (FUTIDRA_SIZES if fut else (DUPOLORN_SIZES if dup else DESIGN_SIZES))
+    dup, fut, rud, bof, rir = (args.design == n for n in ("dupolorn", "futidra", "rudolix", "bofusun", "rirusun"))
+    sizes = RIRUSUN_SIZES if rir else BOFUSUN_SIZES if bof else RUDOLIX_SIZES if rud else (FUTIDRA_SIZES if fut else (DUPOLORN_SIZES if dup else DESIGN_SIZES))
     names = [n for n in sizes if args.design_size in ("all", n)]
     for name in names:
         z = sizes[name]
@@ -830,7 +872,9 @@ def run_design(args):
             z = {k: v for k, v in z.items() if k not in ("groups", "keep")}
         arms = {"bopilorn": Cf.BopilornConfig(name=name, width=z["width"], vocab=z["vocab"], embed_scale=1.0,
                                               layers=[Cf.StackLayerSpec(mixer=att, mlp=moe) for _ in range(z["layers"])])}
-        if bof:
+        if rir:
+            arms = {"rirusun": _rirusun_config(Cf, name, z), "dupolorn": _dupolorn_like_rirusun(Cf, name, z), "bofusun": _bofusun_like_rirusun(Cf, name, z)}
+        elif bof:
             z = dict(sizes[name])
             arms = {"bofusun": _bofusun_config(Cf, name, z), "rudolix": _rudolix_like_bofusun(Cf, name, z)}
         elif rud:
@@ -863,8 +907,9 @@ def run_design(args):
             torch.cuda.empty_cache()
         out.append(rec)
     clocks = sampler.stop(t0, time.monotonic())
-    emit({"metric": "design_compare", "design": "Bofusun" if bof else "Rudolix" if rud else ("Futidra" if fut else ("Dupolorn" if dup else "Bopilorn")),
-          "closest": "rudolix with one stream (attention with a value cache, delta rule and state-space recurrence with state slots, ungated dense feed-forwards)"
+    emit({"metric": "design_compare", "design": "Rirusun" if rir else "Bofusun" if bof else "Rudolix" if rud else ("Futidra" if fut else ("Dupolorn" if dup else "Bopilorn")),
+          "closest": "dupolorn with routed experts in every layer (parallel form, latent attention, matrix memory); bofusun: the like of the pair of mixers"
+                     if rir else "rudolix with one stream (attention with a value cache, delta rule and state-space recurrence with state slots, ungated dense feed-forwards)"
                      if bof else "futidra (attention with a value cache, delta rule on the same scan, state slots, dense feed-forwards)" if rud else
                      "dupolorn with dense feed-forwards (latent attention, matrix-memory recurrence, state slots)" if fut else
                      ("bopilorn (layer-list model with routed experts)" if dup else "llama (fixed decoder stack)"), "dtype": "bf16",
@@ -881,10 +926,10 @@ def main():
     ap.add_argument("--workload", default="llama8b-bs64", choices=sorted(WORKLOADS))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--headline-only", action="store_true", help="skip the `also` and `tp` sections of the default run")
-    ap.add_argument("--design", default=None, choices=["bopilorn", "dupolorn", "futidra", "rudolix", "bofusun"],
+    ap.add_argument("--design", default=None, choices=["bopilorn", "dupolorn", "futidra", "rudolix", "bofusun", "rirusun"],
                     help="instead of the default workload: prefill / decode throughput of this design beside the closest fixed-stack "
                          "model at equal size")
-    ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(DESIGN_SIZES) | set(DUPOLORN_SIZES) | set(FUTIDRA_SIZES) | set(RUDOLIX_SIZES) | set(BOFUSUN_SIZES)))
+    ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(DESIGN_SIZES) | set(DUPOLORN_SIZES) | set(FUTIDRA_SIZES) | set(RUDOLIX_SIZES) | set(BOFUSUN_SIZES) | set(RIRUSUN_SIZES)))
     args = ap.parse_args()
     claim_stdout()
     if args.design:
