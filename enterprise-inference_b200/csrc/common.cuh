@@ -90,6 +90,14 @@ __device__ __forceinline__ float act_apply(float z, int kind) {
   }
   return z / (1.0f + expf(-z));
 }
+// exact gelu for sums that are rounded to bf16 next: gelu(z) = max(z, 0) - |z| erfc(|z| / sqrt 2) / 2 with the rational approximation
+// of erfc by Hastings (Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26; absolute error below 1.5e-7) on the
+// hardware's exponential and reciprocal
+__device__ __forceinline__ float gelu_erf_fast(float z) {
+  const float x = 0.7071067811865476f * fabsf(z), t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+  const float q = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  return fmaf(-0.5f * fabsf(z) * q, __expf(-x * x), fmaxf(z, 0.f));
+}
 // gate and up value of a gated feed-forward -> the activated product.  B200_ACT_SWIGLU_CLAMP: g = min(g, limit),
 // u = clamp(u, -limit, limit), g * sigmoid(1.702 g) * (u + 1)
 __device__ __forceinline__ float gate_combine(float g, float u, int kind, float limit) {

@@ -241,6 +241,9 @@ __device__ __forceinline__ void finalize4(const TcParams& p, int m_tile, int lan
       const float r[4] = {fmaxf(a.x + bb[0], 0.f), fmaxf(a.y + bb[1], 0.f), fmaxf(a.z + bb[2], 0.f), fmaxf(a.w + bb[3], 0.f)};
 #pragma unroll
       for (int e = 0; e < 4; ++e) v[e] = r[e] * r[e];
+    } else if (p.post_act == 1 + B200_ACT_GELU_ERF) {
+      v[0] = gelu_erf_fast(a.x + bb[0]), v[1] = gelu_erf_fast(a.y + bb[1]);
+      v[2] = gelu_erf_fast(a.z + bb[2]), v[3] = gelu_erf_fast(a.w + bb[3]);
     } else if (p.post_act) {
       v[0] = act_apply(a.x + bb[0], p.post_act - 1), v[1] = act_apply(a.y + bb[1], p.post_act - 1);
       v[2] = act_apply(a.z + bb[2], p.post_act - 1), v[3] = act_apply(a.w + bb[3], p.post_act - 1);

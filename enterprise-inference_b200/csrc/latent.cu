@@ -203,6 +203,104 @@ head_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx_, int x_
   }
 }
 
+// Long steps (128 rows and more, 16-byte addressable rows): 128 x 128 tiles, inner chunks of 64 in two cp.async stages, so that a
+// chunk travels while the one before is multiplied.  Eight warps in 4 x 2, each 32 rows x 64 outputs.  Rows, outputs and inner
+// columns past the end are zero-filled.
+constexpr int kHtTile = 128, kHtChunk = 64, kHtStride = kHtChunk + 8, kHtThreads = 256;
+constexpr int kHtSmem = 2 * 2 * kHtTile * kHtStride * 2;
+
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(live ? 16 : 0));
+}
+
+template <typename YT>
+__global__ void __launch_bounds__(kHtThreads, 2)
+head_linear_tile_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx_, int x_hs, const __nv_bfloat16* __restrict__ w, YT* __restrict__ y,
+                        int64_t ldy, int y_hs, const __nv_bfloat16* __restrict__ gate, int64_t ldg, int g_hs, int g_es, int T, int n_out, int k,
+                        int pairs) {
+  extern __shared__ __align__(16) __nv_bfloat16 hts[];   // [2 stages][X tile | W tile][128][72]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * kHtTile, h = blockIdx.y, o0 = blockIdx.z * kHtTile;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wr = warp & 3, wc = warp >> 2;
+  const __nv_bfloat16* xh = x + (int64_t)h * x_hs;
+  const __nv_bfloat16* wh = w + (int64_t)h * n_out * k;
+  auto stage = [&](int c, int buf) {
+    __nv_bfloat16* Xs = hts + buf * 2 * kHtTile * kHtStride;
+    __nv_bfloat16* Ws = Xs + kHtTile * kHtStride;
+#pragma unroll
+    for (int i = 0; i < kHtTile * (kHtChunk / 8) / kHtThreads; ++i) {
+      const int e = tid + kHtThreads * i, r = e / (kHtChunk / 8), col = (e % (kHtChunk / 8)) * 8, kk = c * kHtChunk + col;
+      const bool in = kk < k;
+      cp_async16_or_zero(Xs + r * kHtStride + col, xh + (int64_t)min(t0 + r, T - 1) * ldx_ + (in ? kk : 0), in && t0 + r < T);
+      cp_async16_or_zero(Ws + r * kHtStride + col, wh + (int64_t)min(o0 + r, n_out - 1) * k + (in ? kk : 0), in && o0 + r < n_out);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float acc[2][8][4];
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+  const int nc = (k + kHtChunk - 1) / kHtChunk;
+  stage(0, 0);
+  for (int c = 0; c < nc; ++c) {
+    if (c + 1 < nc) {
+      stage(c + 1, (c + 1) & 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const __nv_bfloat16* Xs = hts + (c & 1) * 2 * kHtTile * kHtStride;
+    const __nv_bfloat16* ap = Xs + (wr * 32 + (lane & 15)) * kHtStride + (lane >> 4) * 8;
+    const __nv_bfloat16* bp = Xs + kHtTile * kHtStride + (wc * 64 + (lane & 7) + (lane >> 4) * 8) * kHtStride + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int kk = 0; kk < kHtChunk; kk += 16) {
+      uint32_t a[2][4];
+      ldsm_x4(a[0], ap + kk);
+      ldsm_x4(a[1], ap + 16 * kHtStride + kk);
+#pragma unroll
+      for (int n2 = 0; n2 < 4; ++n2) {
+        uint32_t b[4];
+        ldsm_x4(b, bp + n2 * 16 * kHtStride + kk);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16(acc[i][2 * n2][0], acc[i][2 * n2][1], acc[i][2 * n2][2], acc[i][2 * n2][3], a[i], b[0], b[1]);
+          mma_bf16(acc[i][2 * n2 + 1][0], acc[i][2 * n2 + 1][1], acc[i][2 * n2 + 1][2], acc[i][2 * n2 + 1][3], a[i], b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = t0 + wr * 32 + i * 16 + (lane >> 2) + half * 8;
+      if (t >= T) continue;
+      YT* dst = y + (int64_t)t * ldy + (int64_t)h * y_hs;
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) {
+        const int o = o0 + wc * 64 + nt * 8 + (lane & 3) * 2;
+        if (o >= n_out) continue;
+        float v[2] = {acc[i][nt][half * 2], acc[i][nt][half * 2 + 1]};
+        if (gate) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+            if (o + e < n_out) v[e] *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(int64_t)t * ldg + (int64_t)h * g_hs + (int64_t)(o + e) * g_es])));
+        }
+        if (pairs) {
+          if constexpr (sizeof(YT) == 4) *reinterpret_cast<float2*>(dst + o) = make_float2(v[0], v[1]);
+          else *reinterpret_cast<__nv_bfloat162*>(dst + o) = __floats2bfloat162_rn(v[0], v[1]);
+        } else {
+          stx<YT>(dst, o, v[0]);
+          if (o + 1 < n_out) stx<YT>(dst, o + 1, v[1]);
+        }
+      }
+    }
+}
+
 }  // namespace
 
 int latent_prep(bool f32, const void* qkv, int64_t ld, const float* norm_w, const int32_t* positions, const int32_t* slots,
@@ -240,6 +338,22 @@ int head_linear(bool f32, bool y_f32, const void* x, int64_t ldx_, int x_hs, con
   static const int mma_env = getenv("B200_HEAD_LINEAR_MMA") ? atoi(getenv("B200_HEAD_LINEAR_MMA")) : 1;
   if (!f32 && mma_env && k % 16 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0) {
     const bool vec = ldx_ % 8 == 0 && x_hs % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0;
+    static const int tile_env = getenv("B200_HEAD_LINEAR_TILE") ? atoi(getenv("B200_HEAD_LINEAR_TILE")) : 1;
+    if (tile_env && vec && T >= kHtTile && n_out >= kHtTile / 2) {
+      const int pairs = n_out % 2 == 0 && ldy % 2 == 0 && y_hs % 2 == 0 && reinterpret_cast<uintptr_t>(y) % 8 == 0;
+      const dim3 grid((T + kHtTile - 1) / kHtTile, heads, (n_out + kHtTile - 1) / kHtTile), block(kHtThreads);
+      static bool done[2][64] = {};
+      if (y_f32) {
+        B200_CUDA(ensure_dynamic_smem(head_linear_tile_kernel<float>, kHtSmem, done[0]));
+        B200_CUDA(launch(head_linear_tile_kernel<float>, grid, block, (size_t)kHtSmem, s, (const __nv_bfloat16*)x, ldx_, x_hs, w, (float*)y, ldy, y_hs,
+                         (const __nv_bfloat16*)gate, ldg, g_hs, g_es, T, n_out, k, pairs));
+      } else {
+        B200_CUDA(ensure_dynamic_smem(head_linear_tile_kernel<__nv_bfloat16>, kHtSmem, done[1]));
+        B200_CUDA(launch(head_linear_tile_kernel<__nv_bfloat16>, grid, block, (size_t)kHtSmem, s, (const __nv_bfloat16*)x, ldx_, x_hs, w,
+                         (__nv_bfloat16*)y, ldy, y_hs, (const __nv_bfloat16*)gate, ldg, g_hs, g_es, T, n_out, k, pairs));
+      }
+      return B200_OK;
+    }
     const dim3 grid((T + kHmRows - 1) / kHmRows, heads, (n_out + kHmOuts - 1) / kHmOuts), block(128);
 #define HM(YT, VEC)                                                                                                               \
   B200_CUDA(launch(head_linear_mma_kernel<YT, VEC>, grid, block, (size_t)0, s, (const __nv_bfloat16*)x, ldx_, x_hs, w, (YT*)y, ldy, y_hs, \

@@ -184,6 +184,26 @@ def test_convolution_without_activation_in_portions_with_dirty_slots(f32, taps, 
     assert float((state[1] - 9.0).abs().max()) == 0.0
 
 
+@pytest.mark.parametrize("y_f32,gated", [(1, 0), (0, 1), (0, 0)])
+@pytest.mark.parametrize("T,heads,n_out,k", [(128, 2, 64, 16), (300, 3, 96, 48), (257, 2, 131, 80), (131, 1, 200, 272), (20, 3, 96, 48)])
+def test_block_products_of_long_and_short_steps(y_f32, gated, T, heads, n_out, k):
+    """Per-head (per-block) products on the tensor cores: tiles with ragged rows, outputs and inner chunks; the long form starts at 128 rows."""
+    g = torch.Generator().manual_seed(T + k)
+    x, w = U.bf16_exact(torch.randn(T, heads * k + 8, generator=g)), U.bf16_exact(torch.randn(heads, n_out, k, generator=g) * k ** -0.5)
+    gate = U.bf16_exact(torch.randn(T, heads * n_out + 3, generator=g))
+    ldy = heads * n_out + 5
+    y = torch.full((T, ldy), 7.0, dtype=torch.float32 if y_f32 else torch.bfloat16, device=DEV)
+    check(lib().b200_head_linear(0, y_f32, dev(x, torch.bfloat16).data_ptr(), heads * k + 8, k, dev(w, torch.bfloat16).data_ptr(), y.data_ptr(), ldy, n_out,
+                                 dev(gate, torch.bfloat16).data_ptr() if gated else None, heads * n_out + 3, n_out, T, heads, n_out, k, None))
+    sync()
+    want = torch.einsum("thk,hok->tho", x[:, :heads * k].double().view(T, heads, k), w.double())
+    if gated:
+        want = want * torch.sigmoid(gate[:, :heads * n_out].double().view(T, heads, n_out))
+    got = y.float().cpu().double()
+    assert torch.allclose(got[:, :heads * n_out].view(T, heads, n_out), want, **(dict(atol=2e-5, rtol=1e-5) if y_f32 else dict(atol=1e-2, rtol=1e-2)))
+    assert float((got[:, heads * n_out:] - 7.0).abs().max()) == 0.0
+
+
 def _run_lru(f32, seqs, sizes, start_at, slots, bias, decay, blocks, slot_f, state):
     width = decay.shape[0]
     blk, adt = width // blocks, _adt(f32)
